@@ -986,6 +986,180 @@ class ZigolixConfig(ModelConfig):
 _ZIGOLIX_MIXERS = {c.kind: c for c in (SinkAttentionConfig, DiffAttentionConfig)}
 
 
+# --------------------------------------------------------------------------- Zusolix
+
+
+@dataclass(frozen=True)
+class TemperedAttentionConfig:
+    """Grouped-query attention over all earlier keys with biased projections and no rotation: positions enter through a
+    factor on the query, ``1 + coef ln(floor((p + 1) / every) + 1)``; scaled scores capped by ``cap tanh(score / cap)``."""
+
+    kind: ClassVar[str] = "attention"
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    softcap: float | None = None
+    temp_coef: float = 0.0
+    temp_every: int | None = None            # None: no query temperature
+
+    @classmethod
+    def from_dict(cls, m: dict, where: str) -> "TemperedAttentionConfig":
+        temp = _sub(m, "q_temp", where, required=False)
+        return cls(heads=_take(m, "heads", int), kv_heads=_take(m, "kv_heads", int), dim=_take(m, "dim", int),
+                   vdim=_take(m, "vdim", int), scale=_take(m, "scale", float), softcap=_take(m, "softcap", float, None),
+                   temp_coef=0.0 if temp is None else _take(temp, "coef", float),
+                   temp_every=None if temp is None else _take(temp, "every", int))
+
+    def check(self, where: str) -> None:
+        if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1 or self.heads % self.kv_heads:
+            raise ConfigError(f"config.json: {where}sizes must be >= 1 and 'heads' a multiple of 'kv_heads'")
+        if self.softcap is not None and not self.softcap > 0:
+            raise ConfigError(f"config.json: {where}softcap must be > 0, got {self.softcap}")
+        if self.temp_every is not None and self.temp_every < 1:
+            raise ConfigError(f"config.json: {where}q_temp.every must be >= 1, got {self.temp_every}")
+
+    def to_dict(self) -> dict:
+        out: dict = {"dim": self.dim, "heads": self.heads, "kv_heads": self.kv_heads, "scale": self.scale, "vdim": self.vdim}
+        if self.softcap is not None:
+            out["softcap"] = self.softcap
+        if self.temp_every is not None:
+            out["q_temp"] = {"coef": self.temp_coef, "every": self.temp_every}
+        return out
+
+
+@dataclass(frozen=True)
+class MinGRUConfig:
+    """A gated recurrence of ``width`` channels whose gates read the current token only."""
+
+    kind: ClassVar[str] = "mingru"
+    width: int
+
+    @classmethod
+    def from_dict(cls, m: dict, where: str) -> "MinGRUConfig":
+        return cls(width=_take(m, "width", int))
+
+    def check(self, where: str) -> None:
+        if self.width < 1:
+            raise ConfigError(f"config.json: {where}width must be >= 1, got {self.width}")
+
+    def to_dict(self) -> dict:
+        return {"width": self.width}
+
+
+@dataclass(frozen=True)
+class InputWeightedExpertsConfig:
+    """A routed mixture of small gated experts: sigmoid scores, the ``top`` largest chosen, each expert fed with its score
+    times the row; optionally a shared expert that every token takes, times one sigmoid number per token."""
+
+    ff: int
+    experts: int
+    top: int
+    shared_ff: int | None = None
+
+    @classmethod
+    def from_dict(cls, f: dict, where: str) -> "InputWeightedExpertsConfig":
+        e, r = _sub(f, "expert", where), _sub(f, "router", where)
+        sh = _sub(f, "shared", where, required=False)
+        return cls(ff=_take(e, "ff", int), experts=_take(r, "experts", int), top=_take(r, "top", int),
+                   shared_ff=None if sh is None else _take(sh, "ff", int))
+
+    def check(self, where: str) -> None:
+        if self.ff < 1 or self.experts < 1 or not (1 <= self.top <= self.experts) or (self.shared_ff is not None and self.shared_ff < 1):
+            raise ConfigError(f"config.json: {where}sizes must be >= 1 and 1 <= router.top <= router.experts")
+
+    def to_dict(self) -> dict:
+        out: dict = {"expert": {"ff": self.ff}, "kind": "moe", "router": {"experts": self.experts, "top": self.top}}
+        if self.shared_ff is not None:
+            out["shared"] = {"ff": self.shared_ff}
+        return out
+
+
+@dataclass(frozen=True)
+class ZusolixLayer:
+    type: str                                   # "attention" or "mingru"
+    mixer: "TemperedAttentionConfig | MinGRUConfig"
+    ff: "int | InputWeightedExpertsConfig | None"       # inner width of the dense gated feed-forward; routed experts; none
+
+
+@dataclass(frozen=True)
+class ZusolixConfig(ModelConfig):
+    """Zusolix: layers ``x + m (mixer(norm1(x)) + ff(norm2(x)))`` with RMS norms in groups, whose mixer is attention with a
+    query temperature or a minGRU and whose feed-forward is gated with silu, or routed experts weighted on their inputs
+    beside a gated shared expert; what goes on from a layer is a learned weighted sum of the token rows and all layers'
+    results so far.  A norm, and an output matrix of its own.  ``config.json`` lists the layers in order."""
+
+    architecture: ClassVar[str] = "Zusolix"
+
+    vocab_size: int
+    hidden_size: int
+    norm_eps: float
+    layers: tuple[ZusolixLayer, ...]
+    norm_groups: int = 1
+    residual_mult: float = 1.0
+    embedding_scale: float = 1.0
+    eos_token_id: tuple[int, ...] = field(default_factory=tuple)
+
+    def __post_init__(self) -> None:
+        if self.vocab_size < 1 or self.hidden_size < 1 or not self.layers:
+            raise ConfigError("config.json: 'vocab', 'width' must be >= 1 and 'layers' non-empty")
+        if not self.norm_eps > 0:
+            raise ConfigError(f"config.json: norm 'eps' must be > 0, got {self.norm_eps}")
+        if self.norm_groups < 1 or self.hidden_size % self.norm_groups:
+            raise ConfigError(f"config.json: norm 'groups' must divide the width {self.hidden_size}, got {self.norm_groups}")
+        for i, layer in enumerate(self.layers):
+            layer.mixer.check(f"layers[{i}].mixer.")
+            if isinstance(layer.ff, InputWeightedExpertsConfig):
+                layer.ff.check(f"layers[{i}].mlp.")
+            elif layer.ff is not None and layer.ff < 1:
+                raise ConfigError(f"config.json: layers[{i}].mlp.ff must be >= 1, got {layer.ff}")
+
+    @classmethod
+    def from_dict(cls, raw: dict) -> "ZusolixConfig":
+        layers_raw = raw.get("layers")
+        if not isinstance(layers_raw, list) or not layers_raw:
+            raise ConfigError("config.json: 'layers' must be a non-empty list")
+        layers = []
+        for i, lr in enumerate(layers_raw):
+            where = f"layers[{i}]."
+            kind = lr.get("type") if isinstance(lr, dict) else None
+            if kind not in _ZUSOLIX_MIXERS:
+                raise ConfigError(f"config.json: {where}'type' must be one of {sorted(_ZUSOLIX_MIXERS)}, got {kind!r}")
+            mixer = _ZUSOLIX_MIXERS[kind].from_dict(_sub(lr, "mixer", where), where + "mixer.")
+            mlp = _sub(lr, "mlp", where, required=False)
+            if mlp is None:
+                ff = None
+            elif mlp.get("kind", "dense") == "dense":
+                ff = _take(mlp, "ff", int)
+            elif mlp.get("kind") == "moe":
+                ff = InputWeightedExpertsConfig.from_dict(mlp, where + "mlp.")
+            else:
+                raise ConfigError(f"config.json: {where}mlp.kind must be 'dense' or 'moe', got {mlp.get('kind')!r}")
+            layers.append(ZusolixLayer(kind, mixer, ff))
+        norm, emb = _sub(raw, "norm", ""), _sub(raw, "embedding", "", required=False)
+        eos = raw.get("eos_token_id")
+        eos_ids = () if eos is None else tuple(int(e) for e in (eos if isinstance(eos, (list, tuple)) else [eos]))
+        return cls(vocab_size=_take(raw, "vocab", int), hidden_size=_take(raw, "width", int),
+                   norm_eps=_take(norm, "eps", float), norm_groups=_take(norm, "groups", int, 1), layers=tuple(layers),
+                   residual_mult=_take(raw, "residual_mult", float, 1.0),
+                   embedding_scale=1.0 if emb is None else _take(emb, "scale", float, 1.0), eos_token_id=eos_ids)
+
+    def to_dict(self) -> dict:
+        out: dict = {"architecture": self.architecture, "vocab": self.vocab_size, "width": self.hidden_size,
+                     "norm": {"eps": self.norm_eps, "groups": self.norm_groups}, "residual_mult": self.residual_mult,
+                     "embedding": {"scale": self.embedding_scale}}
+        out["layers"] = [{"type": l.type, "mixer": l.mixer.to_dict(),
+                          "mlp": None if l.ff is None else l.ff.to_dict() if isinstance(l.ff, InputWeightedExpertsConfig)
+                          else {"ff": l.ff, "kind": "dense"}} for l in self.layers]
+        if self.eos_token_id:
+            out["eos_token_id"] = list(self.eos_token_id)
+        return out
+
+
+_ZUSOLIX_MIXERS = {c.kind: c for c in (TemperedAttentionConfig, MinGRUConfig)}
+
+
 def read_config_json(model_dir: str | Path) -> dict:
     path = Path(model_dir) / "config.json"
     if not path.is_file():

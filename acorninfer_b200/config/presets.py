@@ -1,7 +1,7 @@
 """Sizes of published Qwen3 dense models as ``config.json`` dictionaries, for runs with random
 weights (benchmarks, the random-weights mode): no checkpoint is needed to measure at a model's
 layer sizes.  Only the keys the architecture reads are given.  For Kogonex, of which no model is
-published, two size sets with layers as wide as real models have them; the same for Vagulorn and Tedenex."""
+published, two size sets with layers as wide as real models have them; the same for the other designs."""
 
 from __future__ import annotations
 
@@ -133,6 +133,29 @@ def _zigolix(width: int, vocab: int, heads: int, kv_heads: int, ff: int, window:
 PRESETS.update({
     "zigolix-w1024": _zigolix(1024, 32768, heads=8, kv_heads=2, ff=3072, window=1024, experts=16, top=2),
     "zigolix-w2048": _zigolix(2048, 65536, heads=16, kv_heads=4, ff=6144, window=1024, experts=16, top=2),
+})
+
+
+def _zusolix(width: int, vocab: int, heads: int, kv_heads: int, ff: int, gru: int, experts: int, top: int) -> dict:
+    """Layers in the pattern attention with a dense feed-forward, attention, minGRU, attention with routed experts, twice;
+    heads of 128; the routed layers' active width (the chosen experts and the shared one) is ``ff``."""
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": ff // (2 * top)}, "router": {"experts": experts, "top": top}, "shared": {"ff": ff // 2}}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0,
+           "q_temp": {"coef": 0.1, "every": 1024}}
+    layers = []
+    for _ in range(2):
+        layers.append({"type": "attention", "mixer": dict(att), "mlp": dense})
+        layers.append({"type": "attention", "mixer": dict(att), "mlp": moe})
+        layers.append({"type": "mingru", "mixer": {"width": gru}, "mlp": moe})
+        layers.append({"type": "attention", "mixer": dict(att), "mlp": moe})
+    return {"architecture": "Zusolix", "vocab": vocab, "width": width, "norm": {"eps": 1e-5, "groups": 4},
+            "residual_mult": 0.4, "embedding": {"scale": 2.0}, "layers": layers}
+
+
+PRESETS.update({
+    "zusolix-w1024": _zusolix(1024, 32768, heads=8, kv_heads=2, ff=3072, gru=1536, experts=16, top=2),
+    "zusolix-w2048": _zusolix(2048, 65536, heads=16, kv_heads=4, ff=6144, gru=3072, experts=16, top=2),
 })
 
 

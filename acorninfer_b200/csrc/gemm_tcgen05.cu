@@ -56,6 +56,7 @@ struct TcParams {
     int ss_parts, norm_width;
     float eps;
     float glu_limit;         // TC_MODE_SWIGLU_PAIRS: > 0: the capped form, g = min(gate, L), u = clamp(up, -L, L), g sigmoid(1.702 g) (u + 1)
+    const float* row_scale;  // [M] or nullptr: a factor on the product's rows, before the epilogue's function (without ss_in)
     // TC_MODE_ADD_NORM
     float* resid;            // [M, ldr] float32, updated in place
     int64_t ldr;
@@ -283,7 +284,7 @@ __global__ void __launch_bounds__(TC_THREADS) gemm_tcgen05_kernel(const __grid_c
             inv_s[threadIdx.x] = rsqrtf(tot / (float)p.norm_width + p.eps);
         }
     } else if (threadIdx.x < MB) {
-        inv_s[threadIdx.x] = 1.f;
+        inv_s[threadIdx.x] = p.row_scale != nullptr && m0 + (int)threadIdx.x < p.M ? p.row_scale[m0 + threadIdx.x] : 1.f;
     }
     const int col = threadIdx.x;                                      // 128 threads = 128 columns of the tile
     const bool n_ok = n0 + col < p.N;
@@ -561,10 +562,11 @@ extern "C" int acorn_gemm_tc_qkv_rope(const void* x, int64_t ldx, const void* w,
 // A product per expert on tiles of 128 rows: x [slots, K] holds every expert's rows together (offsets [E + 1]),
 // w [E, N, K] contiguous, out [slots, N] or, with swiglu_pairs (weight rows 2i / 2i + 1 = gate / up of output i),
 // silu(gate) * up [slots, N / 2] (glu_limit L > 0: the capped form min(gate, L) sigmoid(1.702 min(gate, L)) (clamp(up, -L, L) + 1)).
-// Rows beyond an expert's last one in its last tile are computed and not stored.
+// Rows beyond an expert's last one in its last tile are computed and not stored.  slot_scale [slots] or null: a factor on
+// the slot's sums, before the activation.
 extern "C" int acorn_grouped_gemm_tcgen05(const void* x, int64_t ldx, const void* w, void* out, int64_t ldo,
                                           const int* offsets, int slots, int E, int N, int K, int swiglu_pairs,
-                                          float glu_limit, cudaStream_t stream) {
+                                          float glu_limit, const float* slot_scale, cudaStream_t stream) {
     if (slots <= 0 || E <= 0 || N <= 0) return 0;
     if (!acorn_gemm_tc_supported(slots, N, K, ldx, K) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return ACORN_ERR_UNSUPPORTED;
     if (swiglu_pairs && N % 2) return ACORN_ERR_UNSUPPORTED;
@@ -574,6 +576,7 @@ extern "C" int acorn_grouped_gemm_tcgen05(const void* x, int64_t ldx, const void
     p.out = out; p.ldo = ldo; p.M = slots; p.N = N; p.K = K; p.out_f32 = 0;
     p.mode = swiglu_pairs ? TC_MODE_SWIGLU_PAIRS : TC_MODE_PLAIN;
     p.glu_limit = glu_limit;
+    p.row_scale = slot_scale;
     p.g_offsets = offsets; p.g_experts = E; p.g_tiles = (int)tiles;
     p.kblocks = (K + TC_BK - 1) / TC_BK;
     CUtensorMap mw, mx;

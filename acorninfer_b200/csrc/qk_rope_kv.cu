@@ -14,6 +14,8 @@
 // order is the other way round: the head is rotated first and then brought to unit root mean square,
 // x <- x * rsqrt(mean(x^2) + eps) over rotated and unrotated entries alike (times w if a weight is given,
 // no weight otherwise); both are the general kernel's.
+// A query temperature (temp_every > 0): the finished queries, and they alone, are multiplied by
+// 1 + temp_coef ln(floor((position + 1) / temp_every) + 1); the general kernel and the one for unrotated heads know it.
 // With write_kv = 0 only the query heads are processed (a layer that reads another
 // layer's cache).  Value heads may have a width of their own (dv; their pages then hold rows of dv),
 // a row of qkv may be wider than its heads (ld elements), and with v_from_k the values are the keys as
@@ -29,6 +31,15 @@
 #include "common.cuh"
 
 #define QK_MAX_TAPS 16
+
+struct QkTemp {
+    float coef;
+    int every;                // 0: no temperature
+};
+
+__device__ __forceinline__ float query_factor(const QkTemp& tp, int pos) {
+    return tp.every > 0 ? fmaf(tp.coef, logf((float)((pos + 1) / tp.every + 1)), 1.f) : 1.f;
+}
 
 struct QkConv {
     const float* w;           // [channels, taps] or null: no convolution
@@ -50,7 +61,7 @@ __global__ void qk_rope_kv_kernel(T* __restrict__ qkv, const float* __restrict__
                                   int table_stride, T* __restrict__ k_pages, T* __restrict__ v_pages,
                                   int tokens, int nq, int nkv, int d, int rot, int pairing, int P,
                                   float eps, int write_kv, int64_t ld, int dv, int v_from_k, QkConv cv,
-                                  T* __restrict__ q_out, int64_t ld_q, float magnitude, int norm_after) {
+                                  T* __restrict__ q_out, int64_t ld_q, float magnitude, int norm_after, QkTemp tp) {
     extern __shared__ float smem[];
     pdl_wait();
     pdl_trigger();
@@ -112,6 +123,7 @@ __global__ void qk_rope_kv_kernel(T* __restrict__ qkv, const float* __restrict__
         }
         return;
     }
+    const float qf = h < nq ? query_factor(tp, pos) : 1.f;
     float ss = 0.f;
     for (int i = lane; i < d; i += 32) {
         const float v = element(i);
@@ -148,7 +160,7 @@ __global__ void qk_rope_kv_kernel(T* __restrict__ qkv, const float* __restrict__
         ss2 = warp_sum(ss2);
         const float inv = rsqrtf(ss2 / (float)d + eps);
         __syncwarp();
-        for (int i = lane; i < d; i += 32) dst[i] = from_float<T>(x[i] * inv * (w ? w[i] : 1.f));
+        for (int i = lane; i < d; i += 32) dst[i] = from_float<T>(x[i] * inv * (w ? w[i] : 1.f) * qf);
         return;
     }
     for (int j = lane; j < half; j += 32) {
@@ -159,10 +171,10 @@ __global__ void qk_rope_kv_kernel(T* __restrict__ qkv, const float* __restrict__
         s *= magnitude;
         c *= magnitude;
         const float a = x[ia], b = x[ib];
-        dst[ia] = from_float<T>(a * c - b * s);
-        dst[ib] = from_float<T>(b * c + a * s);
+        dst[ia] = from_float<T>((a * c - b * s) * qf);
+        dst[ib] = from_float<T>((b * c + a * s) * qf);
     }
-    for (int i = rot + lane; i < d; i += 32) dst[i] = from_float<T>(x[i]);
+    for (int i = rot + lane; i < d; i += 32) dst[i] = from_float<T>(x[i] * qf);
 }
 
 // Rotation of neighbouring pairs, then the norm (norm_after), for heads of up to 128 entries that are multiples of four:
@@ -350,7 +362,7 @@ __global__ void qk_conv_kv_vec_kernel(T* __restrict__ qkv, const float* __restri
                                       const int* __restrict__ page_base, int table_stride, T* __restrict__ k_pages,
                                       T* __restrict__ v_pages, int tokens, int nq, int nkv, int d, int dv, int P,
                                       float eps, int write_kv, int64_t ld, QkConv cv, T* __restrict__ q_out,
-                                      int64_t ld_q, int lph_log2, int tpt) {
+                                      int64_t ld_q, int lph_log2, int tpt, QkTemp tp) {
     pdl_wait();
     pdl_trigger();
     constexpr int PAST = TAPS > 1 ? TAPS - 1 : 1;
@@ -442,6 +454,10 @@ __global__ void qk_conv_kv_vec_kernel(T* __restrict__ qkv, const float* __restri
             }
             T* dst;
             if (h < nq) {
+                if (tp.every > 0) {
+                    const float qf = query_factor(tp, positions[t]);
+                    x = make_float4(x.x * qf, x.y * qf, x.z * qf, x.w * qf);
+                }
                 dst = q_out ? q_out + t * ld_q + chan : qkv + t * ld + chan;
             } else {
                 const int pos = positions[t];
@@ -459,7 +475,7 @@ template <typename T, int TAPS>
 static int launch_conv_vec(T* qkv, const float* q_w, const float* k_w, const int* positions, const int* token_row,
                            const int* block_table, const int* page_base, int table_stride, T* k_pages, T* v_pages,
                            int tokens, int nq, int nkv, int d, int dv, int P, float eps, int write_kv, int64_t ld,
-                           const QkConv& cv, T* q_out, int64_t ld_q, cudaStream_t stream) {
+                           const QkConv& cv, T* q_out, int64_t ld_q, const QkTemp& tp, cudaStream_t stream) {
     const int widest = (write_kv && dv > d) ? dv : d;
     int lph_log2 = 0;
     while ((4 << lph_log2) < widest) ++lph_log2;
@@ -469,7 +485,7 @@ static int launch_conv_vec(T* qkv, const float* q_w, const float* k_w, const int
     const int block = threads >= 256 ? 256 : 128;
     return acorn_launch(qk_conv_kv_vec_kernel<T, TAPS>, dim3((unsigned)((threads + block - 1) / block)), dim3(block), 0,
                         stream, qkv, q_w, k_w, positions, token_row, block_table, page_base, table_stride, k_pages,
-                        v_pages, tokens, nq, nkv, d, dv, P, eps, write_kv, ld, cv, q_out, ld_q, lph_log2, tpt);
+                        v_pages, tokens, nq, nkv, d, dv, P, eps, write_kv, ld, cv, q_out, ld_q, lph_log2, tpt, tp);
 }
 
 static bool qk_aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
@@ -482,8 +498,10 @@ extern "C" int acorn_qk_rope_kv(void* qkv, const float* q_w, const float* k_w, c
                                 const float* conv_w, int taps, const float* bias, float* state,
                                 int64_t slot_stride, int64_t conv_off, const int* row_start, const int* row_slot,
                                 void* q_out, int64_t ld_q, int update_single, float magnitude, int norm_after,
-                                cudaStream_t stream) {
+                                float temp_coef, int temp_every, cudaStream_t stream) {
     if (tokens <= 0) return 0;
+    if (temp_every < 0) return ACORN_ERR_UNSUPPORTED;
+    const QkTemp tp = {temp_coef, temp_every};
     if (d > 1024 || rot > d || (rot & 1) || dv < 1 || dv > 1024 || (v_from_k && dv != d)) return ACORN_ERR_UNSUPPORTED;
     QkConv cv;
     cv.w = conv_w; cv.bias = bias; cv.state = state; cv.slot_stride = slot_stride; cv.conv_off = conv_off;
@@ -494,7 +512,7 @@ extern "C" int acorn_qk_rope_kv(void* qkv, const float* q_w, const float* k_w, c
         return ACORN_ERR_UNSUPPORTED;
     const bool special = magnitude != 1.f || norm_after;            // the general kernel alone knows these
     const bool plain_rows = conv_w == nullptr && bias == nullptr && q_out == nullptr;
-    if (plain_rows && !special && rot == d && pairing == 0 && dv == d && !v_from_k && ld == (int64_t)(nq + 2 * nkv) * d &&
+    if (plain_rows && !special && temp_every == 0 && rot == d && pairing == 0 && dv == d && !v_from_k && ld == (int64_t)(nq + 2 * nkv) * d &&
         (d == 16 || d == 32 || d == 64 || d == 128 || d == 256)) {
 #define ROPE_VEC(G)                                                                                                  \
     ACORN_DISPATCH_DTYPE(dtype, T, return (launch_rope_vec<T, G>((T*)qkv, q_w, k_w, inv_freq, positions, token_row,   \
@@ -510,7 +528,7 @@ extern "C" int acorn_qk_rope_kv(void* qkv, const float* q_w, const float* k_w, c
         }
 #undef ROPE_VEC
     }
-    if (plain_rows && norm_after && pairing == 1 && d % 4 == 0 && d <= 128 && dv == d && ld % 4 == 0 && qk_aligned16(qkv) &&
+    if (plain_rows && norm_after && temp_every == 0 && pairing == 1 && d % 4 == 0 && d <= 128 && dv == d && ld % 4 == 0 && qk_aligned16(qkv) &&
         qk_aligned16(k_pages) && qk_aligned16(v_pages) && qk_aligned16(q_w) && qk_aligned16(k_w)) {
         const int warps = 4;
         const int64_t items = (int64_t)tokens * (write_kv ? (nq + 2 * nkv) : nq);
@@ -520,7 +538,7 @@ extern "C" int acorn_qk_rope_kv(void* qkv, const float* q_w, const float* k_w, c
             (T*)v_pages, tokens, nq, nkv, d, rot, P, eps, write_kv, ld, v_from_k, magnitude));
     }
     const int vec_taps = conv_w ? taps : 0;
-    if (!plain_rows && !special && rot == 0 && !v_from_k && vec_taps <= 4 && d % 4 == 0 && dv % 4 == 0 && d <= 128 && dv <= 128 &&
+    if ((!plain_rows || temp_every) && !special && rot == 0 && !v_from_k && vec_taps <= 4 && d % 4 == 0 && dv % 4 == 0 && d <= 128 && dv <= 128 &&
         ld % 4 == 0 && ld_q % 4 == 0 && slot_stride % 4 == 0 && conv_off % 4 == 0 && qk_aligned16(qkv) &&
         qk_aligned16(q_out) && qk_aligned16(k_pages) && qk_aligned16(v_pages) && qk_aligned16(q_w) &&
         qk_aligned16(k_w) && qk_aligned16(conv_w) && qk_aligned16(bias) && qk_aligned16(state)) {
@@ -528,7 +546,7 @@ extern "C" int acorn_qk_rope_kv(void* qkv, const float* q_w, const float* k_w, c
     ACORN_DISPATCH_DTYPE(dtype, T, return (launch_conv_vec<T, TAPS>((T*)qkv, q_w, k_w, positions, token_row,           \
                                                                      block_table, page_base, table_stride, (T*)k_pages, \
                                                                      (T*)v_pages, tokens, nq, nkv, d, dv, P, eps,       \
-                                                                     write_kv, ld, cv, (T*)q_out, ld_q, stream)))
+                                                                     write_kv, ld, cv, (T*)q_out, ld_q, tp, stream)))
         switch (vec_taps) {
             case 0: CONV_VEC(0); break;
             case 1: CONV_VEC(1); break;
@@ -546,7 +564,7 @@ extern "C" int acorn_qk_rope_kv(void* qkv, const float* q_w, const float* k_w, c
     ACORN_DISPATCH_DTYPE(dtype, T, return acorn_launch(
         qk_rope_kv_kernel<T>, dim3((unsigned)blocks), dim3(warps * 32), smem, stream, (T*)qkv, q_w, k_w, inv_freq,
         positions, token_row, block_table, page_base, table_stride, (T*)k_pages, (T*)v_pages, tokens, nq, nkv, d, rot,
-        pairing, P, eps, write_kv, ld, dv, v_from_k, cv, (T*)q_out, ld_q, magnitude, norm_after));
+        pairing, P, eps, write_kv, ld, dv, v_from_k, cv, (T*)q_out, ld_q, magnitude, norm_after, tp));
     return ACORN_ERR_UNSUPPORTED;
 }
 

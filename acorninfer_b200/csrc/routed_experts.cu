@@ -1,22 +1,25 @@
 // A routed mixture of experts: the router's choice, the grouping of tokens by expert, a matrix
 // product per expert over its tokens, and the weighted sum.
 //
-//   moe_route     per token: s = softmax(z) over all N router outputs; the choice score is s + correction;
-//                 the outputs form `groups` equal groups of neighbours, a group's score is its largest choice
+//   moe_route     per token: s = softmax(z) over all N router outputs, or sigmoid(z) of each; the choice score is
+//                 s + correction (no correction: z itself, in whose order the scores stand); the outputs form `groups` equal groups of neighbours, a group's score is its largest choice
 //                 score, and only outputs of the `keep` best groups can be chosen; the `top` largest choice
 //                 scores win; their weights are s itself, or with `normalize` s over the chosen's sum
 //                 (+ 1e-20).  float32 throughout.
 //   moe_plan      counts per expert, offsets (exclusive sums) and a slot for every (token, choice) pair,
-//                 so that the pairs of an expert are neighbours: slot_token[slot], slot_of[pair].
-//   grouped_gemm  C[slot, :] = A[row(slot), :] W_e^T for the slots of every expert e < E
-//   moe_combine   out[t] = sum_k weight_k * (chosen_k >= E ? x[t] : y[slot_of(t, k)]) (+ extra[t], if given)
+//                 so that the pairs of an expert are neighbours: slot_token[slot], slot_of[pair]; the pairs' weights
+//                 by slot, if asked for.
+//   grouped_gemm  C[slot, :] = A[row(slot), :] W_e^T for the slots of every expert e < E; a factor per slot, if given, on
+//                 the float32 sums before any activation (a weight on an expert's *input*: the product is linear in it)
+//   moe_combine   out[t] = sum_k weight_k * (chosen_k >= E ? x[t] : y[slot_of(t, k)]) (+ extra[t], if given, times the
+//                 sigmoid of a number per token, if given; no weights given: 1)
 //                 (router outputs from E on are identity experts: they return their input)
 #include "mma_helpers.cuh"
 
 // One warp per token.  Ties go to the lower index.
-__global__ void moe_route_kernel(const float* __restrict__ z, const float* __restrict__ correction,
+__global__ void moe_route_kernel(const float* __restrict__ z, int64_t ldz, const float* __restrict__ correction,
                                  int* __restrict__ idx, float* __restrict__ wts, int tokens, int N, int top, int groups,
-                                 int keep, int normalize) {
+                                 int keep, int normalize, int scoring) {
     extern __shared__ float sm[];                       // per warp: s[N], choice[N]
     pdl_wait();
     pdl_trigger();
@@ -25,20 +28,20 @@ __global__ void moe_route_kernel(const float* __restrict__ z, const float* __res
     if (t >= tokens) return;
     float* s = sm + (size_t)warp * 2 * N;
     float* choice = s + N;
-    const float* zr = z + (int64_t)t * N;
+    const float* zr = z + (int64_t)t * ldz;
     float m = -INFINITY;
     for (int i = lane; i < N; i += 32) m = fmaxf(m, zr[i]);
     m = warp_max(m);
     float sum = 0.f;
     for (int i = lane; i < N; i += 32) {
-        const float e = expf(zr[i] - m);
+        const float e = scoring == 1 ? 1.f / (1.f + expf(-zr[i])) : expf(zr[i] - m);
         s[i] = e;
         sum += e;
     }
-    sum = warp_sum(sum);
+    sum = scoring == 1 ? 1.f : warp_sum(sum);
     for (int i = lane; i < N; i += 32) {
         s[i] = s[i] / sum;
-        choice[i] = s[i] + correction[i];
+        choice[i] = correction ? s[i] + correction[i] : zr[i];
     }
     __syncwarp();
     if (groups > 1 && keep < groups) {
@@ -107,9 +110,11 @@ __global__ void moe_route_kernel(const float* __restrict__ z, const float* __res
     }
 }
 
-extern "C" int acorn_moe_route(const float* z, const float* correction, int* idx, float* wts, int tokens, int N, int top,
-                               int groups, int keep, int normalize, cudaStream_t stream) {
+// scoring 0: softmax over the outputs; 1: the sigmoid of each.  correction may be null.
+extern "C" int acorn_moe_route(const float* z, int64_t ldz, const float* correction, int* idx, float* wts, int tokens, int N,
+                               int top, int groups, int keep, int normalize, int scoring, cudaStream_t stream) {
     if (tokens <= 0) return 0;
+    if (scoring < 0 || scoring > 1 || ldz < N) return ACORN_ERR_UNSUPPORTED;
     if (N < 1 || top < 1 || top > N || groups < 1 || groups > 64 || N % groups || keep < 1 || keep > groups || N > 2048)
         return ACORN_ERR_UNSUPPORTED;
     const int warps = 4;
@@ -120,15 +125,16 @@ extern "C" int acorn_moe_route(const float* z, const float* correction, int* idx
         if (e != cudaSuccess) return (int)e;
         configured.mark();
     }
-    return acorn_launch(moe_route_kernel, dim3((tokens + warps - 1) / warps), dim3(32 * warps), smem, stream, z, correction,
-                        idx, wts, tokens, N, top, groups, keep, normalize);
+    return acorn_launch(moe_route_kernel, dim3((tokens + warps - 1) / warps), dim3(32 * warps), smem, stream, z, ldz, correction,
+                        idx, wts, tokens, N, top, groups, keep, normalize, scoring);
 }
 
 // One block: histogram of the chosen outputs, exclusive sums, then a slot for every pair.  Within an
 // expert the slots are handed out in whatever order the threads arrive: a row's result does not
 // depend on its slot.
 __global__ void moe_plan_kernel(const int* __restrict__ idx, int* __restrict__ offsets, int* __restrict__ slot_of,
-                                int* __restrict__ slot_token, int pairs, int N, int top) {
+                                int* __restrict__ slot_token, int pairs, int N, int top,
+                                const float* __restrict__ wts, float* __restrict__ slot_wts) {
     extern __shared__ int cnt[];                        // [N] counts, then [N] cursors
     pdl_wait();
     pdl_trigger();
@@ -151,15 +157,17 @@ __global__ void moe_plan_kernel(const int* __restrict__ idx, int* __restrict__ o
         const int slot = atomicAdd(&cursor[idx[i]], 1);
         slot_of[i] = slot;
         slot_token[slot] = i / top;
+        if (slot_wts) slot_wts[slot] = wts[i];
     }
 }
 
+// slot_wts [pairs], if given, receives the pairs' weights (wts) by slot
 extern "C" int acorn_moe_plan(const int* idx, int* offsets, int* slot_of, int* slot_token, int pairs, int N, int top,
-                              cudaStream_t stream) {
+                              const float* wts, float* slot_wts, cudaStream_t stream) {
     if (pairs <= 0) return 0;
     if (N > 4096) return ACORN_ERR_UNSUPPORTED;
     return acorn_launch(moe_plan_kernel, dim3(1), dim3(1024), (size_t)2 * N * sizeof(int), stream, idx, offsets, slot_of,
-                        slot_token, pairs, N, top);
+                        slot_token, pairs, N, top, wts, slot_wts);
 }
 
 // out[i, :] = x[rows[i], :]: the tokens' rows in the order of the slots, for a product whose operand tiles are
@@ -198,7 +206,8 @@ extern "C" int acorn_gather_rows(const void* x, const int* rows, void* out, int 
 template <typename T>
 __global__ void __launch_bounds__(256) grouped_gemm_kernel(const T* __restrict__ A, int64_t lda, const int* __restrict__ a_rows,
                                                            const T* __restrict__ W, T* __restrict__ C, int64_t ldc,
-                                                           const int* __restrict__ offsets, int E, int N, int K) {
+                                                           const int* __restrict__ offsets, int E, int N, int K,
+                                                           const float* __restrict__ slot_scale) {
     __shared__ float as[GG_BM][GG_BK + 1];
     __shared__ float ws[GG_BN][GG_BK + 1];
     __shared__ int s_e, s_first, s_end;
@@ -262,10 +271,11 @@ __global__ void __launch_bounds__(256) grouped_gemm_kernel(const T* __restrict__
     for (int i = 0; i < 2; ++i) {
         const int slot = first + ty + 16 * i;
         if (slot >= end) continue;
+        const float f = slot_scale ? slot_scale[slot] : 1.f;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx + 16 * j;
-            if (n < N) C[(int64_t)slot * ldc + n] = from_float<T>(acc[i][j]);
+            if (n < N) C[(int64_t)slot * ldc + n] = from_float<T>(acc[i][j] * f);
         }
     }
 }
@@ -286,7 +296,7 @@ __global__ void __launch_bounds__(256) grouped_gemm_tc_kernel(const bf16* __rest
                                                               const int* __restrict__ a_rows, const bf16* __restrict__ W,
                                                               bf16* __restrict__ C, int64_t ldc,
                                                               const int* __restrict__ offsets, int E, int N, int K, int swiglu,
-                                                              float glu_limit) {
+                                                              float glu_limit, const float* __restrict__ slot_scale) {
     extern __shared__ __align__(16) unsigned char gt_smem[];
     bf16* sA = reinterpret_cast<bf16*>(gt_smem);                               // [STAGES][BM][LDS]
     bf16* sW = sA + GT_STAGES * BM * GT_LDS;                                   // [STAGES][BN][LDS]
@@ -389,10 +399,11 @@ __global__ void __launch_bounds__(256) grouped_gemm_tc_kernel(const bf16* __rest
         for (int half = 0; half < 2; ++half) {
             const int slot = first + wm * (BM / WM) + mt * 16 + g + half * 8;
             if (slot >= end) continue;
+            const float f = slot_scale ? slot_scale[slot] : 1.f;
 #pragma unroll
             for (int nt = 0; nt < NT; ++nt) {
                 const int n = n0 + wn * (GT_BN / WN) + nt * 8 + 2 * t;
-                const float v0 = acc[mt][nt][half * 2], v1 = acc[mt][nt][half * 2 + 1];
+                const float v0 = acc[mt][nt][half * 2] * f, v1 = acc[mt][nt][half * 2 + 1] * f;
                 if (swiglu) {
                     // weight rows 2i and 2i + 1 are the gate and the up row of output i: both are this thread's
                     float g = v0, u = v1, z = v0;
@@ -418,7 +429,7 @@ __global__ void __launch_bounds__(256) grouped_gemm_tc_kernel(const bf16* __rest
 template <int BM>
 static int grouped_gemm_tc_launch(const bf16* A, int64_t lda, const int* a_rows, const bf16* W, bf16* C, int64_t ldc,
                                   const int* offsets, int slots, int E, int N, int K, int swiglu, float glu_limit,
-                                  cudaStream_t stream) {
+                                  const float* slot_scale, cudaStream_t stream) {
     const int64_t tiles = (slots + BM - 1) / BM + E;
     if (tiles > 65535) return ACORN_ERR_UNSUPPORTED;
     const size_t smem = (size_t)GT_STAGES * (BM + GT_BN) * GT_LDS * sizeof(bf16);
@@ -429,7 +440,8 @@ static int grouped_gemm_tc_launch(const bf16* A, int64_t lda, const int* a_rows,
         configured.mark();
     }
     dim3 grid((N + GT_BN - 1) / GT_BN, (unsigned)tiles);
-    return acorn_launch(grouped_gemm_tc_kernel<BM>, grid, dim3(256), smem, stream, A, lda, a_rows, W, C, ldc, offsets, E, N, K, swiglu, glu_limit);
+    return acorn_launch(grouped_gemm_tc_kernel<BM>, grid, dim3(256), smem, stream, A, lda, a_rows, W, C, ldc, offsets, E, N, K, swiglu, glu_limit,
+                        slot_scale);
 }
 
 extern "C" int acorn_grouped_gemm_fuses_swiglu(int N, int K, int64_t lda, int dtype) {
@@ -438,26 +450,27 @@ extern "C" int acorn_grouped_gemm_fuses_swiglu(int N, int K, int64_t lda, int dt
 
 // swiglu: W holds, per output i, the gate row 2i and the up row 2i + 1; C [slots, N / 2] receives
 // silu(gate) * up computed from the float32 sums (tensor-core kernel only: see the query above); glu_limit L > 0:
-// the capped form min(gate, L) sigmoid(1.702 min(gate, L)) (clamp(up, -L, L) + 1).
+// the capped form min(gate, L) sigmoid(1.702 min(gate, L)) (clamp(up, -L, L) + 1).  slot_scale [slots] or null: a factor on
+// the slot's sums, before the activation.
 extern "C" int acorn_grouped_gemm(const void* A, int64_t lda, const int* a_rows, const void* W, void* C, int64_t ldc,
                                   const int* offsets, int slots, int E, int N, int K, int dtype, int swiglu, float glu_limit,
-                                  cudaStream_t stream) {
+                                  const float* slot_scale, cudaStream_t stream) {
     if (slots <= 0 || E <= 0 || N <= 0) return 0;
     if (swiglu && !(acorn_grouped_gemm_fuses_swiglu(N, K, lda, dtype) && ((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0))
         return ACORN_ERR_UNSUPPORTED;
     if (dtype == ACORN_DTYPE_BF16 && K % 8 == 0 && lda % 8 == 0 && ((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0) {
         // few rows an expert on average: the small tile (a decode step); else the large one
         if ((int64_t)slots <= (int64_t)16 * E)
-            return grouped_gemm_tc_launch<16>((const bf16*)A, lda, a_rows, (const bf16*)W, (bf16*)C, ldc, offsets, slots, E, N, K, swiglu, glu_limit, stream);
+            return grouped_gemm_tc_launch<16>((const bf16*)A, lda, a_rows, (const bf16*)W, (bf16*)C, ldc, offsets, slots, E, N, K, swiglu, glu_limit, slot_scale, stream);
         if ((int64_t)slots >= (int64_t)256 * E)          // several full tiles an expert: the tall tile (64 x 32 a warp)
-            return grouped_gemm_tc_launch<128>((const bf16*)A, lda, a_rows, (const bf16*)W, (bf16*)C, ldc, offsets, slots, E, N, K, swiglu, glu_limit, stream);
-        return grouped_gemm_tc_launch<64>((const bf16*)A, lda, a_rows, (const bf16*)W, (bf16*)C, ldc, offsets, slots, E, N, K, swiglu, glu_limit, stream);
+            return grouped_gemm_tc_launch<128>((const bf16*)A, lda, a_rows, (const bf16*)W, (bf16*)C, ldc, offsets, slots, E, N, K, swiglu, glu_limit, slot_scale, stream);
+        return grouped_gemm_tc_launch<64>((const bf16*)A, lda, a_rows, (const bf16*)W, (bf16*)C, ldc, offsets, slots, E, N, K, swiglu, glu_limit, slot_scale, stream);
     }
     const int64_t tiles = (slots + GG_BM - 1) / GG_BM + E;       // every expert may end in a partly filled tile
     if (tiles > 65535) return ACORN_ERR_UNSUPPORTED;
     dim3 grid((N + GG_BN - 1) / GG_BN, (unsigned)tiles);
     ACORN_DISPATCH_DTYPE(dtype, T, return acorn_launch(grouped_gemm_kernel<T>, grid, dim3(256), 0, stream, (const T*)A, lda,
-                                                       a_rows, (const T*)W, (T*)C, ldc, offsets, E, N, K));
+                                                       a_rows, (const T*)W, (T*)C, ldc, offsets, E, N, K, slot_scale));
     return ACORN_ERR_UNSUPPORTED;
 }
 
@@ -468,21 +481,22 @@ template <typename T>
 __global__ void moe_combine_kernel(const T* __restrict__ y, const T* __restrict__ x, const int* __restrict__ slot_of,
                                    const int* __restrict__ idx, const float* __restrict__ wts, T* __restrict__ out, int H,
                                    int top, int E, float* __restrict__ resid32, const float* __restrict__ norm_w, float eps,
-                                   const T* __restrict__ extra) {
+                                   const T* __restrict__ extra, const float* __restrict__ extra_z, int64_t ldz) {
     extern __shared__ float row_s[];                    // [H] the row's sums (fused form only)
     __shared__ float scratch[32];
     pdl_wait();
     pdl_trigger();
     const int64_t t = blockIdx.x;
     float ss = 0.f;
+    const float gate = extra_z ? 1.f / (1.f + expf(-extra_z[t * ldz])) : 1.f;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
         float acc = 0.f;
         for (int k = 0; k < top; ++k) {
             const int64_t p = t * top + k;
             const float v = idx[p] >= E ? to_float(x[t * H + i]) : to_float(y[(int64_t)slot_of[p] * H + i]);
-            acc = fmaf(wts[p], v, acc);
+            acc = fmaf(wts ? wts[p] : 1.f, v, acc);
         }
-        if (extra) acc += to_float(extra[t * H + i]);      // what every token takes beside its choices (a shared expert)
+        if (extra) acc = fmaf(gate, to_float(extra[t * H + i]), acc);      // what every token takes beside its choices (a shared expert)
         if (resid32) {
             row_s[i] = acc;
             ss += acc * acc;
@@ -502,12 +516,12 @@ __global__ void moe_combine_kernel(const T* __restrict__ y, const T* __restrict_
 
 extern "C" int acorn_moe_combine(const void* y, const void* x, const int* slot_of, const int* idx, const float* wts, void* out,
                                  int tokens, int H, int top, int E, int dtype, float* resid32, const float* norm_w, float eps,
-                                 const void* extra, cudaStream_t stream) {
+                                 const void* extra, const float* extra_z, int64_t ldz, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     const size_t smem = resid32 ? (size_t)H * sizeof(float) : 0;
     if (smem > 48 * 1024) return ACORN_ERR_UNSUPPORTED;
     ACORN_DISPATCH_DTYPE(dtype, T, return acorn_launch(moe_combine_kernel<T>, dim3(tokens), dim3(256), smem, stream, (const T*)y,
                                                        (const T*)x, slot_of, idx, wts, (T*)out, H, top, E, resid32, norm_w, eps,
-                                                       (const T*)extra));
+                                                       (const T*)extra, extra_z, ldz));
     return ACORN_ERR_UNSUPPORTED;
 }

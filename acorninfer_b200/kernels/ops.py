@@ -109,7 +109,7 @@ class _Sigs:
     acorn_qk_rope_kv = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                         c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
                         c_int, c_int64, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int64, c_int64, c_void_p,
-                        c_void_p, c_void_p, c_int64, c_int, c_float, c_int, c_void_p]
+                        c_void_p, c_void_p, c_int64, c_int, c_float, c_int, c_float, c_int, c_void_p]
     acorn_attention_plain = [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                              c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
                              c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_float, c_int, c_void_p]
@@ -142,16 +142,22 @@ class _Sigs:
                         c_void_p]
     acorn_delta_fold = [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]
     acorn_delta_out = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p]
-    acorn_moe_route = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
-    acorn_moe_plan = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
+    acorn_moe_route = [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                       c_void_p]
+    acorn_moe_plan = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p]
     acorn_grouped_gemm = [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int,
-                          c_int, c_int, c_int, c_float, c_void_p]
+                          c_int, c_int, c_int, c_float, c_void_p, c_void_p]
     acorn_grouped_gemm_fuses_swiglu = [c_int, c_int, c_int64, c_int]
     acorn_grouped_gemm_tcgen05 = [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                  c_float, c_void_p]
+                                  c_float, c_void_p, c_void_p]
     acorn_gather_rows = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
     acorn_moe_combine = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                         c_void_p, c_void_p, c_float, c_void_p, c_void_p]
+                         c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int64, c_void_p]
+    acorn_stream_norm = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
+                         c_int64, c_float, c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                         c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p]
+    acorn_min_gru = [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                     c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p]
     acorn_diff_combine = [c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_int,
                           c_void_p]
     acorn_pair_rows = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
@@ -432,7 +438,7 @@ def qk_rope_kv(qkv: torch.Tensor, q_weight32: torch.Tensor | None, k_weight32: t
                rotary_dim: int, interleaved: bool, eps: float, write_kv: bool = True,
                value_dim: int | None = None, values_from_keys: bool = False, bias32: torch.Tensor | None = None,
                conv: "ShortConv | None" = None, q_out: torch.Tensor | None = None, magnitude: float = 1.0,
-               norm_after: bool = False) -> None:
+               norm_after: bool = False, q_temp: tuple[float, int] | None = None) -> None:
     """Per-head q/k norm, rotary encoding, K/V page write; q is updated in place inside ``qkv``, or written
     to ``q_out`` [T, >= nq d] if that is given.  ``bias32`` (float32, one entry per channel of a row) is added to
     the row first; ``conv`` then runs a short causal convolution over time on every channel (``q_out`` is needed
@@ -441,7 +447,8 @@ def qk_rope_kv(qkv: torch.Tensor, q_weight32: torch.Tensor | None, k_weight32: t
     that width).  ``values_from_keys``: the values are the keys as projected, before norm and rotation; a
     row of ``qkv`` is then ``[q | k]``.  A row may be wider than its heads (further columns are ignored).
     ``magnitude``: a factor on cos and sin.  ``norm_after``: q and k heads are brought to unit root mean square
-    (``eps`` inside the root) after the rotation instead of before it, times their weight if one is given."""
+    (``eps`` inside the root) after the rotation instead of before it, times their weight if one is given.
+    ``q_temp`` (coef, every): the finished queries times ``1 + coef ln(floor((position + 1) / every) + 1)``."""
     _check(qkv, "qkv", None, 2)
     T = qkv.shape[0]
     dv = head_dim if value_dim is None else int(value_dim)
@@ -462,6 +469,8 @@ def qk_rope_kv(qkv: torch.Tensor, q_weight32: torch.Tensor | None, k_weight32: t
             _check(w, n, torch.float32, 1)
             if w.numel() != head_dim:
                 raise KernelError(f"{n} must have head_dim entries")
+    if q_temp is not None and int(q_temp[1]) < 1:
+        raise KernelError(f"qk_rope_kv: q_temp needs every >= 1, got {q_temp}")
     P = 0
     if write_kv:
         _check(k_pages, "k_pages", qkv.dtype, 4)
@@ -501,7 +510,8 @@ def qk_rope_kv(qkv: torch.Tensor, q_weight32: torch.Tensor | None, k_weight32: t
                                _ptr(conv.row_slot) if conv is not None else None,
                                _ptr(q_out), q_out.stride(0) if q_out is not None else 0,
                                1 if (conv is not None and conv.update_single) else 0, float(magnitude),
-                               1 if norm_after else 0, _stream()),
+                               1 if norm_after else 0, float(q_temp[0]) if q_temp is not None else 0.0,
+                               int(q_temp[1]) if q_temp is not None else 0, _stream()),
         "qk_rope_kv")
 
 
@@ -1573,6 +1583,11 @@ def add_layernorm(resid32: torch.Tensor, delta, weight32: torch.Tensor, bias32: 
     H = resid32.shape[1]
     if weight32.numel() != H or (bias32 is not None and bias32.numel() != H):
         raise KernelError(f"norm weight / bias do not have the width {H}")
+    if isinstance(delta, DeltaPair) and not delta.plain:
+        if row_idx is not None:
+            raise KernelError("add_layernorm: a pair that is more than two plain results is settled first")
+        delta.settle(resid32)
+        delta = None
     d1, d2 = (delta.a, delta.b) if isinstance(delta, DeltaPair) else (delta, None)
     for d in (d1, d2):
         if d is not None:
@@ -1594,10 +1609,107 @@ def add_layernorm(resid32: torch.Tensor, delta, weight32: torch.Tensor, bias32: 
 
 class DeltaPair:
     """Two results that are both still to be added to the residual stream (the mixer's and the
-    feed-forward's of a block whose sublayers read the same normed rows)."""
+    feed-forward's of a block whose sublayers read the same normed rows), each times ``scale``.  ``b`` may be None, or
+    the feed-forward's result undone (``ExpertsPending``): both, like a scale other than one, are for
+    ``stream_norm`` alone (``settle`` adds them where nobody else takes them)."""
 
-    def __init__(self, a: torch.Tensor, b: torch.Tensor):
-        self.a, self.b = a, b
+    def __init__(self, a: torch.Tensor | None, b, scale: float = 1.0):
+        self.a, self.b, self.scale = a, b, float(scale)
+
+    @property
+    def plain(self) -> bool:
+        return self.scale == 1.0 and isinstance(self.a, torch.Tensor) and isinstance(self.b, torch.Tensor)
+
+    def settle(self, resid32: torch.Tensor) -> None:
+        stream_norm(resid32, self)
+
+
+@dataclass
+class ExpertsPending:
+    """A routed feed-forward's result before its sum: ``sum_k y[slot_of[t, k]] (+ sigmoid(extra_z[t]) extra[t])``, every
+    choice counted once (its weight went into the expert)."""
+
+    y: torch.Tensor                          # [slots, width]
+    slot_of: torch.Tensor                    # [tokens, choices] int32
+    extra: torch.Tensor | None = None        # [tokens, width]
+    extra_z: torch.Tensor | None = None      # [tokens, 1] float32
+
+
+class NormedStream:
+    """The norms through which the next layer's sublayers read the stream, already taken (nothing is left to add): one
+    tensor per norm that the next block named (``Block.entry_norms``)."""
+
+    def __init__(self, rows: tuple[torch.Tensor, ...]):
+        self.rows = rows
+
+
+def stream_norm(x32: torch.Tensor, delta=None, norms=(), out_dtype: torch.dtype | None = None,
+                rows: torch.Tensor | None = None, history: torch.Tensor | None = None, coef32: torch.Tensor | None = None,
+                x_out: torch.Tensor | None = None) -> tuple[torch.Tensor, ...]:
+    """What lies between two layers, in one kernel (float32): ``v = x32 + scale * (a + b)`` with ``delta`` None, a tensor (a
+    alone) or a ``DeltaPair``; with ``history`` ([>= n + 1, T, W] float32, its first n entries earlier streams) and
+    ``coef32`` [n + 1] the new stream is ``sum_j coef_j history[j] + coef_n v`` and ``history[n]`` becomes v, else it is v;
+    then the RMS norms ``norms`` (up to two of ``(weight32, eps, groups)`` that agree in eps and groups: every one of
+    ``groups`` equal parts of a row over its own root mean square) of it in ``out_dtype``, which are returned.  The new
+    stream goes to ``x_out`` (default: into ``x32``).  With ``rows`` (int32) only the norms of those rows are made and
+    nothing else is written."""
+    _check(x32, "x32", torch.float32, 2)
+    T, H = x32.shape
+    a, b, scale = (delta.a, delta.b, delta.scale) if isinstance(delta, DeltaPair) else (delta, None, 1.0)
+    experts = b if isinstance(b, ExpertsPending) else None
+    if experts is not None:
+        b = None
+    results = [t for t in (a, b, experts.y if experts is not None else None, experts.extra if experts is not None else None)
+               if t is not None]
+    dtype = out_dtype or (results[0].dtype if results else torch.float32)
+    for t in results:
+        _check(t, "pending result", dtype, 2)
+        if t.shape[1] != H or (t.shape[0] != T and not (experts is not None and t is experts.y)):
+            raise KernelError(f"stream_norm: a pending result {tuple(t.shape)} does not fit the stream {tuple(x32.shape)}")
+    top, z = 1, None
+    if experts is not None:
+        _check(experts.slot_of, "slot_of", torch.int32, 2)
+        top, z = experts.slot_of.shape[1], experts.extra_z
+        if experts.slot_of.shape[0] != T or experts.y.shape[0] < T * top or (z is not None and (
+                experts.extra is None or z.dtype != torch.float32 or z.shape != (T, 1) or not z.is_cuda)):
+            raise KernelError("stream_norm: the experts' pending result does not fit")
+    n = 0
+    if (history is None) != (coef32 is None):
+        raise KernelError("stream_norm: a history and its coefficients go together")
+    if coef32 is not None:
+        _check(coef32, "coef", torch.float32, 1)
+        _check(history, "history", torch.float32, 3)
+        n = coef32.numel() - 1
+        if n < 0 or history.shape[0] < n or history.shape[1:] != (T, H):
+            raise KernelError(f"stream_norm: history {tuple(history.shape)} does not hold {n} streams of {tuple(x32.shape)}")
+    if len(norms) > 2 or len({(float(e), int(g)) for _, e, g in norms}) > 1:
+        raise KernelError("stream_norm: at most two norms, of equal eps and groups")
+    eps, groups = (float(norms[0][1]), int(norms[0][2])) if norms else (0.0, 1)
+    for w, _, _ in norms:
+        _check(w, "norm weight", torch.float32, 1)
+        if w.numel() != H or H % groups:
+            raise KernelError(f"stream_norm: weight of {w.numel()} / {groups} groups for a width of {H}")
+    count = T
+    if rows is not None:
+        _check(rows, "rows", torch.int32, 1)
+        count = rows.numel()
+    if x_out is not None:
+        _check(x_out, "x_out", torch.float32, 2)
+        if x_out.shape != x32.shape:
+            raise KernelError("stream_norm: x_out does not fit")
+    writes = rows is None and (bool(results) or coef32 is not None or x_out is not None)
+    dst = (x32 if x_out is None else x_out) if writes else None
+    keep = history[n] if coef32 is not None and rows is None and history.shape[0] > n else None
+    outs = tuple(torch.empty((count, H), dtype=dtype, device=x32.device) for _ in norms)
+    w = [t for t, _, _ in norms] + [None, None]
+    o = list(outs) + [None, None]
+    _ok(lib().acorn_stream_norm(
+        x32.data_ptr(), _ptr(dst), _ptr(rows), _ptr(a), _ptr(b), _ptr(experts.y) if experts is not None else None,
+        _ptr(experts.slot_of) if experts is not None else None, top, _ptr(experts.extra) if experts is not None else None,
+        _ptr(z), z.stride(0) if z is not None else 0, scale, _ptr(history) if n else None, T * H, n, _ptr(keep), _ptr(coef32),
+        _ptr(w[0]), _ptr(o[0]), _ptr(w[1]), _ptr(o[1]), count, H, groups, eps, dtype_code(dtype), _stream()), "stream_norm",
+        f"{n} earlier" if n else "")
+    return outs
 
 
 def add_into(resid32: torch.Tensor, delta: torch.Tensor) -> None:
@@ -1611,8 +1723,12 @@ def add_into(resid32: torch.Tensor, delta: torch.Tensor) -> None:
 
 
 def fold_pair(resid32: torch.Tensor, delta):
-    """A ``DeltaPair`` as one pending result: the first is added to the stream now, the second handed on."""
+    """A ``DeltaPair`` as one pending result: the first is added to the stream now, the second handed on (or both are
+    added now, where they are more than two plain results: None)."""
     if isinstance(delta, DeltaPair):
+        if not delta.plain:
+            delta.settle(resid32)
+            return None
         add_into(resid32, delta.a)
         return delta.b
     return delta
@@ -1764,48 +1880,116 @@ def gated_norm(y32: torch.Tensor, gate: torch.Tensor, weight32: torch.Tensor, ep
     return out
 
 
+# ------------------------------------------------------------------ minimal gated recurrence
+
+GRU_MIN_SEGMENT = 32              # tokens: shorter segments are not worth a second pass
+GRU_MAX_SEGMENTS = 64
+GRU_ENOUGH_BLOCKS = 296           # blocks that keep the device busy (148 SMs, two a piece)
+
+
+def gru_segments(longest_row: int, num_rows: int, width: int) -> tuple[int, int]:
+    """(tokens a segment, segments a row) for ``min_gru``, (0, 1) for rows in one piece.  Rows run side by side with blocks
+    of channels; where those are too few to fill the device and a row is long, rows are cut into segments that run
+    side by side (at the price of a second pass over them)."""
+    blocks = max(1, num_rows) * max(1, -(-width // 512))
+    nseg = min(GRU_MAX_SEGMENTS, longest_row // GRU_MIN_SEGMENT, -(-GRU_ENOUGH_BLOCKS // blocks), 65535 // max(1, num_rows))
+    if nseg < 2:
+        return 0, 1
+    seg = -(-longest_row // nseg)
+    return seg, -(-longest_row // seg)
+
+
+def min_gru(proj: torch.Tensor, bias32: torch.Tensor, state: torch.Tensor, state_off: int, row_start: torch.Tensor,
+            row_slot: torch.Tensor, num_rows: int, longest_row: int = 1) -> torch.Tensor:
+    """``z = sigmoid(proj_z + b_z), u = proj_u + b_u, c = u + 1/2 (u >= 0) or sigmoid(u);  S <- (1 - z) S + z c;  S silu(proj_g)``
+    for every token of every row, from the state in the row's slot (``[width]`` float32 at ``state_off``, updated in
+    place).  proj [T, 3 width] holds ``[z | u | g]``; bias32 [2 width].  ``longest_row``: a bound on the tokens of a row (a
+    host number); long rows run in segments side by side (``gru_segments``).  Returns [T, width] in proj's dtype."""
+    _rows2(proj, "proj")
+    _check(bias32, "bias", torch.float32, 1)
+    _check(state, "state", torch.float32, 2)
+    T, W3 = proj.shape
+    width = W3 // 3
+    if W3 != 3 * width or bias32.numel() != 2 * width or state.shape[1] < state_off + width:
+        raise KernelError(f"min_gru: proj {tuple(proj.shape)}, bias {bias32.numel()}, state {tuple(state.shape)} do not fit")
+    out = torch.empty((T, width), dtype=proj.dtype, device=proj.device)
+    seg, nseg = gru_segments(int(longest_row), num_rows, width)
+    seg_a = seg_b = None
+    if nseg > 1:
+        seg_a = torch.empty((num_rows, nseg, width), dtype=torch.float32, device=proj.device)
+        seg_b = torch.empty((num_rows, nseg + 1, width), dtype=torch.float32, device=proj.device)
+    for pass_ in ((0,) if nseg == 1 else (1, 2)):
+        _ok(lib().acorn_min_gru(proj.data_ptr(), proj.stride(0), bias32.data_ptr(), state.data_ptr(), state.stride(0),
+                                int(state_off), row_start.data_ptr(), row_slot.data_ptr(), out.data_ptr(), num_rows, width,
+                                pass_, seg, nseg, _ptr(seg_a), _ptr(seg_b), dtype_code(proj.dtype), _stream()), "min_gru",
+            f"pass {pass_}")
+    return out
+
+
 # ------------------------------------------------------------------ routed experts
 
 
-def moe_route(z32: torch.Tensor, correction32: torch.Tensor, top: int, groups: int, keep: int, normalize: bool = False):
-    """(chosen [T, top] int32, weights [T, top] float32) from router logits z [T, N].  ``normalize``: the
+MOE_SCORINGS = {"softmax": 0, "sigmoid": 1}
+
+
+def moe_route(z32: torch.Tensor, correction32: torch.Tensor | None, top: int, groups: int, keep: int, normalize: bool = False,
+              scoring: str = "softmax"):
+    """(chosen [T, top] int32, weights [T, top] float32) from router logits z [T, N] (columns of a wider product are
+    allowed).  ``scoring``: an output's score is its softmax, or the sigmoid of its logit.  Outputs are ranked by score +
+    correction; without a correction by the logits, in whose order the scores stand.  ``normalize``: the
     chosen outputs' scores are divided by their sum (+ 1e-20)."""
-    _check(z32, "router logits", torch.float32, 2)
-    _check(correction32, "correction", torch.float32, 1)
+    _rows2(z32, "router logits", torch.float32)
     T, N = z32.shape
-    if correction32.numel() != N:
-        raise KernelError("moe_route: correction must have one entry per router output")
+    if correction32 is not None:
+        _check(correction32, "correction", torch.float32, 1)
+        if correction32.numel() != N:
+            raise KernelError("moe_route: correction must have one entry per router output")
+    if scoring not in MOE_SCORINGS:
+        raise KernelError(f"moe_route: scoring must be one of {sorted(MOE_SCORINGS)}, got {scoring!r}")
     idx = torch.empty((T, top), dtype=torch.int32, device=z32.device)
     wts = torch.empty((T, top), dtype=torch.float32, device=z32.device)
-    _ok(lib().acorn_moe_route(z32.data_ptr(), correction32.data_ptr(), idx.data_ptr(), wts.data_ptr(), T, N, int(top),
-                              int(groups), int(keep), 1 if normalize else 0, _stream()), "moe_route")
+    _ok(lib().acorn_moe_route(z32.data_ptr(), z32.stride(0), _ptr(correction32), idx.data_ptr(), wts.data_ptr(), T, N, int(top),
+                              int(groups), int(keep), 1 if normalize else 0, MOE_SCORINGS[scoring], _stream()), "moe_route")
     return idx, wts
 
 
-def moe_plan(idx: torch.Tensor, num_outputs: int):
+def moe_plan(idx: torch.Tensor, num_outputs: int, wts: torch.Tensor | None = None):
     """Groups the (token, choice) pairs by chosen output: (offsets [N + 1], slot_of [T, top], slot_token
-    [T * top]), all int32."""
+    [T * top]), all int32; with the pairs' weights ``wts`` also these by slot ([T * top] float32)."""
     _check(idx, "idx", torch.int32, 2)
     T, top = idx.shape
     dev = idx.device
     offsets = torch.empty(num_outputs + 1, dtype=torch.int32, device=dev)
     slot_of = torch.empty((T, top), dtype=torch.int32, device=dev)
     slot_token = torch.empty(T * top, dtype=torch.int32, device=dev)
+    slot_wts = None
+    if wts is not None:
+        _check(wts, "wts", torch.float32, 2)
+        if wts.shape != idx.shape:
+            raise KernelError("moe_plan: one weight per choice")
+        slot_wts = torch.empty(T * top, dtype=torch.float32, device=dev)
     _ok(lib().acorn_moe_plan(idx.data_ptr(), offsets.data_ptr(), slot_of.data_ptr(), slot_token.data_ptr(), T * top,
-                             num_outputs, top, _stream()), "moe_plan")
-    return offsets, slot_of, slot_token
+                             num_outputs, top, _ptr(wts), _ptr(slot_wts), _stream()), "moe_plan")
+    return (offsets, slot_of, slot_token) if wts is None else (offsets, slot_of, slot_token, slot_wts)
 
 
 GROUPED_TCGEN05_MIN_ROWS = 64      # rows an expert on average from which the grouped product takes the tcgen05 kernel
 
 
 def grouped_gemm(a: torch.Tensor, a_rows: torch.Tensor | None, w: torch.Tensor, offsets: torch.Tensor, slots: int,
-                 swiglu_pairs: bool = False, activation: str = "silu", limit: float = 0.0) -> torch.Tensor:
+                 swiglu_pairs: bool = False, activation: str = "silu", limit: float = 0.0,
+                 slot_scale: torch.Tensor | None = None) -> torch.Tensor:
     """out[slot] = a[a_rows[slot]] @ w[e]^T for the slots offsets[e] .. offsets[e + 1] - 1 of every
     expert e (w [E, N, K]); rows of other slots are left unwritten.  ``swiglu_pairs``: rows 2i and 2i + 1 of
     ``w[e]`` are the gate and the up row of output i, and what is returned is ``silu(gate) * up``
     [slots, N / 2]: inside the product's epilogue on the tensor-core kernel, by the SwiGLU kernel after it
-    otherwise.  ``activation="capped_swish"`` with ``limit`` L: the capped form instead of silu (see ``swiglu``)."""
+    otherwise.  ``activation="capped_swish"`` with ``limit`` L: the capped form instead of silu (see ``swiglu``).
+    ``slot_scale`` (float32 [slots]): a factor on a slot's product before the activation, which is a factor on the row
+    that entered it."""
+    if slot_scale is not None:
+        _check(slot_scale, "slot_scale", torch.float32, 1)
+        if slot_scale.numel() != slots:
+            raise KernelError("grouped_gemm: one factor per slot")
     if activation not in ("silu", "capped_swish") or (activation == "capped_swish" and not limit > 0):
         raise KernelError(f"grouped_gemm: activation {activation!r} with limit {limit}")
     glu_limit = float(limit) if activation == "capped_swish" else 0.0
@@ -1828,26 +2012,33 @@ def grouped_gemm(a: torch.Tensor, a_rows: torch.Tensor | None, w: torch.Tensor, 
             rows_in = a
         out = torch.empty((slots, N // 2 if swiglu_pairs else N), dtype=a.dtype, device=a.device)
         _ok(lib().acorn_grouped_gemm_tcgen05(rows_in.data_ptr(), rows_in.stride(0), w.data_ptr(), out.data_ptr(), out.stride(0),
-                                             offsets.data_ptr(), slots, E, N, K, 1 if swiglu_pairs else 0, glu_limit, _stream()),
+                                             offsets.data_ptr(), slots, E, N, K, 1 if swiglu_pairs else 0, glu_limit,
+                                             _ptr(slot_scale), _stream()),
             "grouped_gemm_tcgen05", f"{slots}x{N}x{K}")
         return out
     out = torch.empty((slots, N // 2 if fused else N), dtype=a.dtype, device=a.device)
     _ok(lib().acorn_grouped_gemm(a.data_ptr(), a.stride(0), _ptr(a_rows), w.data_ptr(), out.data_ptr(), out.stride(0),
-                                 offsets.data_ptr(), slots, E, N, K, dtype_code(a.dtype), 1 if fused else 0, glu_limit, _stream()),
+                                 offsets.data_ptr(), slots, E, N, K, dtype_code(a.dtype), 1 if fused else 0, glu_limit,
+                                 _ptr(slot_scale), _stream()),
         "grouped_gemm", f"{slots}x{N}x{K}")
     if swiglu_pairs and not fused:
         return swiglu(out, block=1, activation=activation, limit=limit)
     return out
 
 
-def moe_combine(y: torch.Tensor, x: torch.Tensor, slot_of: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor,
+def moe_combine(y: torch.Tensor, x: torch.Tensor, slot_of: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor | None,
                 num_experts: int, resid32: torch.Tensor | None = None, weight32: torch.Tensor | None = None,
-                eps: float = 0.0, extra: torch.Tensor | None = None) -> torch.Tensor | None:
+                eps: float = 0.0, extra: torch.Tensor | None = None, extra_z: torch.Tensor | None = None) -> torch.Tensor | None:
     """out[t] = sum_k wts[t, k] * (idx[t, k] >= num_experts ? x[t] : y[slot_of[t, k]]).  With ``resid32`` the
     float32 sum is not returned but RMS-normed (``weight32``, ``eps``) and added to ``resid32`` in place; what
     is returned is then the new stream rounded to ``x``'s dtype (None if that is float32).  ``extra`` [T, H]: added
-    to every token's sum (what all tokens take beside their choices: a shared expert)."""
+    to every token's sum (what all tokens take beside their choices: a shared expert), times ``sigmoid(extra_z[t])`` if that
+    is given ([T, 1], a column of a wider product).  ``wts`` None: every choice counts once."""
     _check(y, "y", x.dtype, 2)
+    if extra_z is not None:
+        _rows2(extra_z, "extra_z", torch.float32)
+        if extra is None or extra_z.shape != (x.shape[0], 1):
+            raise KernelError("moe_combine: extra_z is one number per token beside extra")
     if extra is not None:
         _check(extra, "extra", x.dtype, 2)
         if extra.shape != x.shape:
@@ -1861,9 +2052,10 @@ def moe_combine(y: torch.Tensor, x: torch.Tensor, slot_of: torch.Tensor, idx: to
         if resid32.shape != x.shape or weight32.numel() != H:
             raise KernelError("moe_combine: residual or norm weight do not fit")
     out = None if (fused and x.dtype == torch.float32) else torch.empty_like(x)
-    _ok(lib().acorn_moe_combine(y.data_ptr(), x.data_ptr(), slot_of.data_ptr(), idx.data_ptr(), wts.data_ptr(), _ptr(out),
+    _ok(lib().acorn_moe_combine(y.data_ptr(), x.data_ptr(), slot_of.data_ptr(), idx.data_ptr(), _ptr(wts), _ptr(out),
                                 T, H, idx.shape[1], int(num_experts), dtype_code(x.dtype), _ptr(resid32), _ptr(weight32),
-                                float(eps), _ptr(extra), _stream()), "moe_combine")
+                                float(eps), _ptr(extra), _ptr(extra_z), extra_z.stride(0) if extra_z is not None else 0,
+                                _stream()), "moe_combine")
     return out
 
 

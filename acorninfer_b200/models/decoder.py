@@ -18,7 +18,7 @@ import torch
 from .. import parts as _parts  # noqa: F401  (registers the built-in part kinds)
 from ..kernels import ops
 from ..parts.base import (BLOCKS, FEED_FORWARDS, LAYER_EXTRAS, MIXERS, NORMS, PASS_ENTRIES, POSITION_ENCODINGS, STAGES,
-                          BuildContext, KVNeeds, ModelSpec, StateNeeds, TensorSpec, build_part)
+                          STREAM_MIXES, BuildContext, KVNeeds, ModelSpec, StateNeeds, TensorSpec, build_part)
 
 
 @dataclass
@@ -70,6 +70,12 @@ class Decoder:
         if spec.pass_entry is not None:
             self.pass_entry = build_part(PASS_ENTRIES, spec.pass_entry, self.ctx)
             self._named_parts.append((spec.pass_entry.prefix, self.pass_entry))
+        self.stream_mix = None
+        if spec.stream_mix is not None:
+            if any(e.opens_pass is not None or e.add_embedding for e in spec.schedule):
+                raise ValueError("a stream mix does not go with schedule entries that take the token rows in again")
+            self.stream_mix = build_part(STREAM_MIXES, spec.stream_mix, self.ctx)
+            self._named_parts.append((spec.stream_mix.prefix, self.stream_mix))
         for i, e in enumerate(spec.schedule):
             if e.opens_pass is not None and self.pass_entry is None:
                 raise ValueError(f"schedule entry {i} opens a pass, but the model names no pass_entry part")
@@ -97,7 +103,7 @@ class Decoder:
 
     def ignorable_tensors(self) -> tuple[str, ...]:
         # A tied model's file may still carry a copy of the output matrix.
-        return ("lm_head.weight",) if self.spec.head is None else ()
+        return (("lm_head.weight",) if self.spec.head is None else ()) + self.spec.ignorable
 
     def bind(self, tensors: dict[str, torch.Tensor]) -> None:
         s = self.spec
@@ -169,9 +175,14 @@ class Decoder:
 
     def forward(self, inputs, caches: list[EntryCache]) -> torch.Tensor | None:
         """Runs the step's tokens; returns float32 logits [wanted, vocab] (None if none wanted)."""
-        resid32 = ops.embed(inputs.token_ids, self.embedding, scale=self.spec.embedding_scale)
+        history = self.stream_mix.open(inputs.num_tokens, self.spec.hidden_size) if self.stream_mix is not None else None
+        resid32 = ops.embed(inputs.token_ids, self.embedding, scale=self.spec.embedding_scale,
+                            out32=history[0] if history is not None else None)
         for stage in self.stages["after_embedding"]:
             resid32 = stage.forward(resid32, inputs)
+        if history is not None:
+            h = self._run_mixed(resid32, history, inputs, caches)
+            return self._head(h, inputs) if h is not None else None
         delta = None
         sched = self.spec.schedule
         # a run that takes the tokens in again adds the stream as it was here
@@ -216,7 +227,40 @@ class Decoder:
             return None
         if isinstance(delta, ops.RoundedRows):          # the last block already added its result
             delta = None
-        h = self.final_norm.add_forward(resid32, delta, rows=inputs.logit_tokens)
+        return self._head(self.final_norm.add_forward(resid32, delta, rows=inputs.logit_tokens), inputs)
+
+    def _run_mixed(self, resid32, history, inputs, caches):
+        """The layer runs of a model whose stream goes on through ``stream_mix``: returns the final norm of the rows whose
+        logits are wanted, or None.  What a run still has to add, the mix of all results so far and the norms through
+        which the next run reads the stream are one call of the mix."""
+        sched = self.spec.schedule
+        if resid32.data_ptr() != history[0].data_ptr():
+            history[0].copy_(resid32)
+        delta, owned = None, False          # X_0 lies in the history: the stream that goes on gets memory of its own
+        for i, e in enumerate(sched):
+            block = self.blocks[e.layer]
+            if not owned and not getattr(block, "leaves_stream", False):
+                resid32, owned = resid32.clone(), True
+            resid32, delta = block.forward(resid32, delta, inputs, caches[i])
+            if isinstance(delta, ops.NormedPending):
+                delta.settle(resid32)
+                delta = None
+            if isinstance(delta, ops.RoundedRows):
+                delta = None
+            x_out = None
+            if not owned:
+                x_out, owned = torch.empty_like(resid32), True
+            if i + 1 < len(sched):
+                resid32, rows = self.stream_mix.forward(history, i, resid32, delta, self.blocks[sched[i + 1].layer].entry_norms(),
+                                                        x_out=x_out)
+                delta = ops.NormedStream(rows) if rows is not None else None
+            elif inputs.num_logits:
+                resid32, rows = self.stream_mix.forward(history, i, resid32, delta, (self.final_norm,), rows=inputs.logit_tokens,
+                                                        x_out=x_out)
+                return rows[0] if rows is not None else self.final_norm.add_forward(resid32, None, rows=inputs.logit_tokens)
+        return None
+
+    def _head(self, h, inputs):
         for stage in self.stages["before_head"]:
             h = stage.forward(h, inputs)
         logits = ops.linear(h, self.head, out_dtype=torch.float32)

@@ -21,7 +21,9 @@ are its state, float32, in its state slot); a penalty on the distance to the key
 (``slope_exponent``); the q/k norm applied after the rotation instead of before it (``norm_after_rotation``) and
 without weights (``qk_norm_weights`` false: the heads are only brought to unit root mean square); a learned sink per
 head, a term ``exp(sink_h)`` in the softmax denominator that has no key and no value (``sink``); a cap on the scaled
-scores, ``cap tanh(score / cap)`` (``softcap``).  A position encoding's factor on cos and sin (``magnitude``) is applied.
+scores, ``cap tanh(score / cap)`` (``softcap``); a query temperature, the finished query of position p times
+``1 + coef ln(floor((p + 1) / every) + 1)`` (``q_temp`` = (coef, every)).  A position encoding's factor on cos and sin
+(``magnitude``) is applied.
 
 All sizes are parameters.  The q, k, v (and gate) matrices are concatenated when bound so that one
 matrix product yields a token's whole row.  A run that reads another run's
@@ -54,7 +56,7 @@ class Attention(Mixer):
                  value_dim: int | None = None, values_from_keys: bool = False, head_gate: bool = False,
                  names: dict | None = None, bias: bool = False, conv_taps: int | None = None,
                  slope_exponent: float | None = None, norm_after_rotation: bool = False, qk_norm_weights: bool = True,
-                 sink: bool = False, softcap: float | None = None):
+                 sink: bool = False, softcap: float | None = None, q_temp: tuple[float, int] | None = None):
         """``names``: the tensors' names relative to the part's prefix (keys q, k, v, o, q_norm, k_norm, gate,
         q_bias, k_bias, v_bias, q_conv, k_conv, v_conv, sink)."""
         if (norm_after_rotation or not qk_norm_weights) and (qk_norm_eps is None or conv_taps or bias):
@@ -63,6 +65,9 @@ class Attention(Mixer):
             raise ValueError("a q/k norm without weights is built for the norm after the rotation only")
         if softcap is not None and (not softcap > 0 or slope_exponent is not None):
             raise ValueError("softcap must be > 0 and does not go with a distance penalty")
+        if q_temp is not None and int(q_temp[1]) < 1:
+            raise ValueError(f"q_temp must give every >= 1, got {q_temp}")
+        self.q_temp = None if q_temp is None else (float(q_temp[0]), int(q_temp[1]))
         if conv_taps is not None and (conv_taps < 1 or values_from_keys):
             raise ValueError("conv_taps must be >= 1 or None, and needs value columns of their own")
         if num_heads % num_kv_heads:
@@ -97,7 +102,8 @@ class Attention(Mixer):
         self.norm_after, self.norm_weights, self.sink, self.softcap = bool(norm_after_rotation), bool(qk_norm_weights), bool(sink), softcap
         self.sink32 = None
         magnitude = getattr(self.position, "magnitude", 1.0) if self.position is not None else 1.0
-        self.plain = (not (values_from_keys or head_gate or bias or conv_taps or self.norm_after or self.sink or softcap)
+        self.plain = (not (values_from_keys or head_gate or bias or conv_taps or self.norm_after or self.sink or softcap
+                           or q_temp is not None)
                       and self.norm_weights and magnitude == 1.0 and self.dv == head_dim)
         self.gate_col = (self.nq + self.nkv) * self.d + (0 if values_from_keys else self.nkv * self.dv)
         self.w_qkv = self.w_o = self.q_norm32 = self.k_norm32 = None
@@ -205,7 +211,7 @@ class Attention(Mixer):
                            pos.rotary_dim if pos is not None else 0, pos.interleaved if pos is not None else False,
                            self.qk_norm_eps if self.qk_norm_eps is not None else 0.0, write_kv=True,
                            value_dim=self.dv, bias32=self.bias32, conv=conv, q_out=qkv,
-                           magnitude=getattr(pos, "magnitude", 1.0) if pos is not None else 1.0)
+                           magnitude=getattr(pos, "magnitude", 1.0) if pos is not None else 1.0, q_temp=self.q_temp)
             if self.taps and self.taps > 1 and inputs.plan.max_q_len > 1:     # rows of one token shifted their memory above
                 ops.conv_state_update(proj, cache.state, 0, inputs.row_start, inputs.row_slot, inputs.num_rows,
                                       self.channels, self.taps, bias32=self.bias32, skip_single=True)
@@ -219,7 +225,7 @@ class Attention(Mixer):
                            self.qk_norm_eps if self.qk_norm_eps is not None else 0.0, write_kv=cache.write,
                            value_dim=self.dv, values_from_keys=self.values_from_keys,
                            magnitude=getattr(pos, "magnitude", 1.0) if pos is not None else 1.0,
-                           norm_after=self.norm_after)
+                           norm_after=self.norm_after, q_temp=self.q_temp)
         heads = attn_kernels.paged_attention(qkv, inputs, g, cache, self.nq, self.nkv, self.d, self.scale, self.window,
                                              chunk=self.chunk, keep_first=self.keep_first, value_dim=self.dv,
                                              slopes32=self.slopes32, sink32=self.sink32, softcap=self.softcap)

@@ -17,6 +17,8 @@ Interfaces
 ``Stage``             ``forward(x, inputs) -> x`` outside the layers (after the token table, around the head)
 ``LayerExtra``        ``forward(resid32, rows, inputs)``: a further sublayer that adds to the stream itself
 ``PassEntry``         ``forward(resid32, entered32, pass_index, inputs) -> resid32``: what opens a pass of a span of layers
+``StreamMix``         ``forward(history, run, x32, delta, norms, rows) -> (x32, normed)``: the stream that goes on from a layer run,
+                      as a function of the results of all runs so far
 
 All activations are ``[tokens, width]`` over the flat token dimension of one step.
 The residual stream is kept in float32 (``resid32``); what a part adds to it
@@ -104,6 +106,8 @@ class ModelSpec:
     after_head: tuple[PartSpec, ...] = ()         # on the float32 logits [wanted, vocab]
     embedding_scale: float = 1.0                  # factor on the token rows as they enter the stream (not on a tied head)
     pass_entry: PartSpec | None = None            # kind of the PASS_ENTRIES registry: runs before entries with ``opens_pass``
+    stream_mix: PartSpec | None = None            # kind of the STREAM_MIXES registry: runs after every layer run
+    ignorable: tuple[str, ...] = ()               # tensors a folder may hold although the model does not read them
     logit_scale: float = 1.0                      # factor on the logits
 
 
@@ -292,6 +296,22 @@ class PassEntry(Part):
         raise NotImplementedError
 
 
+class StreamMix(Part):
+    """The stream that goes on to the next layer run (and after the last run to the output) as a function of the results of
+    all runs so far.  The results are kept for the step (``open``), float32, X_0 the stream as it enters the first layer."""
+
+    def open(self, num_tokens: int, width: int) -> torch.Tensor:
+        """Room for the results of a step: [runs + 1 (or runs), tokens, width] float32; the caller fills entry 0."""
+        raise NotImplementedError
+
+    def forward(self, history: torch.Tensor, run: int, x32: torch.Tensor, delta, norms: tuple["Norm", ...] = (),
+                rows: torch.Tensor | None = None, x_out: torch.Tensor | None = None):
+        """After run ``run``: its result is ``x32`` plus what ``delta`` still adds.  Returns (the stream that goes on, the
+        ``norms`` of it as a tuple, or None where the part did not take them).  ``rows``: only those rows' norms are
+        wanted (the part may then return None for the stream).  ``x_out``: where the stream may go (``x32`` otherwise)."""
+        raise NotImplementedError
+
+
 class Block(Part):
     """Arrangement of a mixer, a feed-forward and norms around the residual stream."""
 
@@ -313,6 +333,14 @@ class Block(Part):
         tokens the block accepts it already applied up to the RMS factor (``NormedRows``);
         None otherwise."""
         return None
+
+    # True: ``forward`` never changes ``resid32`` in place unless it was given something to add
+    leaves_stream = False
+
+    def entry_norms(self) -> "tuple[Norm, ...]":
+        """The norms through which this block's sublayers read the incoming stream, if the block takes them ready made
+        (``ops.NormedStream`` as ``delta``); empty otherwise."""
+        return ()
 
 
 # --------------------------------------------------------------------------- registries
@@ -357,6 +385,7 @@ BLOCKS = Registry("block arrangement")
 STAGES = Registry("model stage")
 LAYER_EXTRAS = Registry("layer extra")
 PASS_ENTRIES = Registry("pass entry")
+STREAM_MIXES = Registry("stream mix")
 
 
 def build_part(registry: Registry, spec: PartSpec, ctx: BuildContext, **extra):

@@ -14,6 +14,9 @@ is what the next sublayer reads (``RoundedRows``).  A layer may have no feed-for
 ``parallel``: ``h = norm(x); x += mixer(h) + feed_forward(h)``: one norm, both sublayers read its
 output.  Both results are added in float32: by the product that made them where it can add into the
 stream itself, else by the norm kernel of the next block (``DeltaPair``).  A layer may have no feed-forward.
+With norms ``mixer`` and ``feed_forward`` instead of ``input`` each sublayer reads the same stream through a norm of its
+own; ``residual_scale`` m: ``x += m (mixer(norm_m(x)) + feed_forward(norm_f(x)))``.  A feed-forward that can leaves its last
+sum to the kernel that adds both results (``defers``).
 
 ``sandwich``: ``x += norm_mo(mixer(norm_mi(x))); x += norm_fo(feed_forward(norm_fi(x)))``: a norm before and
 after every sublayer (norms ``mixer_in``, ``mixer_out``, ``feed_forward_in``, ``feed_forward_out``), the sums in
@@ -28,6 +31,7 @@ import torch
 
 from ..kernels import ops
 from .base import BLOCKS, Block
+from .norms import take_stream_norms
 
 
 @BLOCKS.register("prenorm")
@@ -117,19 +121,37 @@ class ParallelBlock(Block):
     graph_safe = True
     accepts_pair = True           # takes an ``ops.DeltaPair`` as the pending result of the block before
 
-    def __init__(self, ctx, mixer, feed_forward, norms):
+    def __init__(self, ctx, mixer, feed_forward, norms, residual_scale: float = 1.0):
         super().__init__(mixer, feed_forward, norms)
-        if "input" not in norms:
-            raise ValueError("parallel block needs a norm named 'input'")
-        if not getattr(norms["input"], "accepts_pair", False):
+        self.ctx = ctx
+        own = {"mixer"} | ({"feed_forward"} if feed_forward is not None else set())
+        if "input" not in norms and own - set(norms):
+            raise ValueError(f"parallel block needs a norm named 'input', or norms named {sorted(own)}")
+        self.read = (norms["input"],) if "input" in norms else tuple(norms[k] for k in ("mixer", "feed_forward") if k in own)
+        if not getattr(self.read[0], "accepts_pair", False):
             raise ValueError("the norm of a parallel block must take two pending results (accepts_pair)")
+        self.scale = float(residual_scale)
+        # products may add into the stream only where nobody reads it afterwards and no factor comes in between
+        self.in_place = self.scale == 1.0 and len(self.read) == 1
+        self.leaves_stream = not self.in_place
+
+    def entry_norms(self):
+        return self.read
 
     def forward(self, resid32, delta, inputs, cache, next_norm=None):
         if isinstance(delta, ops.RoundedRows):          # the block before added its result itself
             delta = None
         if isinstance(delta, ops.NormedRows):
             raise ValueError("a parallel block cannot follow a block that fused the next norm into its last product")
-        h = self.norms["input"].add_forward(resid32, delta)
+        normed = delta.rows if isinstance(delta, ops.NormedStream) else take_stream_norms(resid32, delta, self.read, self.ctx.dtype)
+        h, h_ff = normed[0], normed[-1]
+        if not self.in_place:
+            a = self.mixer.forward(h, inputs, cache)
+            b = None
+            if self.feed_forward is not None:
+                b = self.feed_forward.forward(h_ff, inputs, defer=True) if getattr(self.feed_forward, "defers", False) \
+                    else self.feed_forward.forward(h_ff, inputs)
+            return resid32, ops.DeltaPair(a, b, self.scale)
         # each sublayer adds its result to the stream itself where its last product can (None comes back)
         a = self.mixer.forward(h, inputs, cache, residual32=resid32) if self.mixer.adds_residual \
             else self.mixer.forward(h, inputs, cache)

@@ -1,6 +1,7 @@
 """RMSNorm: ``x * rsqrt(mean(x^2) + eps) * w`` in float32, one rounding at the end (``one_plus``: the stored
 weight is the distance of ``w`` from one); and LayerNorm with
-weight and bias: ``(x - mean) * rsqrt(var + eps) * w + b``, var the mean of the squared deviations.
+weight and bias: ``(x - mean) * rsqrt(var + eps) * w + b``, var the mean of the squared deviations.  ``grouped_rmsnorm``:
+the vector in equal neighbouring parts, each over its own root mean square, then the whole times ``w``.
 
 Reference: ``RMSNorm`` in ``acorninfer/models/qwen3.py:50-60`` (the weight multiplies in
 float32 before the cast) and the fused residual-add form in ``acorninfer/ops/rmsnorm.py:15-36``.
@@ -92,3 +93,45 @@ class LayerNorm(Norm):
 
     def add_forward(self, resid32, delta, out=None, rows=None):
         return ops.add_layernorm(resid32, delta, self.weight32, self.bias32, self.eps, self.ctx.dtype, row_idx=rows, out=out)
+
+
+@NORMS.register("grouped_rmsnorm")
+class GroupedRMSNorm(Norm):
+    """The row split into ``groups`` equal neighbouring parts, each divided by ``sqrt(mean(part^2) + eps)``, the whole times
+    ``w``; float32, one rounding.  Runs on ``ops.stream_norm``, which also takes what is still to be added to the stream
+    and two such norms of one stream at once."""
+
+    graph_safe = True
+    accepts_pair = True           # add_forward takes an ``ops.DeltaPair`` (any kind)
+
+    def __init__(self, ctx: BuildContext, width: int, eps: float, groups: int = 1, tensor: str = "weight"):
+        if groups < 1 or width % groups:
+            raise ValueError(f"a norm in groups needs a width ({width}) that splits into {groups} equal parts")
+        self.ctx, self.width, self.eps, self.groups, self.tensor = ctx, width, float(eps), int(groups), tensor
+        self.scale32: torch.Tensor | None = None
+
+    def tensor_specs(self):
+        return {self.tensor: TensorSpec((self.width,), "norm")}
+
+    def bind(self, tensors):
+        self.scale32 = tensors[self.tensor].to(torch.float32).contiguous()
+
+    def stream_spec(self):
+        """What ``ops.stream_norm`` needs of this norm."""
+        return self.scale32, self.eps, self.groups
+
+    def forward(self, x32, out=None, rows=None):
+        return self.add_forward(x32, None, out=out, rows=rows)
+
+    def add_forward(self, resid32, delta, out=None, rows=None):
+        if out is not None:
+            raise ValueError("a grouped norm makes its own output")
+        return ops.stream_norm(resid32, delta, (self.stream_spec(),), self.ctx.dtype, rows=rows)[0]
+
+
+def take_stream_norms(resid32, delta, norms, dtype):
+    """The norms ``norms`` of ``resid32 + delta`` (added in place): in one kernel where they allow it."""
+    if all(hasattr(n, "stream_spec") for n in norms) and len({n.stream_spec()[1:] for n in norms}) == 1 and len(norms) <= 2:
+        return ops.stream_norm(resid32, delta, tuple(n.stream_spec() for n in norms), dtype)
+    first = norms[0].add_forward(resid32, delta)
+    return (first, *(n.forward(resid32) for n in norms[1:]))

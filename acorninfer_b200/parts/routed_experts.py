@@ -12,13 +12,19 @@ Options: no correction (``correction`` false: experts are ranked by their scores
 scores divided by their sum (``normalize``); experts of the capped form (``activation="capped_swish"`` with
 ``limit`` L: ``g = min(gate h, L), u = clamp(up h, -L, L), down(g sigmoid(1.702 g) (u + 1))``); a shared expert of
 the same form (``shared_size``, ``shared_limit``; tensors ``shared.gate`` / ``up`` / ``down``) that every token
-takes, added to the weighted sum.
+takes, added to the weighted sum; scores ``sigmoid(z)`` of each output instead of the softmax (``scoring="sigmoid"``);
+the chosen outputs' weights on the experts' *inputs* instead of their outputs (``weight_on="input"``: the sum over the
+chosen of ``expert(s h)``); the shared expert's result times ``sigmoid(W_sg h)``, one number per token (``shared_gate``;
+tensor ``shared.sg``).
 
 On the device: the router's choice (one kernel), the (token, choice) pairs grouped by expert (one
 kernel), one product per expert over its own rows for gate/up (SwiGLU in its epilogue on the tensor-core
 kernel) and for down (a kernel each, walking the per-expert offsets on the device: nothing of the routing
 is read on the host), and the weighted sum in the order of the choices, which also norms the result and
-adds it to the stream when the block asks.
+adds it to the stream when the block asks.  A weight on an expert's input is a factor on its gate/up product's float32 sums
+(the product is linear), in that product's epilogue; the sum over the choices then has no weights, and can be left to the
+kernel that adds the layer's results to the stream (``forward(..., defer=True)``).  The shared expert's gate row rides in
+the router's product.
 """
 
 from __future__ import annotations
@@ -27,6 +33,7 @@ import torch
 
 from ..kernels import ops
 from .base import FEED_FORWARDS, BuildContext, FeedForward, TensorSpec
+from .feed_forward import SwiGLU
 
 
 @FEED_FORWARDS.register("routed_experts")
@@ -36,12 +43,24 @@ class RoutedExperts(FeedForward):
     def __init__(self, ctx: BuildContext, hidden_size: int, expert_size: int, num_experts: int, num_identity: int,
                  top: int, groups: int = 1, keep: int = 1, correction: bool = True, normalize: bool = False,
                  activation: str = "silu", limit: float = 0.0, shared_size: int | None = None,
-                 shared_limit: float | None = None):
+                 shared_limit: float | None = None, scoring: str = "softmax", weight_on: str = "output",
+                 shared_gate: bool = False):
+        if scoring not in ops.MOE_SCORINGS:
+            raise ValueError(f"scoring must be one of {sorted(ops.MOE_SCORINGS)}, got {scoring!r}")
+        if weight_on not in ("output", "input") or (weight_on == "input" and (num_identity or num_experts < 1)):
+            raise ValueError("weight_on must be 'output' or 'input', the latter without identity experts")
+        if shared_gate and not shared_size:
+            raise ValueError("shared_gate needs a shared expert")
+        self.scoring, self.weight_on, self.shared_gate = scoring, weight_on, bool(shared_gate)
+        self.defers = weight_on == "input"      # ``forward(..., defer=True)`` leaves the sum over the choices undone
         if activation not in ("silu", "capped_swish"):
             raise ValueError(f"expert activation must be 'silu' or 'capped_swish', got {activation!r}")
         self.correction, self.normalize, self.activation, self.limit = bool(correction), bool(normalize), activation, float(limit)
         self.shared_size, self.shared_limit = shared_size, float(shared_limit if shared_limit is not None else limit)
         self.w_shared_gu = self.w_shared_down = None
+        # a shared expert of the uncapped form is a gated feed-forward like any other
+        self.shared_ff = SwiGLU(ctx, hidden_size, shared_size, "silu", {"gate": "gate", "up": "up", "down": "down"}) \
+            if shared_size and activation == "silu" else None
         n = num_experts + num_identity
         if n < 1 or n % groups or not (1 <= keep <= groups) or top > keep * (n // groups):
             raise ValueError(f"{n} router outputs do not split into {groups} groups of which {keep} hold {top} choices")
@@ -55,6 +74,8 @@ class RoutedExperts(FeedForward):
         specs = {"router": TensorSpec((n, self.hidden_size))}
         if self.correction:
             specs["correction"] = TensorSpec((n,), "bias")
+        if self.shared_gate:
+            specs["shared.sg"] = TensorSpec((1, self.hidden_size))
         if self.shared_size:
             specs["shared.gate"] = TensorSpec((self.shared_size, self.hidden_size))
             specs["shared.up"] = TensorSpec((self.shared_size, self.hidden_size))
@@ -71,13 +92,19 @@ class RoutedExperts(FeedForward):
         # exact in float32, so the tensor-core product with float32 accumulation is the float32 computation
         # on the rounded input, up to the order of the sum.
         self.w_router = t["router"].contiguous()
-        self.correction32 = t["correction"].to(torch.float32).contiguous() if self.correction else \
-            torch.zeros(self.E + self.I, dtype=torch.float32, device=self.w_router.device)
+        if self.shared_gate:                       # one more row of the router's product: [router | shared gate]
+            sg = t["shared.sg"]
+            dtype = sg.dtype if sg.dtype == self.w_router.dtype else torch.float32
+            self.w_router = torch.cat([self.w_router.to(dtype), sg.to(dtype)], dim=0).contiguous()
+        self.correction32 = t["correction"].to(torch.float32).contiguous() if self.correction else None
         if self.shared_size:
             g, u = t["shared.gate"], t["shared.up"]
             dtype = g.dtype if g.dtype == u.dtype else torch.float32
-            self.w_shared_gu = torch.cat([g.to(dtype), u.to(dtype)], dim=0).contiguous()       # [gate | up]
-            self.w_shared_down = t["shared.down"].contiguous()
+            if self.shared_ff is not None:
+                self.shared_ff.bind({n: t["shared." + n] for n in ("gate", "up", "down")})
+            else:
+                self.w_shared_gu = torch.cat([g.to(dtype), u.to(dtype)], dim=0).contiguous()       # [gate | up]
+                self.w_shared_down = t["shared.down"].contiguous()
         if self.E:
             mats = [t[f"e{e}.{n}"] for e in range(self.E) for n in ("gate", "up", "down")]
             dtype = mats[0].dtype if all(m.dtype == mats[0].dtype for m in mats) else torch.float32
@@ -89,27 +116,38 @@ class RoutedExperts(FeedForward):
 
     adds_normed_residual = True     # ``forward(..., add_normed=(resid32, norm))`` adds the normed result to the stream itself
 
-    def forward(self, x, inputs, add_normed=None):
-        T = x.shape[0]
+    def forward(self, x, inputs, add_normed=None, defer=False):
+        T, n = x.shape[0], self.E + self.I
         z = ops.linear(x, self.w_router, out_dtype=torch.float32)
-        idx, wts = ops.moe_route(z, self.correction32, self.top, self.groups, self.keep, normalize=self.normalize)
-        offsets, slot_of, slot_token = ops.moe_plan(idx, self.E + self.I)
+        idx, wts = ops.moe_route(z[:, :n], self.correction32, self.top, self.groups, self.keep, normalize=self.normalize,
+                                 scoring=self.scoring)
+        slot_wts = None
+        if self.weight_on == "input":
+            offsets, slot_of, slot_token, slot_wts = ops.moe_plan(idx, n, wts)
+            wts = None                       # the weights go in with the rows: the choices are summed as they are
+        else:
+            offsets, slot_of, slot_token = ops.moe_plan(idx, n)
         slots = T * self.top
         if self.E:
             w_gu = self.w_gate_up if self.w_gate_up.dtype == x.dtype else self.w_gate_up.to(x.dtype)
             w_dn = self.w_down if self.w_down.dtype == x.dtype else self.w_down.to(x.dtype)
             hidden = ops.grouped_gemm(x, slot_token, w_gu, offsets, slots, swiglu_pairs=True, activation=self.activation,
-                                      limit=self.limit)
+                                      limit=self.limit, slot_scale=slot_wts)
             y = ops.grouped_gemm(hidden, None, w_dn, offsets, slots)
         else:
             y = x
         shared = None
-        if self.shared_size:
+        if self.shared_ff is not None:
+            shared = self.shared_ff.forward(x, inputs)
+        elif self.shared_size:
             gu = ops.linear(x, self.w_shared_gu, out_dtype=self.ctx.dtype)
             shared = ops.linear(ops.swiglu(gu, activation=self.activation, limit=self.shared_limit), self.w_shared_down,
                                 out_dtype=self.ctx.dtype)
+        shared_z = z[:, n:n + 1] if self.shared_gate else None
+        if defer and self.defers:
+            return ops.ExpertsPending(y, slot_of, shared, shared_z)
         if add_normed is not None:
             resid32, norm = add_normed
             return ops.moe_combine(y, x, slot_of, idx, wts, self.E, resid32=resid32, weight32=norm.weight32, eps=norm.eps,
-                                   extra=shared)
-        return ops.moe_combine(y, x, slot_of, idx, wts, self.E, extra=shared)
+                                   extra=shared, extra_z=shared_z)
+        return ops.moe_combine(y, x, slot_of, idx, wts, self.E, extra=shared, extra_z=shared_z)

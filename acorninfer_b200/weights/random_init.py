@@ -170,6 +170,15 @@ INIT_KINDS.register("conv", lambda d: d.normal(0.5, 1.0 / d.shape[-1]))        #
 INIT_KINDS.register("decay_log", lambda d: d.normal(0.5, -1.0))        # log of a decay rate: exp(.) around 0.4
 INIT_KINDS.register("norm_offset", lambda d: d.normal(d.sigma_norm))     # a norm weight stored as its distance from one
 INIT_KINDS.register("lambda_part", lambda d: d.normal(0.3))             # vectors whose products' sum is an exponent: kept small
+def _depth_average(d: Draw) -> torch.Tensor:
+    """Coefficients of earlier results around 0.1, the newest one's around 1."""
+    t = d.normal(0.1, 0.05)
+    if d.rows is None or d.rows[1] == d.shape[0] > d.rows[0]:
+        t[-1] += 0.85
+    return t
+
+
+INIT_KINDS.register("depth_average", _depth_average)
 INIT_KINDS.register("blend", lambda d: d.normal(0.2, 0.5))             # shares of the row before in a blend of two rows
 
 
