@@ -17,17 +17,11 @@
 #include "mma_helpers.cuh"
 
 // One warp per token.  Ties go to the lower index.
-__global__ void moe_route_kernel(const float* __restrict__ z, int64_t ldz, const float* __restrict__ correction,
-                                 int* __restrict__ idx, float* __restrict__ wts, int tokens, int N, int top, int groups,
-                                 int keep, int normalize, int scoring) {
-    extern __shared__ float sm[];                       // per warp: s[N], choice[N]
-    pdl_wait();
-    pdl_trigger();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int t = blockIdx.x * (blockDim.x >> 5) + warp;
-    if (t >= tokens) return;
-    float* s = sm + (size_t)warp * 2 * N;
-    float* choice = s + N;
+__device__ __forceinline__ void route_token(const float* __restrict__ z, int64_t ldz, const float* __restrict__ correction,
+                                            int* __restrict__ idx, float* __restrict__ wts, int t, int N, int top, int groups,
+                                            int keep, int normalize, int scoring, float* s) {
+    const int lane = threadIdx.x & 31;
+    float* choice = s + N;                              // s[N], choice[N]: this warp's
     const float* zr = z + (int64_t)t * ldz;
     float m = -INFINITY;
     for (int i = lane; i < N; i += 32) m = fmaxf(m, zr[i]);
@@ -110,6 +104,18 @@ __global__ void moe_route_kernel(const float* __restrict__ z, int64_t ldz, const
     }
 }
 
+__global__ void moe_route_kernel(const float* __restrict__ z, int64_t ldz, const float* __restrict__ correction,
+                                 int* __restrict__ idx, float* __restrict__ wts, int tokens, int N, int top, int groups,
+                                 int keep, int normalize, int scoring) {
+    extern __shared__ float sm[];
+    pdl_wait();
+    pdl_trigger();
+    const int warp = threadIdx.x >> 5;
+    const int t = blockIdx.x * (blockDim.x >> 5) + warp;
+    if (t >= tokens) return;
+    route_token(z, ldz, correction, idx, wts, t, N, top, groups, keep, normalize, scoring, sm + (size_t)warp * 2 * N);
+}
+
 // scoring 0: softmax over the outputs; 1: the sigmoid of each.  correction may be null.
 extern "C" int acorn_moe_route(const float* z, int64_t ldz, const float* correction, int* idx, float* wts, int tokens, int N,
                                int top, int groups, int keep, int normalize, int scoring, cudaStream_t stream) {
@@ -132,13 +138,10 @@ extern "C" int acorn_moe_route(const float* z, int64_t ldz, const float* correct
 // One block: histogram of the chosen outputs, exclusive sums, then a slot for every pair.  Within an
 // expert the slots are handed out in whatever order the threads arrive: a row's result does not
 // depend on its slot.
-__global__ void moe_plan_kernel(const int* __restrict__ idx, int* __restrict__ offsets, int* __restrict__ slot_of,
-                                int* __restrict__ slot_token, int pairs, int N, int top,
-                                const float* __restrict__ wts, float* __restrict__ slot_wts) {
-    extern __shared__ int cnt[];                        // [N] counts, then [N] cursors
-    pdl_wait();
-    pdl_trigger();
-    int* cursor = cnt + N;
+__device__ __forceinline__ void plan_pairs(const int* idx, int* __restrict__ offsets, int* __restrict__ slot_of,
+                                           int* __restrict__ slot_token, int pairs, int N, int top, const float* wts,
+                                           float* __restrict__ slot_wts, int* cnt) {
+    int* cursor = cnt + N;                              // [N] counts, then [N] cursors
     for (int i = threadIdx.x; i < N; i += blockDim.x) cnt[i] = 0;
     __syncthreads();
     for (int i = threadIdx.x; i < pairs; i += blockDim.x) atomicAdd(&cnt[idx[i]], 1);
@@ -159,6 +162,51 @@ __global__ void moe_plan_kernel(const int* __restrict__ idx, int* __restrict__ o
         slot_token[slot] = i / top;
         if (slot_wts) slot_wts[slot] = wts[i];
     }
+}
+
+__global__ void moe_plan_kernel(const int* __restrict__ idx, int* __restrict__ offsets, int* __restrict__ slot_of,
+                                int* __restrict__ slot_token, int pairs, int N, int top, const float* __restrict__ wts,
+                                float* __restrict__ slot_wts) {
+    extern __shared__ int cnt[];
+    pdl_wait();
+    pdl_trigger();
+    plan_pairs(idx, offsets, slot_of, slot_token, pairs, N, top, wts, slot_wts, cnt);
+}
+
+// Both for a step of few tokens: one block, a warp a token at a time, then the grouping of what they chose.
+#define MOE_SMALL_TOKENS 128
+#define MOE_SMALL_OUTPUTS 160
+
+__global__ void __launch_bounds__(1024) moe_route_plan_kernel(const float* __restrict__ z, int64_t ldz, const float* __restrict__ correction,
+                                                              int* idx, float* wts, int tokens, int N, int top, int groups, int keep,
+                                                              int normalize, int scoring, int* __restrict__ offsets,
+                                                              int* __restrict__ slot_of, int* __restrict__ slot_token,
+                                                              float* __restrict__ slot_wts) {
+    extern __shared__ float sm[];                       // per warp: s[N], choice[N]; then the counts
+    pdl_wait();
+    pdl_trigger();
+    const int warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    for (int t = warp; t < tokens; t += warps) {
+        route_token(z, ldz, correction, idx, wts, t, N, top, groups, keep, normalize, scoring, sm + (size_t)warp * 2 * N);
+        __syncwarp();
+    }
+    __syncthreads();                                    // what the block's warps wrote to idx and wts is read by all of it
+    plan_pairs(idx, offsets, slot_of, slot_token, tokens * top, N, top, wts, slot_wts, reinterpret_cast<int*>(sm));
+}
+
+extern "C" int acorn_moe_route_plan_supported(int tokens, int N) { return tokens <= MOE_SMALL_TOKENS && N <= MOE_SMALL_OUTPUTS; }
+
+extern "C" int acorn_moe_route_plan(const float* z, int64_t ldz, const float* correction, int* idx, float* wts, int tokens,
+                                    int N, int top, int groups, int keep, int normalize, int scoring, int* offsets,
+                                    int* slot_of, int* slot_token, float* slot_wts, cudaStream_t stream) {
+    if (tokens <= 0) return 0;
+    if (!acorn_moe_route_plan_supported(tokens, N) || scoring < 0 || scoring > 1 || ldz < N || N < 1 || top < 1 || top > N ||
+        groups < 1 || groups > 64 || N % groups || keep < 1 || keep > groups)
+        return ACORN_ERR_UNSUPPORTED;
+    const int warps = tokens < 8 ? 8 : (tokens > 32 ? 32 : tokens);
+    return acorn_launch(moe_route_plan_kernel, dim3(1), dim3(32 * warps), (size_t)warps * 2 * N * sizeof(float), stream, z, ldz,
+                        correction, idx, wts, tokens, N, top, groups, keep, normalize, scoring, offsets, slot_of, slot_token,
+                        slot_wts);
 }
 
 // slot_wts [pairs], if given, receives the pairs' weights (wts) by slot

@@ -145,6 +145,9 @@ class _Sigs:
     acorn_moe_route = [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                        c_void_p]
     acorn_moe_plan = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p]
+    acorn_moe_route_plan = [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                            c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]
+    acorn_moe_route_plan_supported = [c_int, c_int]
     acorn_grouped_gemm = [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int,
                           c_int, c_int, c_int, c_float, c_void_p, c_void_p]
     acorn_grouped_gemm_fuses_swiglu = [c_int, c_int, c_int64, c_int]
@@ -157,7 +160,8 @@ class _Sigs:
                          c_int64, c_float, c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                          c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p]
     acorn_min_gru = [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                     c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p]
+                     c_int, c_int, c_void_p, c_void_p, c_int, c_void_p]
+    acorn_min_gru_segment_tokens = []
     acorn_diff_combine = [c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_int,
                           c_void_p]
     acorn_pair_rows = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
@@ -1882,21 +1886,15 @@ def gated_norm(y32: torch.Tensor, gate: torch.Tensor, weight32: torch.Tensor, ep
 
 # ------------------------------------------------------------------ minimal gated recurrence
 
-GRU_MIN_SEGMENT = 32              # tokens: shorter segments are not worth a second pass
-GRU_MAX_SEGMENTS = 64
-GRU_ENOUGH_BLOCKS = 296           # blocks that keep the device busy (148 SMs, two a piece)
+GRU_WALK_TOKENS = 4               # rows of at most so many tokens: a thread walks them
+GRU_SEGMENT = 128                 # tokens a block takes of a longer row
 
 
-def gru_segments(longest_row: int, num_rows: int, width: int) -> tuple[int, int]:
-    """(tokens a segment, segments a row) for ``min_gru``, (0, 1) for rows in one piece.  Rows run side by side with blocks
-    of channels; where those are too few to fill the device and a row is long, rows are cut into segments that run
-    side by side (at the price of a second pass over them)."""
-    blocks = max(1, num_rows) * max(1, -(-width // 512))
-    nseg = min(GRU_MAX_SEGMENTS, longest_row // GRU_MIN_SEGMENT, -(-GRU_ENOUGH_BLOCKS // blocks), 65535 // max(1, num_rows))
-    if nseg < 2:
-        return 0, 1
-    seg = -(-longest_row // nseg)
-    return seg, -(-longest_row // seg)
+def gru_segments(longest_row: int, num_rows: int) -> int:
+    """Segments a row for ``min_gru``; 0: a thread walks its channels token by token (short rows, or so many
+    segments that they do not fit a grid)."""
+    nseg = -(-longest_row // GRU_SEGMENT)
+    return 0 if longest_row <= GRU_WALK_TOKENS or num_rows * nseg > 65535 else nseg
 
 
 def min_gru(proj: torch.Tensor, bias32: torch.Tensor, state: torch.Tensor, state_off: int, row_start: torch.Tensor,
@@ -1913,15 +1911,15 @@ def min_gru(proj: torch.Tensor, bias32: torch.Tensor, state: torch.Tensor, state
     if W3 != 3 * width or bias32.numel() != 2 * width or state.shape[1] < state_off + width:
         raise KernelError(f"min_gru: proj {tuple(proj.shape)}, bias {bias32.numel()}, state {tuple(state.shape)} do not fit")
     out = torch.empty((T, width), dtype=proj.dtype, device=proj.device)
-    seg, nseg = gru_segments(int(longest_row), num_rows, width)
+    nseg = gru_segments(int(longest_row), num_rows)
     seg_a = seg_b = None
     if nseg > 1:
         seg_a = torch.empty((num_rows, nseg, width), dtype=torch.float32, device=proj.device)
         seg_b = torch.empty((num_rows, nseg + 1, width), dtype=torch.float32, device=proj.device)
-    for pass_ in ((0,) if nseg == 1 else (1, 2)):
+    for pass_ in ((0,), (2,))[nseg] if nseg < 2 else (1, 2):
         _ok(lib().acorn_min_gru(proj.data_ptr(), proj.stride(0), bias32.data_ptr(), state.data_ptr(), state.stride(0),
                                 int(state_off), row_start.data_ptr(), row_slot.data_ptr(), out.data_ptr(), num_rows, width,
-                                pass_, seg, nseg, _ptr(seg_a), _ptr(seg_b), dtype_code(proj.dtype), _stream()), "min_gru",
+                                pass_, nseg, _ptr(seg_a), _ptr(seg_b), dtype_code(proj.dtype), _stream()), "min_gru",
             f"pass {pass_}")
     return out
 
@@ -1971,6 +1969,30 @@ def moe_plan(idx: torch.Tensor, num_outputs: int, wts: torch.Tensor | None = Non
     _ok(lib().acorn_moe_plan(idx.data_ptr(), offsets.data_ptr(), slot_of.data_ptr(), slot_token.data_ptr(), T * top,
                              num_outputs, top, _ptr(wts), _ptr(slot_wts), _stream()), "moe_plan")
     return (offsets, slot_of, slot_token) if wts is None else (offsets, slot_of, slot_token, slot_wts)
+
+
+def moe_route_plan(z32: torch.Tensor, correction32: torch.Tensor | None, top: int, groups: int, keep: int,
+                   normalize: bool = False, scoring: str = "softmax", by_slot: bool = False):
+    """``moe_route`` followed by ``moe_plan``: (chosen, weights, offsets, slot_of, slot_token, weights by slot if ``by_slot``
+    else None); one kernel for steps of few tokens."""
+    T, N = z32.shape
+    if not lib().acorn_moe_route_plan_supported(T, N):
+        idx, wts = moe_route(z32, correction32, top, groups, keep, normalize, scoring)
+        offsets, slot_of, slot_token, *rest = moe_plan(idx, N, wts if by_slot else None)
+        return idx, wts, offsets, slot_of, slot_token, (rest[0] if by_slot else None)
+    _rows2(z32, "router logits", torch.float32)
+    if correction32 is not None:
+        _check(correction32, "correction", torch.float32, 1)
+        if correction32.numel() != N:
+            raise KernelError("moe_route: correction must have one entry per router output")
+    i32 = lambda *shape: torch.empty(shape, dtype=torch.int32, device=z32.device)
+    f32 = lambda *shape: torch.empty(shape, dtype=torch.float32, device=z32.device)
+    idx, wts, offsets, slot_of, slot_token = i32(T, top), f32(T, top), i32(N + 1), i32(T, top), i32(T * top)
+    slot_wts = f32(T * top) if by_slot else None
+    _ok(lib().acorn_moe_route_plan(z32.data_ptr(), z32.stride(0), _ptr(correction32), idx.data_ptr(), wts.data_ptr(), T, N, int(top),
+                                   int(groups), int(keep), 1 if normalize else 0, MOE_SCORINGS[scoring], offsets.data_ptr(),
+                                   slot_of.data_ptr(), slot_token.data_ptr(), _ptr(slot_wts), _stream()), "moe_route_plan")
+    return idx, wts, offsets, slot_of, slot_token, slot_wts
 
 
 GROUPED_TCGEN05_MIN_ROWS = 64      # rows an expert on average from which the grouped product takes the tcgen05 kernel

@@ -17,8 +17,8 @@ the chosen outputs' weights on the experts' *inputs* instead of their outputs (`
 chosen of ``expert(s h)``); the shared expert's result times ``sigmoid(W_sg h)``, one number per token (``shared_gate``;
 tensor ``shared.sg``).
 
-On the device: the router's choice (one kernel), the (token, choice) pairs grouped by expert (one
-kernel), one product per expert over its own rows for gate/up (SwiGLU in its epilogue on the tensor-core
+On the device: the router's choice and the (token, choice) pairs grouped by expert (a kernel each, one for both in
+steps of few tokens), one product per expert over its own rows for gate/up (SwiGLU in its epilogue on the tensor-core
 kernel) and for down (a kernel each, walking the per-expert offsets on the device: nothing of the routing
 is read on the host), and the weighted sum in the order of the choices, which also norms the result and
 adds it to the stream when the block asks.  A weight on an expert's input is a factor on its gate/up product's float32 sums
@@ -119,14 +119,11 @@ class RoutedExperts(FeedForward):
     def forward(self, x, inputs, add_normed=None, defer=False):
         T, n = x.shape[0], self.E + self.I
         z = ops.linear(x, self.w_router, out_dtype=torch.float32)
-        idx, wts = ops.moe_route(z[:, :n], self.correction32, self.top, self.groups, self.keep, normalize=self.normalize,
-                                 scoring=self.scoring)
-        slot_wts = None
+        idx, wts, offsets, slot_of, slot_token, slot_wts = ops.moe_route_plan(
+            z[:, :n], self.correction32, self.top, self.groups, self.keep, self.normalize, self.scoring,
+            by_slot=self.weight_on == "input")
         if self.weight_on == "input":
-            offsets, slot_of, slot_token, slot_wts = ops.moe_plan(idx, n, wts)
             wts = None                       # the weights go in with the rows: the choices are summed as they are
-        else:
-            offsets, slot_of, slot_token = ops.moe_plan(idx, n)
         slots = T * self.top
         if self.E:
             w_gu = self.w_gate_up if self.w_gate_up.dtype == x.dtype else self.w_gate_up.to(x.dtype)

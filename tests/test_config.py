@@ -100,6 +100,8 @@ def test_presets_of_the_family_are_valid_configurations():
         elif name.startswith("zigolix"):
             assert [l.type for l in cfg.layers[:3]] == ["attention_2", "attention_2", "attention"]
             assert len(spec_for(cfg).schedule) == 8          # layers 1 and 2 twice among six
+        elif name.startswith("zusolix"):
+            assert [l.type for l in cfg.layers[:4]] == ["attention", "attention", "mingru", "attention"]
         else:
             assert name.startswith("tedenex") and [l.type for l in cfg.layers[:3]] == ["wkv", "attention", "latent_attention"]
             assert len(spec_for(cfg).schedule) == 9          # the first three layers twice, then the other three
