@@ -16,8 +16,8 @@
 //              (tcgen05.ld / st) only when a row's maximum has grown by more than 2^8 since its
 //              reference was set, so most blocks skip that pass.  At the end the thread reads
 //              its row of O, divides by the row sum and writes the output.  Options of the scores:
-//              a penalty per head on the distance to the key, a cap c (c tanh(score / c), two more
-//              special-function operations a score), a sink per head (exp(sink) joins the row sum
+//              a penalty per head on the distance to the key, a cap c (c tanh(score / c): a polynomial where the
+//              scores are small against the cap, else two more special-function operations a score), a sink per head (exp(sink) joins the row sum
 //              at the end, against the same reference maximum).
 //   warp 8     producer: TMA loads of Q (once) and of the K and V tiles of each block
 //              ((page, kv head) tiles are contiguous [page_size x 128] in the cache) into a ring
@@ -78,8 +78,27 @@ __device__ __forceinline__ void atc_distance(float (&s)[64], float step) {
 }
 
 // s[c] <- (cap / scale) tanh(s[c] scale / cap): the capped score in units of the raw one, tanh(z) = 1 - 2 / (1 + e^(2z))
-// by the fast exponential and quotient (two more special-function operations a score beside the softmax's own)
+// by the fast exponential and quotient (two more special-function operations a score beside the softmax's own); where no
+// score of the warp's rows comes to 0.4 of the cap, by the Taylor series of tanh up to z^11 (the next term is below 6e-8 of
+// the first), which needs none.
 __device__ __forceinline__ void atc_cap(float (&s)[64], float k, float c2) {
+    float m[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int c = 0; c < 64; c += 4) {
+        m[0] = fmaxf(m[0], fabsf(s[c])); m[1] = fmaxf(m[1], fabsf(s[c + 1]));
+        m[2] = fmaxf(m[2], fabsf(s[c + 2])); m[3] = fmaxf(m[3], fabsf(s[c + 3]));
+    }
+    if (__all_sync(0xffffffffu, fmaxf(fmaxf(m[0], m[1]), fmaxf(m[2], m[3])) <= 0.4f * c2)) {
+        const float r = 1.f / (c2 * c2);                 // z^2 = r s^2
+        const float k1 = -r / 3.f, k2 = r * r * (2.f / 15.f), k3 = r * r * r * (-17.f / 315.f),
+                    k4 = r * r * r * r * (62.f / 2835.f), k5 = r * r * r * r * r * (-1382.f / 155925.f);
+#pragma unroll
+        for (int c = 0; c < 64; ++c) {
+            const float t = s[c] * s[c];
+            s[c] = fmaf(s[c] * t, fmaf(fmaf(fmaf(fmaf(k5, t, k4), t, k3), t, k2), t, k1), s[c]);
+        }
+        return;
+    }
 #pragma unroll
     for (int c = 0; c < 64; ++c) s[c] = c2 * (1.f - __fdividef(2.f, 1.f + fast_exp2(s[c] * k)));
 }

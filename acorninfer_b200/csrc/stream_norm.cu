@@ -40,6 +40,7 @@ __device__ __forceinline__ float sn_sigmoid(float z) { return 1.f / (1.f + expf(
 
 // H / groups a multiple of 128: a warp's 32 vectors of four lie in one part, so a part's sum of squares is the sum
 // of its chunks of 128; a thread's NV vectors stay in registers from the first read to the last write.
+// Loads have no condition between them (threads beyond the row read its last vector again): they are in flight together.
 template <typename T, int NV>
 __global__ void stream_norm_vec_kernel(const StreamParams<T> p) {
     __shared__ float chunk_ss[512];                     // H / 128 chunks
@@ -49,63 +50,71 @@ __global__ void stream_norm_vec_kernel(const StreamParams<T> p) {
     const int64_t row = p.row_idx ? p.row_idx[r] : r;
     const bool writes = p.row_idx == nullptr;
     const int n4 = p.H >> 2;
-    const bool pending = p.a || p.b || p.y;
-    const float* x = p.x + row * p.H;
+    int at[NV];                                         // this thread's elements
+    bool in[NV];
     float4 v[NV];
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
         const int i = threadIdx.x + k * blockDim.x;
-        v[k] = i < n4 ? *reinterpret_cast<const float4*>(x + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        in[k] = i < n4;
+        at[k] = 4 * min(i, n4 - 1);
+        v[k] = *reinterpret_cast<const float4*>(p.x + row * p.H + at[k]);
     }
-    if (pending) {
+    if (p.a || p.b || p.y) {
         float gate = 1.f;
         if (p.extra && p.extra_z) gate = sn_sigmoid(p.extra_z[row * p.ld_z]);
+        float4 d[NV];
+#pragma unroll
+        for (int k = 0; k < NV; ++k) d[k] = p.a ? Vec4<T>::load(p.a + row * p.H + at[k]) : make_float4(0.f, 0.f, 0.f, 0.f);
+        auto add = [&](const T* src, float f) {
+            float4 e[NV];
+#pragma unroll
+            for (int k = 0; k < NV; ++k) e[k] = Vec4<T>::load(src + at[k]);
+#pragma unroll
+            for (int k = 0; k < NV; ++k) {
+                d[k].x = fmaf(f, e[k].x, d[k].x); d[k].y = fmaf(f, e[k].y, d[k].y);
+                d[k].z = fmaf(f, e[k].z, d[k].z); d[k].w = fmaf(f, e[k].w, d[k].w);
+            }
+        };
+        if (p.b) add(p.b + row * p.H, 1.f);
+        if (p.y) {
+#pragma unroll 2
+            for (int c = 0; c < p.top; ++c) add(p.y + (int64_t)p.slot_of[row * p.top + c] * p.H, 1.f);
+            if (p.extra) add(p.extra + row * p.H, gate);
+        }
 #pragma unroll
         for (int k = 0; k < NV; ++k) {
-            const int i = threadIdx.x + k * blockDim.x;
-            if (i >= n4) continue;
-            float4 d = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (p.a) d = Vec4<T>::load(p.a + row * p.H + 4 * i);
-            if (p.b) {
-                const float4 e = Vec4<T>::load(p.b + row * p.H + 4 * i);
-                d.x += e.x; d.y += e.y; d.z += e.z; d.w += e.w;
-            }
-            if (p.y) {
-                float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-                for (int c = 0; c < p.top; ++c) {
-                    const float4 e = Vec4<T>::load(p.y + (int64_t)p.slot_of[row * p.top + c] * p.H + 4 * i);
-                    s.x += e.x; s.y += e.y; s.z += e.z; s.w += e.w;
-                }
-                if (p.extra) {
-                    const float4 e = Vec4<T>::load(p.extra + row * p.H + 4 * i);
-                    s.x = fmaf(gate, e.x, s.x); s.y = fmaf(gate, e.y, s.y); s.z = fmaf(gate, e.z, s.z); s.w = fmaf(gate, e.w, s.w);
-                }
-                d.x += s.x; d.y += s.y; d.z += s.z; d.w += s.w;
-            }
-            v[k].x = fmaf(p.scale, d.x, v[k].x); v[k].y = fmaf(p.scale, d.y, v[k].y);
-            v[k].z = fmaf(p.scale, d.z, v[k].z); v[k].w = fmaf(p.scale, d.w, v[k].w);
+            v[k].x = fmaf(p.scale, d[k].x, v[k].x); v[k].y = fmaf(p.scale, d[k].y, v[k].y);
+            v[k].z = fmaf(p.scale, d[k].z, v[k].z); v[k].w = fmaf(p.scale, d[k].w, v[k].w);
         }
     }
     if (p.coef) {
-        float4 acc[NV];
         const float cn = p.coef[p.n_hist];
+        float4 acc[NV];
 #pragma unroll
         for (int k = 0; k < NV; ++k) {
-            const int i = threadIdx.x + k * blockDim.x;
-            if (i < n4 && writes && p.hist_out) *reinterpret_cast<float4*>(p.hist_out + row * p.H + 4 * i) = v[k];
+            if (in[k] && writes && p.hist_out) *reinterpret_cast<float4*>(p.hist_out + row * p.H + at[k]) = v[k];
             acc[k] = make_float4(cn * v[k].x, cn * v[k].y, cn * v[k].z, cn * v[k].w);
         }
         const float* h = p.hist + row * p.H;
-#pragma unroll 4
-        for (int j = 0; j < p.n_hist; ++j) {
-            const float c = p.coef[j];
+        constexpr int AHEAD = NV >= 4 ? 2 : 4;
+        for (int j = 0; j < p.n_hist; j += AHEAD) {
+            float4 e[AHEAD][NV];
+            float c[AHEAD];
 #pragma unroll
-            for (int k = 0; k < NV; ++k) {
-                const int i = threadIdx.x + k * blockDim.x;
-                if (i < n4) {
-                    const float4 e = *reinterpret_cast<const float4*>(h + j * p.hist_stride + 4 * i);
-                    acc[k].x = fmaf(c, e.x, acc[k].x); acc[k].y = fmaf(c, e.y, acc[k].y);
-                    acc[k].z = fmaf(c, e.z, acc[k].z); acc[k].w = fmaf(c, e.w, acc[k].w);
+            for (int q = 0; q < AHEAD; ++q) {
+                const int jj = min(j + q, p.n_hist - 1);
+                c[q] = j + q < p.n_hist ? p.coef[jj] : 0.f;
+#pragma unroll
+                for (int k = 0; k < NV; ++k) e[q][k] = *reinterpret_cast<const float4*>(h + jj * p.hist_stride + at[k]);
+            }
+#pragma unroll
+            for (int q = 0; q < AHEAD; ++q) {
+                if (j + q >= p.n_hist) break;
+#pragma unroll
+                for (int k = 0; k < NV; ++k) {
+                    acc[k].x = fmaf(c[q], e[q][k].x, acc[k].x); acc[k].y = fmaf(c[q], e[q][k].y, acc[k].y);
+                    acc[k].z = fmaf(c[q], e[q][k].z, acc[k].z); acc[k].w = fmaf(c[q], e[q][k].w, acc[k].w);
                 }
             }
         }
@@ -114,10 +123,8 @@ __global__ void stream_norm_vec_kernel(const StreamParams<T> p) {
     }
     if (writes && p.x_out) {
 #pragma unroll
-        for (int k = 0; k < NV; ++k) {
-            const int i = threadIdx.x + k * blockDim.x;
-            if (i < n4) *reinterpret_cast<float4*>(p.x_out + row * p.H + 4 * i) = v[k];
-        }
+        for (int k = 0; k < NV; ++k)
+            if (in[k]) *reinterpret_cast<float4*>(p.x_out + row * p.H + at[k]) = v[k];
     }
     if (!p.out1) return;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
@@ -137,13 +144,12 @@ __global__ void stream_norm_vec_kernel(const StreamParams<T> p) {
         float ss = 0.f;
         for (int q = lane; q < per; q += 32) ss += chunk_ss[first + q];
         const float inv = rsqrtf(warp_sum(ss) / (float)(p.H / p.groups) + p.eps);
-        const int i = threadIdx.x + k * blockDim.x;
         const float4 n = make_float4(v[k].x * inv, v[k].y * inv, v[k].z * inv, v[k].w * inv);
-        const float4 w = *reinterpret_cast<const float4*>(p.w1 + 4 * i);
-        Vec4<T>::store(p.out1 + (int64_t)r * p.H + 4 * i, make_float4(n.x * w.x, n.y * w.y, n.z * w.z, n.w * w.w));
+        const float4 w = *reinterpret_cast<const float4*>(p.w1 + at[k]);
+        Vec4<T>::store(p.out1 + (int64_t)r * p.H + at[k], make_float4(n.x * w.x, n.y * w.y, n.z * w.z, n.w * w.w));
         if (p.out2) {
-            const float4 u = *reinterpret_cast<const float4*>(p.w2 + 4 * i);
-            Vec4<T>::store(p.out2 + (int64_t)r * p.H + 4 * i, make_float4(n.x * u.x, n.y * u.y, n.z * u.z, n.w * u.w));
+            const float4 u = *reinterpret_cast<const float4*>(p.w2 + at[k]);
+            Vec4<T>::store(p.out2 + (int64_t)r * p.H + at[k], make_float4(n.x * u.x, n.y * u.y, n.z * u.z, n.w * u.w));
         }
     }
 }

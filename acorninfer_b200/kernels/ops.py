@@ -46,6 +46,7 @@ def _load():
                 fn.argtypes = getattr(_Sigs, name)
                 fn.restype = c_int
         _lib.acorn_uniform.restype = c_float
+        _lib.acorn_min_gru_scratch.restype = c_int64
         _init_error_word(_lib)
     return _lib
 
@@ -160,8 +161,8 @@ class _Sigs:
                          c_int64, c_float, c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                          c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p]
     acorn_min_gru = [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                     c_int, c_int, c_void_p, c_void_p, c_int, c_void_p]
-    acorn_min_gru_segment_tokens = []
+                     c_int, c_int, c_void_p, c_int, c_void_p]
+    acorn_min_gru_scratch = [c_int, c_int, c_int]
     acorn_diff_combine = [c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_int,
                           c_void_p]
     acorn_pair_rows = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
@@ -234,6 +235,37 @@ def _stream() -> int:
             _device_index = torch.cuda.current_device()      # the engine works on one device
         return _raw_stream(_device_index)
     return torch.cuda.current_stream().cuda_stream
+
+
+_branch_streams: list = []
+
+
+class Branch:
+    """``fn()`` beside whatever the caller launches until ``join``: while a step of few single tokens is captured, on a stream of
+    its own, so that the graph holds both as branches that run side by side (the kernels of such a step leave most of the
+    device idle); otherwise at once, in order.  What ``fn`` reads must stay referenced until ``join``, which returns its
+    result.  Larger steps fill the device anyway; and their kernels hold so much tensor memory that two of them on one
+    multiprocessor could wait for one another's (the attention of prompts takes all of it, the paired product's CTAs and
+    a cluster's wait for their partners), while a product of at most ``GEMM_TC_MAX_ROWS`` rows takes a sixteenth."""
+
+    MAX_TOKENS = 128
+
+    def __init__(self, fn, inputs):
+        self.stream = None
+        if not (inputs.plan.all_decode and inputs.num_tokens <= self.MAX_TOKENS and torch.cuda.is_current_stream_capturing()):
+            self.result = fn()
+            return
+        self.stream = _branch_streams.pop() if _branch_streams else torch.cuda.Stream()
+        self.stream.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(self.stream):
+            self.result = fn()
+
+    def join(self):
+        if self.stream is not None:
+            torch.cuda.current_stream().wait_stream(self.stream)
+            _branch_streams.append(self.stream)
+            self.stream = None
+        return self.result
 
 
 def dtype_code(dtype: torch.dtype) -> int:
@@ -315,7 +347,7 @@ class _TimedLib:
 
     def __getattr__(self, name):
         fn = getattr(self._library, name)
-        if not name.startswith("acorn_") or name.endswith(("_supported", "_error", "_merges")):
+        if not name.startswith("acorn_") or name.endswith(("_supported", "_error", "_merges", "_scratch")):
             return fn
 
         def timed(*args):
@@ -1886,15 +1918,13 @@ def gated_norm(y32: torch.Tensor, gate: torch.Tensor, weight32: torch.Tensor, ep
 
 # ------------------------------------------------------------------ minimal gated recurrence
 
-GRU_WALK_TOKENS = 4               # rows of at most so many tokens: a thread walks them
-GRU_SEGMENT = 128                 # tokens a block takes of a longer row
+GRU_WALK_TOKENS = 32              # rows of at most so many tokens: a thread walks them
 
 
-def gru_segments(longest_row: int, num_rows: int) -> int:
-    """Segments a row for ``min_gru``; 0: a thread walks its channels token by token (short rows, or so many
-    segments that they do not fit a grid)."""
-    nseg = -(-longest_row // GRU_SEGMENT)
-    return 0 if longest_row <= GRU_WALK_TOKENS or num_rows * nseg > 65535 else nseg
+def gru_walks(longest_row: int, num_rows: int) -> bool:
+    """Whether ``min_gru`` lets a thread walk a row's tokens one by one: short rows, and steps with so many and so unequal
+    rows that the chunks of the longest do not fit a grid for all."""
+    return longest_row <= GRU_WALK_TOKENS or num_rows * -(-longest_row // 8) > 65535
 
 
 def min_gru(proj: torch.Tensor, bias32: torch.Tensor, state: torch.Tensor, state_off: int, row_start: torch.Tensor,
@@ -1902,7 +1932,7 @@ def min_gru(proj: torch.Tensor, bias32: torch.Tensor, state: torch.Tensor, state
     """``z = sigmoid(proj_z + b_z), u = proj_u + b_u, c = u + 1/2 (u >= 0) or sigmoid(u);  S <- (1 - z) S + z c;  S silu(proj_g)``
     for every token of every row, from the state in the row's slot (``[width]`` float32 at ``state_off``, updated in
     place).  proj [T, 3 width] holds ``[z | u | g]``; bias32 [2 width].  ``longest_row``: a bound on the tokens of a row (a
-    host number); long rows run in segments side by side (``gru_segments``).  Returns [T, width] in proj's dtype."""
+    host number); long rows run in chunks side by side, in two passes (``gru_walks``: when not).  Returns [T, width] in proj's dtype."""
     _rows2(proj, "proj")
     _check(bias32, "bias", torch.float32, 1)
     _check(state, "state", torch.float32, 2)
@@ -1911,15 +1941,14 @@ def min_gru(proj: torch.Tensor, bias32: torch.Tensor, state: torch.Tensor, state
     if W3 != 3 * width or bias32.numel() != 2 * width or state.shape[1] < state_off + width:
         raise KernelError(f"min_gru: proj {tuple(proj.shape)}, bias {bias32.numel()}, state {tuple(state.shape)} do not fit")
     out = torch.empty((T, width), dtype=proj.dtype, device=proj.device)
-    nseg = gru_segments(int(longest_row), num_rows)
-    seg_a = seg_b = None
-    if nseg > 1:
-        seg_a = torch.empty((num_rows, nseg, width), dtype=torch.float32, device=proj.device)
-        seg_b = torch.empty((num_rows, nseg + 1, width), dtype=torch.float32, device=proj.device)
-    for pass_ in ((0,), (2,))[nseg] if nseg < 2 else (1, 2):
+    walks = gru_walks(int(longest_row), num_rows)
+    scratch = None
+    if not walks:
+        scratch = torch.empty(lib().acorn_min_gru_scratch(num_rows, width, int(longest_row)), dtype=torch.float32, device=proj.device)
+    for pass_ in (0,) if walks else (1, 2):
         _ok(lib().acorn_min_gru(proj.data_ptr(), proj.stride(0), bias32.data_ptr(), state.data_ptr(), state.stride(0),
                                 int(state_off), row_start.data_ptr(), row_slot.data_ptr(), out.data_ptr(), num_rows, width,
-                                pass_, nseg, _ptr(seg_a), _ptr(seg_b), dtype_code(proj.dtype), _stream()), "min_gru",
+                                pass_, int(longest_row), _ptr(scratch), dtype_code(proj.dtype), _stream()), "min_gru",
             f"pass {pass_}")
     return out
 

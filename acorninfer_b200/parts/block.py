@@ -15,7 +15,8 @@ is what the next sublayer reads (``RoundedRows``).  A layer may have no feed-for
 output.  Both results are added in float32: by the product that made them where it can add into the
 stream itself, else by the norm kernel of the next block (``DeltaPair``).  A layer may have no feed-forward.
 With norms ``mixer`` and ``feed_forward`` instead of ``input`` each sublayer reads the same stream through a norm of its
-own; ``residual_scale`` m: ``x += m (mixer(norm_m(x)) + feed_forward(norm_f(x)))``.  A feed-forward that can leaves its last
+own; ``residual_scale`` m: ``x += m (mixer(norm_m(x)) + feed_forward(norm_f(x)))``; in captured steps the two then are
+branches of the graph that run side by side.  A feed-forward that can leaves its last
 sum to the kernel that adds both results (``defers``).
 
 ``sandwich``: ``x += norm_mo(mixer(norm_mi(x))); x += norm_fo(feed_forward(norm_fi(x)))``: a norm before and
@@ -146,12 +147,12 @@ class ParallelBlock(Block):
         normed = delta.rows if isinstance(delta, ops.NormedStream) else take_stream_norms(resid32, delta, self.read, self.ctx.dtype)
         h, h_ff = normed[0], normed[-1]
         if not self.in_place:
+            if self.feed_forward is None:
+                return resid32, ops.DeltaPair(self.mixer.forward(h, inputs, cache), None, self.scale)
+            more = {"defer": True} if getattr(self.feed_forward, "defers", False) else {}
+            beside = ops.Branch(lambda: self.feed_forward.forward(h_ff, inputs, **more), inputs)
             a = self.mixer.forward(h, inputs, cache)
-            b = None
-            if self.feed_forward is not None:
-                b = self.feed_forward.forward(h_ff, inputs, defer=True) if getattr(self.feed_forward, "defers", False) \
-                    else self.feed_forward.forward(h_ff, inputs)
-            return resid32, ops.DeltaPair(a, b, self.scale)
+            return resid32, ops.DeltaPair(a, beside.join(), self.scale)
         # each sublayer adds its result to the stream itself where its last product can (None comes back)
         a = self.mixer.forward(h, inputs, cache, residual32=resid32) if self.mixer.adds_residual \
             else self.mixer.forward(h, inputs, cache)

@@ -118,6 +118,7 @@ class RoutedExperts(FeedForward):
 
     def forward(self, x, inputs, add_normed=None, defer=False):
         T, n = x.shape[0], self.E + self.I
+        beside = ops.Branch(lambda: self.shared_ff.forward(x, inputs), inputs) if self.shared_ff is not None else None
         z = ops.linear(x, self.w_router, out_dtype=torch.float32)
         idx, wts, offsets, slot_of, slot_token, slot_wts = ops.moe_route_plan(
             z[:, :n], self.correction32, self.top, self.groups, self.keep, self.normalize, self.scoring,
@@ -135,7 +136,7 @@ class RoutedExperts(FeedForward):
             y = x
         shared = None
         if self.shared_ff is not None:
-            shared = self.shared_ff.forward(x, inputs)
+            shared = beside.join()
         elif self.shared_size:
             gu = ops.linear(x, self.w_shared_gu, out_dtype=self.ctx.dtype)
             shared = ops.linear(ops.swiglu(gu, activation=self.activation, limit=self.shared_limit), self.w_shared_down,

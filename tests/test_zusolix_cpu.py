@@ -8,7 +8,7 @@ import pytest
 import torch
 
 from acorninfer_b200.config.model_config import ConfigError, ZusolixConfig
-from acorninfer_b200.kernels.ops import GRU_SEGMENT, GRU_WALK_TOKENS, gru_segments
+from acorninfer_b200.kernels.ops import GRU_WALK_TOKENS, gru_walks
 from acorninfer_b200.models.decoder import Decoder, expected_tensors
 from acorninfer_b200.parts.base import TensorSpec
 from acorninfer_b200.registry import config_from_dict, spec_for
@@ -112,11 +112,9 @@ def test_coefficients_drawn_at_random_lean_on_the_newest_result():
         assert torch.equal(random_tensor("l4.dwa", spec, 3, 0.02, 0.0, torch.float32, rows=(a, b)), t[a:b])
 
 
-def test_segments_of_the_recurrence():
-    assert gru_segments(1, 64) == 0 and gru_segments(GRU_WALK_TOKENS, 3) == 0
-    assert gru_segments(GRU_WALK_TOKENS + 1, 1) == 1 and gru_segments(GRU_SEGMENT, 1) == 1
-    assert gru_segments(GRU_SEGMENT + 1, 2) == 2 and gru_segments(2048, 1) == 2048 // GRU_SEGMENT
-    assert gru_segments(8192, 2000) == 0                       # more blocks than a grid holds
+def test_rows_of_the_recurrence_that_are_walked():
+    assert gru_walks(1, 64) and gru_walks(GRU_WALK_TOKENS, 3) and not gru_walks(GRU_WALK_TOKENS + 1, 1) and not gru_walks(8192, 16)
+    assert gru_walks(8192, 2000)                               # more chunks than a grid holds
 
 
 def test_plain_implementation_properties(tmp_path):

@@ -476,7 +476,7 @@ def test_min_gru_kernel(width, dtype, tol):
                       torch.tensor(slot_ids, dtype=torch.int32, device=DEV), len(parts), longest_row=longest)
         return [t.float().cpu() for t in torch.split(y, [p.shape[0] for p in parts])]
 
-    for lens in ([1, 1, 1], [4, 1, 3], [5, 2, 8, 1], [128, 127, 9], [129, 1, 128], [300, 2, 40, 257], [2200, 130]):
+    for lens in ([1, 1, 1], [7, 1, 9], [32, 2, 8, 31], [33, 1, 8], [128, 127, 9], [129, 1, 128], [300, 2, 40, 257], [2048, 130], [2300]):
         if sum(lens) > 1000 and width > 140:
             continue
         rows = [_rand(g, n, 3 * width, dtype=dtype) for n in lens]
@@ -493,7 +493,7 @@ def test_min_gru_kernel(width, dtype, tol):
         for i in ids:
             touched[i, off:off + width] = True
         assert torch.equal(after[~touched], before[~touched])
-        for cut in (1, 2, 127, 128, 130):
+        for cut in (1, 2, 33, 127, 128, 130):
             if cut >= lens[0]:
                 continue
             st = before.to(DEV)
