@@ -148,6 +148,26 @@ def test_mixed_trace_uses_pages_and_slots_again(case):
     assert sum(1 for users in pages.values() if len(users) >= 2) >= 2, pages
 
 
+def test_branches_of_a_captured_step_change_nothing(case):
+    """Decoding four requests at a time from captured graphs, whose layers run their two sublayers (and the shared expert) as
+    branches side by side, against the same steps launched one by one."""
+    from acorninfer_b200.engine.batch import StepEntry
+    from acorninfer_b200.engine.runner import ModelRunner
+    tiny, d, reqs, _ = case
+    for dtype, tol in (("float32", 1e-6), ("bfloat16", 1e-3)):
+        out = {}
+        for graph in (True, False):
+            runner = ModelRunner.from_model_dir(d, dtype=dtype, num_blocks=96, page_size=tiny["page_size"], max_requests=4,
+                                                max_step_tokens=256, decode_graph=graph)
+            rcs = [runner.open(f"g{i}") for i in range(4)]
+            toks = [reqs[f"r{i}"][:28] for i in range(4)]
+            runner.step([StepEntry(rc, t[:5], [4]) for rc, t in zip(rcs, toks)])
+            out[graph] = torch.stack([runner.step([StepEntry(rc, [t[j]], [0]) for rc, t in zip(rcs, toks)]).clone()
+                                      for j in range(5, 28)])
+            assert (runner.graph_replays > 10) == graph
+        assert (out[True] - out[False]).abs().max() < tol * max(1.0, float(out[False].abs().max())), dtype
+
+
 def test_first_step_of_one_token_and_requests_left_out(case):
     """A request whose first step is a single token (a recurrence from the zero state, a softmax of one key), then
     portions beside another request that decodes and is left out of some steps."""
