@@ -1160,6 +1160,224 @@ class ZusolixConfig(ModelConfig):
 _ZUSOLIX_MIXERS = {c.kind: c for c in (TemperedAttentionConfig, MinGRUConfig)}
 
 
+# --------------------------------------------------------------------------- Badepel
+
+
+@dataclass(frozen=True)
+class RowNormAttentionConfig:
+    """Grouped-query attention with biased projections, a short convolution over time on q, k and v, a q/k norm over whole
+    projected rows, neighbouring rotary pairs, capped scores, a sliding window and one added to the softmax denominator."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    conv: int | None = None
+    softcap: float | None = None
+    window: int | None = None
+    rot_dims: int = 0
+    rot_base: float = 10000.0
+
+    @classmethod
+    def from_dict(cls, m: dict, where: str) -> "RowNormAttentionConfig":
+        mask, rot = _sub(m, "mask", where, required=False), _sub(m, "rot", where, required=False)
+        return cls(heads=_take(m, "heads", int), kv_heads=_take(m, "kv_heads", int), dim=_take(m, "dim", int),
+                   vdim=_take(m, "vdim", int), scale=_take(m, "scale", float), conv=_take(m, "conv", int, None),
+                   softcap=_take(m, "softcap", float, None), window=None if mask is None else _take(mask, "size", int, None),
+                   rot_dims=0 if rot is None else _take(rot, "dims", int), rot_base=10000.0 if rot is None else _take(rot, "base", float))
+
+    def check(self, where: str) -> None:
+        if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1 or self.heads % self.kv_heads:
+            raise ConfigError(f"config.json: {where}sizes must be >= 1 and 'heads' a multiple of 'kv_heads'")
+        if self.conv is not None and self.conv < 1:
+            raise ConfigError(f"config.json: {where}conv must be >= 1, got {self.conv}")
+        if self.softcap is not None and not self.softcap > 0:
+            raise ConfigError(f"config.json: {where}softcap must be > 0, got {self.softcap}")
+        if self.window is not None and self.window < 1:
+            raise ConfigError(f"config.json: {where}mask.size must be >= 1, got {self.window}")
+        if self.rot_dims % 2 or not (0 <= self.rot_dims <= self.dim) or not self.rot_base > 0:
+            raise ConfigError(f"config.json: {where}rot.dims must be even and in 0..{self.dim} and rot.base > 0")
+
+    def to_dict(self) -> dict:
+        out: dict = {"dim": self.dim, "heads": self.heads, "kv_heads": self.kv_heads, "scale": self.scale, "vdim": self.vdim}
+        if self.conv is not None:
+            out["conv"] = self.conv
+        if self.softcap is not None:
+            out["softcap"] = self.softcap
+        if self.window is not None:
+            out["mask"] = {"size": self.window}
+        if self.rot_dims:
+            out["rot"] = {"base": self.rot_base, "dims": self.rot_dims}
+        return out
+
+
+@dataclass(frozen=True)
+class GatedLinearConfig:
+    """Gated linear attention: a decay per key channel, ``sigmoid(.)^(1 / tau)``.  ``decay_rank`` is not in ``config.json``: the
+    checkpoint's tensor shapes fix it (it is needed only to make a model from nothing)."""
+
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    decay_rank: int | None = None
+
+    @classmethod
+    def from_dict(cls, m: dict, where: str) -> "GatedLinearConfig":
+        return cls(heads=_take(m, "heads", int), dim=_take(m, "dim", int), vdim=_take(m, "vdim", int), tau=_take(m, "tau", float),
+                   decay_rank=_take(m, "decay_rank", int, None))
+
+    def check(self, where: str) -> None:
+        if min(self.heads, self.dim, self.vdim) < 1 or (self.decay_rank is not None and self.decay_rank < 1):
+            raise ConfigError(f"config.json: {where}sizes must be >= 1")
+        if not self.tau > 0:
+            raise ConfigError(f"config.json: {where}tau must be > 0, got {self.tau}")
+
+    def to_dict(self) -> dict:
+        out: dict = {"dim": self.dim, "heads": self.heads, "tau": self.tau, "vdim": self.vdim}
+        if self.decay_rank is not None:
+            out["decay_rank"] = self.decay_rank
+        return out
+
+
+@dataclass(frozen=True)
+class AttentionBesideLinearConfig:
+    """Attention (left) and gated linear attention (right) on the same input, their results scaled and added."""
+
+    kind: ClassVar[str] = "parallel"
+    left: RowNormAttentionConfig
+    right: GatedLinearConfig
+    left_scale: float
+    right_scale: float
+
+    @classmethod
+    def from_dict(cls, m: dict, where: str) -> "AttentionBesideLinearConfig":
+        return cls(left=RowNormAttentionConfig.from_dict(_sub(m, "left", where), where + "left."),
+                   right=GatedLinearConfig.from_dict(_sub(m, "right", where), where + "right."),
+                   left_scale=_take(m, "left_scale", float), right_scale=_take(m, "right_scale", float))
+
+    def check(self, where: str) -> None:
+        self.left.check(where + "left.")
+        self.right.check(where + "right.")
+
+    def to_dict(self) -> dict:
+        return {"left": self.left.to_dict(), "left_scale": self.left_scale, "right": self.right.to_dict(),
+                "right_scale": self.right_scale}
+
+
+@dataclass(frozen=True)
+class HeadDeltaConfig:
+    """A gated delta rule with one decay per head and short convolutions on q, k and v."""
+
+    kind: ClassVar[str] = "delta"
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int | None = None
+
+    @classmethod
+    def from_dict(cls, m: dict, where: str) -> "HeadDeltaConfig":
+        return cls(heads=_take(m, "heads", int), kv_heads=_take(m, "kv_heads", int), dim=_take(m, "dim", int),
+                   vdim=_take(m, "vdim", int), conv=_take(m, "conv", int, None))
+
+    def check(self, where: str) -> None:
+        if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1 or self.heads % self.kv_heads:
+            raise ConfigError(f"config.json: {where}sizes must be >= 1 and 'heads' a multiple of 'kv_heads'")
+        if self.conv is not None and self.conv < 1:
+            raise ConfigError(f"config.json: {where}conv must be >= 1, got {self.conv}")
+
+    def to_dict(self) -> dict:
+        out: dict = {"dim": self.dim, "heads": self.heads, "kv_heads": self.kv_heads, "vdim": self.vdim}
+        if self.conv is not None:
+            out["conv"] = self.conv
+        return out
+
+
+@dataclass(frozen=True)
+class BadepelLayer:
+    type: str                                   # "parallel" or "delta"
+    mixer: "AttentionBesideLinearConfig | HeadDeltaConfig"
+    ff: "int | CappedExpertsConfig | None"      # inner width of the dense gated feed-forward; routed experts; none
+
+
+@dataclass(frozen=True)
+class BadepelConfig(ModelConfig):
+    """Badepel: pre-norm layers between several residual streams (hyper-connections), whose mixer is attention beside gated
+    linear attention, or a gated delta rule with one decay per head; the feed-forward is gated with silu, or a routed mixture
+    of capped experts (weights: the softmax over the chosen) beside a shared one.  The streams' sum, a norm and an output
+    matrix of its own end the model.  ``config.json`` lists the layers in order; ``streams`` absent: one plain residual stream."""
+
+    architecture: ClassVar[str] = "Badepel"
+
+    vocab_size: int
+    hidden_size: int
+    norm_eps: float
+    layers: tuple[BadepelLayer, ...]
+    streams: int | None = None
+    residual_mult: float = 1.0
+    eos_token_id: tuple[int, ...] = field(default_factory=tuple)
+
+    def __post_init__(self) -> None:
+        if self.vocab_size < 1 or self.hidden_size < 1 or not self.layers:
+            raise ConfigError("config.json: 'vocab', 'width' must be >= 1 and 'layers' non-empty")
+        if not self.norm_eps > 0:
+            raise ConfigError(f"config.json: norm 'eps' must be > 0, got {self.norm_eps}")
+        if self.streams is not None and not (1 <= self.streams <= MAX_STREAMS):
+            raise ConfigError(f"config.json: 'streams' must be in 1..{MAX_STREAMS}, got {self.streams}")
+        for i, layer in enumerate(self.layers):
+            layer.mixer.check(f"layers[{i}].mixer.")
+            if isinstance(layer.ff, CappedExpertsConfig):
+                layer.ff.check(f"layers[{i}].mlp.")
+            elif layer.ff is not None and layer.ff < 1:
+                raise ConfigError(f"config.json: layers[{i}].mlp.ff must be >= 1, got {layer.ff}")
+
+    @classmethod
+    def from_dict(cls, raw: dict) -> "BadepelConfig":
+        layers_raw = raw.get("layers")
+        if not isinstance(layers_raw, list) or not layers_raw:
+            raise ConfigError("config.json: 'layers' must be a non-empty list")
+        layers = []
+        for i, lr in enumerate(layers_raw):
+            where = f"layers[{i}]."
+            kind = lr.get("type") if isinstance(lr, dict) else None
+            if kind not in _BADEPEL_MIXERS:
+                raise ConfigError(f"config.json: {where}'type' must be one of {sorted(_BADEPEL_MIXERS)}, got {kind!r}")
+            mixer = _BADEPEL_MIXERS[kind].from_dict(_sub(lr, "mixer", where), where + "mixer.")
+            mlp = _sub(lr, "mlp", where, required=False)
+            if mlp is None:
+                ff = None
+            elif mlp.get("kind", "dense") == "dense":
+                ff = _take(mlp, "ff", int)
+            elif mlp.get("kind") == "moe":
+                ff = CappedExpertsConfig.from_dict(mlp, where + "mlp.")
+            else:
+                raise ConfigError(f"config.json: {where}mlp.kind must be 'dense' or 'moe', got {mlp.get('kind')!r}")
+            layers.append(BadepelLayer(kind, mixer, ff))
+        eos = raw.get("eos_token_id")
+        eos_ids = () if eos is None else tuple(int(e) for e in (eos if isinstance(eos, (list, tuple)) else [eos]))
+        return cls(vocab_size=_take(raw, "vocab", int), hidden_size=_take(raw, "width", int),
+                   norm_eps=_take(_sub(raw, "norm", ""), "eps", float), layers=tuple(layers), streams=_take(raw, "streams", int, None),
+                   residual_mult=_take(raw, "residual_mult", float, 1.0), eos_token_id=eos_ids)
+
+    def to_dict(self) -> dict:
+        out: dict = {"architecture": self.architecture, "vocab": self.vocab_size, "width": self.hidden_size,
+                     "norm": {"eps": self.norm_eps}, "residual_mult": self.residual_mult}
+        if self.streams is not None:
+            out["streams"] = self.streams
+        out["layers"] = [{"type": l.type, "mixer": l.mixer.to_dict(),
+                          "mlp": None if l.ff is None else l.ff.to_dict() if isinstance(l.ff, CappedExpertsConfig)
+                          else {"ff": l.ff, "kind": "dense"}} for l in self.layers]
+        if self.eos_token_id:
+            out["eos_token_id"] = list(self.eos_token_id)
+        return out
+
+
+MAX_STREAMS = 8                  # residual streams the kernel between sublayers takes
+_BADEPEL_MIXERS = {c.kind: c for c in (AttentionBesideLinearConfig, HeadDeltaConfig)}
+
+
 def read_config_json(model_dir: str | Path) -> dict:
     path = Path(model_dir) / "config.json"
     if not path.is_file():

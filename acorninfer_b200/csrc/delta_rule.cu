@@ -166,7 +166,12 @@ __device__ __forceinline__ void cp_async_4(float* dst, const float* src) {
 //     o = S^T q + (sum_d q[d] u[d] k[d]) v,      S[d] = g[d] S[d] + k[d] v.
 // It is the same loop with gq = q, no sum against gk, beta = 1 and the bonus inside the k . q sum.
 //
-// In that form the state moves by S <- diag(g) S + k v^T, so a long row can be cut into segments that run side
+// DELTA_FORM_LINEAR (gated linear attention): S[d] = g[d] S[d] + k[d] v, then o = S^T q, so the token's own write counts:
+// the loop with gq = g q, no sum against gk, beta = 1 and the plain k . q sum.
+//
+// The decay may be one number per head and token instead of one per key channel (g_heads): g is then [T, H].
+//
+// In the two forms without the delta correction the state moves by S <- diag(g) S + k v^T, so a long row can be cut into segments that run side
 // by side (a recurrence is sequential over a row's tokens, and a prompt alone in its step would otherwise keep
 // a few dozen blocks busy): pass 1 runs every segment from a zero state to its end state E_j and multiplies up its
 // decays P_j; delta_fold walks the segments, S_j = diag(P_(j-1)) S_(j-1) + E_(j-1), leaving each segment's true
@@ -179,12 +184,17 @@ struct DeltaSegments {
     float* seg_decay;         // [rows * nseg, H, dim]
 };
 // CPT: columns a thread holds (an entry read from shared memory then serves them all); NT: threads a block.
-template <int DPT, int DELTA_SLICES, bool PRE, int CPT, int NT>
+#define DELTA_FORM_RULE 0
+#define DELTA_FORM_PRE 1
+#define DELTA_FORM_LINEAR 2
+template <int DPT, int DELTA_SLICES, int FORM, int CPT, int NT>
 __global__ void __launch_bounds__(NT) delta_rule_kernel(
     const float* __restrict__ qn, const float* __restrict__ kn, const float* __restrict__ vv,
     const float* __restrict__ beta, const float* __restrict__ g, float* __restrict__ state, int64_t slot_stride,
     const int* __restrict__ row_start, const int* __restrict__ row_slot, float* __restrict__ out, int H, int KH, int dim,
-    int vdim, int stage, const float* __restrict__ bonus, DeltaSegments sg) {
+    int vdim, int stage, const float* __restrict__ bonus, int g_heads, DeltaSegments sg) {
+    constexpr bool PRE = FORM == DELTA_FORM_PRE;
+    constexpr bool RULE = FORM == DELTA_FORM_RULE;
     constexpr int DELTA_COLS = NT / DELTA_SLICES * CPT;                // value channels a block
     extern __shared__ __align__(16) float sm[];
     constexpr int DIMP = DPT * DELTA_SLICES;                           // dim rounded up: entries beyond dim are zero
@@ -193,6 +203,7 @@ __global__ void __launch_bounds__(NT) delta_rule_kernel(
     float* sv = raw + (size_t)2 * stage * 3 * dim;                     // [2][stage][COLS]
     float* sb = sv + 2 * stage * DELTA_COLS;                           // [2][stage]
     float* skq = sb + 2 * stage;                                       // [stage]
+    float* sgh = skq + stage;                                          // [2][stage] decays, where they are per head
     pdl_wait();
     pdl_trigger();
     const int r = sg.pass ? blockIdx.x / sg.nseg : blockIdx.x, seg = sg.pass ? blockIdx.x % sg.nseg : 0;
@@ -229,7 +240,7 @@ __global__ void __launch_bounds__(NT) delta_rule_kernel(
             const int64_t t = t0 + tt;
             cp_async_4(rw + (tt * 3 + 0) * dim + d, qn + (t * KH + kh) * dim + d);
             cp_async_4(rw + (tt * 3 + 1) * dim + d, kn + (t * KH + kh) * dim + d);
-            cp_async_4(rw + (tt * 3 + 2) * dim + d, g + (t * H + h) * dim + d);
+            if (!g_heads) cp_async_4(rw + (tt * 3 + 2) * dim + d, g + (t * H + h) * dim + d);
         }
         for (int e = threadIdx.x; e < n * DELTA_COLS; e += blockDim.x) {
             const int tt = e / DELTA_COLS, cc = e % DELTA_COLS;
@@ -237,7 +248,8 @@ __global__ void __launch_bounds__(NT) delta_rule_kernel(
             if (c0 + cc < vdim) cp_async_4(dst, vv + ((int64_t)(t0 + tt) * H + h) * vdim + c0 + cc);
             else *dst = 0.f;
         }
-        if (!PRE && threadIdx.x < n) cp_async_4(sb + (s & 1) * stage + threadIdx.x, beta + (int64_t)(t0 + threadIdx.x) * H + h);
+        if (g_heads && threadIdx.x < n) cp_async_4(sgh + (s & 1) * stage + threadIdx.x, g + (int64_t)(t0 + threadIdx.x) * H + h);
+        if (RULE && threadIdx.x < n) cp_async_4(sb + (s & 1) * stage + threadIdx.x, beta + (int64_t)(t0 + threadIdx.x) * H + h);
     };
 
     if (stages > 0) fetch(0);
@@ -253,7 +265,8 @@ __global__ void __launch_bounds__(NT) delta_rule_kernel(
             const int tt = e / DIMP, d = e % DIMP;
             float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
             if (d < dim) {
-                const float q = rw[(tt * 3 + 0) * dim + d], k = rw[(tt * 3 + 1) * dim + d], gg = rw[(tt * 3 + 2) * dim + d];
+                const float q = rw[(tt * 3 + 0) * dim + d], k = rw[(tt * 3 + 1) * dim + d], 
+                            gg = g_heads ? sgh[(s & 1) * stage + tt] : rw[(tt * 3 + 2) * dim + d];
                 v = PRE ? make_float4(0.f, q, gg, k) : make_float4(gg * k, gg * q, gg, k);
             }
             pack[e] = v;
@@ -279,31 +292,31 @@ __global__ void __launch_bounds__(NT) delta_rule_kernel(
 #pragma unroll
             for (int j = 0; j < CPT; ++j) {
                 float a = 0.f, b = 0.f;
-                if (!PRE || sg.pass != 1) {                            // a segment's first pass writes no output
+                if (RULE || sg.pass != 1) {                            // a segment's first pass writes no output
                     float a0 = 0.f, a1 = 0.f, b0 = 0.f, b1 = 0.f;
 #pragma unroll
                     for (int i = 0; i < DPT; i += 2) {
-                        if (!PRE) a0 = fmaf(S[j][i], e[i].x, a0);
+                        if (RULE) a0 = fmaf(S[j][i], e[i].x, a0);
                         b0 = fmaf(S[j][i], e[i].y, b0);
-                        if (!PRE) a1 = fmaf(S[j][i + 1], e[i + 1].x, a1);
+                        if (RULE) a1 = fmaf(S[j][i + 1], e[i + 1].x, a1);
                         b1 = fmaf(S[j][i + 1], e[i + 1].y, b1);
                     }
                     a = a0 + a1;
                     b = b0 + b1;
 #pragma unroll
                     for (int o = 1; o < DELTA_SLICES; o <<= 1) {
-                        if (!PRE) a += __shfl_xor_sync(0xffffffffu, a, o);
+                        if (RULE) a += __shfl_xor_sync(0xffffffffu, a, o);
                         b += __shfl_xor_sync(0xffffffffu, b, o);
                     }
                 }
                 const float vj = v_s[tt * DELTA_COLS + col * CPT + j];
-                const float u = PRE ? vj : b_s[tt] * (vj - a);
+                const float u = RULE ? b_s[tt] * (vj - a) : vj;
                 if (slice == 0 && live[j] && sg.pass != 1)
                     out[((int64_t)(t0 + tt) * H + h) * vdim + column + j] = fmaf(skq[tt], u, b);
 #pragma unroll
                 for (int i = 0; i < DPT; ++i) S[j][i] = fmaf(e[i].w, u, e[i].z * S[j][i]);
             }
-            if (PRE && sg.pass == 1) {
+            if (!RULE && sg.pass == 1) {
 #pragma unroll
                 for (int i = 0; i < DPT; ++i) Pd[i] *= e[i].z;
             }
@@ -346,39 +359,41 @@ __global__ void delta_fold_kernel(float* __restrict__ state, int64_t slot_stride
 
 extern "C" int acorn_delta_rule(const float* qn, const float* kn, const float* vv, const float* beta, const float* g,
                                 float* state, int64_t slot_stride, const int* row_start, const int* row_slot, float* out,
-                                int rows, int H, int KH, int dim, int vdim, const float* bonus, int pass, int nseg,
+                                int rows, int H, int KH, int dim, int vdim, const float* bonus, int form, int g_heads, int pass, int nseg,
                                 int seg_len, float* seg_state, float* seg_decay, cudaStream_t stream) {
     if (rows <= 0) return 0;
     if (H > 65535 || vdim > 65535 || dim > 256 || H % KH) return ACORN_ERR_UNSUPPORTED;
-    if (bonus == nullptr && beta == nullptr) return ACORN_ERR_UNSUPPORTED;
+    if (form < 0 || form > 2 || (form == DELTA_FORM_RULE && beta == nullptr) || (form == DELTA_FORM_PRE && bonus == nullptr))
+        return ACORN_ERR_UNSUPPORTED;
     DeltaSegments sg = {pass, nseg, seg_len, seg_state, seg_decay};
-    if (pass != 0 && (bonus == nullptr || pass < 0 || pass > 2 || nseg < 1 || seg_len < 1 || seg_state == nullptr ||
+    if (pass != 0 && (form == DELTA_FORM_RULE || pass < 0 || pass > 2 || nseg < 1 || seg_len < 1 || seg_state == nullptr ||
                       seg_decay == nullptr || (int64_t)rows * nseg > 0x7fffffff))
-        return ACORN_ERR_UNSUPPORTED;                   // segments fold only in the form that reads the state first
+        return ACORN_ERR_UNSUPPORTED;                   // segments fold only in the forms without the delta correction
     const int grid_rows = pass ? rows * nseg : rows;
     const int stage = dim <= 64 ? 32 : (dim <= 128 ? 16 : 8);
 #define DELTA_LAUNCH(N, SL)                                                                                                   \
     do {                                                                                                                      \
-        if (bonus) DELTA_LAUNCH_AS(N, SL, true, 1, DELTA_THREADS);                                                            \
-        DELTA_LAUNCH_AS(N, SL, false, 1, DELTA_THREADS);                                                                      \
+        if (form == DELTA_FORM_PRE) DELTA_LAUNCH_AS(N, SL, DELTA_FORM_PRE, 1, DELTA_THREADS);                                 \
+        if (form == DELTA_FORM_LINEAR) DELTA_LAUNCH_AS(N, SL, DELTA_FORM_LINEAR, 1, DELTA_THREADS);                           \
+        DELTA_LAUNCH_AS(N, SL, DELTA_FORM_RULE, 1, DELTA_THREADS);                                                            \
     } while (0)
-#define DELTA_LAUNCH_AS(N, SL, PRE, CPT, NT)                                                                                  \
+#define DELTA_LAUNCH_AS(N, SL, FORM, CPT, NT)                                                                                  \
     do {                                                                                                                      \
         const int cols = (NT) / (SL) * (CPT);                                                                                 \
         dim3 block(NT);                                                                                                       \
         dim3 grid(grid_rows, H, (vdim + cols - 1) / cols);                                                                    \
-        const size_t smem = ((size_t)stage * (N) * (SL) * 4 + (size_t)2 * stage * 3 * dim + 2 * stage * cols + 3 * stage) *    \
+        const size_t smem = ((size_t)stage * (N) * (SL) * 4 + (size_t)2 * stage * 3 * dim + 2 * stage * cols + 5 * stage) *    \
                             sizeof(float);                                                                                    \
         static AcornPerDevice configured;                                                                                     \
         if (!configured.seen()) {                                                                                             \
-            cudaError_t e = cudaFuncSetAttribute(delta_rule_kernel<N, SL, PRE, CPT, NT>,                                      \
+            cudaError_t e = cudaFuncSetAttribute(delta_rule_kernel<N, SL, FORM, CPT, NT>,                                      \
                                                  cudaFuncAttributeMaxDynamicSharedMemorySize,                                 \
                                                  100 * 1024);                                                                 \
             if (e != cudaSuccess) return (int)e;                                                                              \
             configured.mark();                                                                                                \
         }                                                                                                                     \
-        return acorn_launch(delta_rule_kernel<N, SL, PRE, CPT, NT>, grid, block, smem, stream, qn, kn, vv, beta, g, state,    \
-                            slot_stride, row_start, row_slot, out, H, KH, dim, vdim, stage, bonus, sg);                       \
+        return acorn_launch(delta_rule_kernel<N, SL, FORM, CPT, NT>, grid, block, smem, stream, qn, kn, vv, beta, g, state,    \
+                            slot_stride, row_start, row_slot, out, H, KH, dim, vdim, stage, bonus, g_heads, sg);                       \
     } while (0)
     // a thread holds few state entries (4; 8 for the widest heads): a warp is alone on its scheduler, so the
     // time of a token is the number of instructions a thread issues for it, and spreading a column over more
@@ -388,10 +403,16 @@ extern "C" int acorn_delta_rule(const float* qn, const float* kn, const float* v
     // that the reads of the packed entries from shared memory weigh most: a column over fewer lanes (more entries a
     // thread, more columns a warp, which share the entries they read) and several columns a thread cut them down
     if (pass != 0) {
-        if (dim <= 32) DELTA_LAUNCH_AS(8, 4, true, 1, 256);
-        if (dim <= 64) DELTA_LAUNCH_AS(8, 8, true, 4, 128);
-        if (dim <= 128) DELTA_LAUNCH_AS(16, 8, true, 2, 256);
-        DELTA_LAUNCH_AS(16, 16, true, 1, 256);
+        if (form == DELTA_FORM_PRE) {
+            if (dim <= 32) DELTA_LAUNCH_AS(8, 4, DELTA_FORM_PRE, 1, 256);
+            if (dim <= 64) DELTA_LAUNCH_AS(8, 8, DELTA_FORM_PRE, 4, 128);
+            if (dim <= 128) DELTA_LAUNCH_AS(16, 8, DELTA_FORM_PRE, 2, 256);
+            DELTA_LAUNCH_AS(16, 16, DELTA_FORM_PRE, 1, 256);
+        }
+        if (dim <= 32) DELTA_LAUNCH_AS(8, 4, DELTA_FORM_LINEAR, 1, 256);
+        if (dim <= 64) DELTA_LAUNCH_AS(8, 8, DELTA_FORM_LINEAR, 4, 128);
+        if (dim <= 128) DELTA_LAUNCH_AS(16, 8, DELTA_FORM_LINEAR, 2, 256);
+        DELTA_LAUNCH_AS(16, 16, DELTA_FORM_LINEAR, 1, 256);
     }
     if (dim <= 16) DELTA_LAUNCH(4, 4);
     if (dim <= 32) DELTA_LAUNCH(4, 8);

@@ -434,8 +434,10 @@ extern "C" int acorn_linear_scan(const float* b, int64_t ldb, const float* c, in
     }
 }
 
+__device__ __forceinline__ float lr_gate(float z, int mode) { return mode == 2 ? z * lr_sigmoid(z) : lr_sigmoid(z); }
+
 // y32 [T, W] in `groups` equal parts.  mode 0: u = y silu(z), out = u / rms_part(u) * weight;
-// mode 1: out = y / rms_part(y) * weight * sigmoid(z).  z = gate[t * ldg + i]; out[t * ldo + i], times out_scale.
+// mode 1: out = y / rms_part(y) * weight * sigmoid(z); mode 2: the same times silu(z).  z = gate[t * ldg + i]; out[t * ldo + i], times out_scale.
 template <typename T>
 __global__ void gated_norm_kernel(const float* __restrict__ y, const T* __restrict__ gate, int64_t ldg,
                                   const float* __restrict__ weight, T* __restrict__ out, int64_t ldo, int W, int groups,
@@ -478,7 +480,7 @@ __global__ void gated_norm_kernel(const float* __restrict__ y, const T* __restri
         for (int k = 0; k < GN_KEEP; ++k) {
             const int i = threadIdx.x + k * blockDim.x;
             if (i < part) {
-                const float u = mode == 0 ? uu[k] * inv * weight[i0 + i] : uu[k] * inv * weight[i0 + i] * lr_sigmoid(zz[k]);
+                const float u = mode == 0 ? uu[k] * inv * weight[i0 + i] : uu[k] * inv * weight[i0 + i] * lr_gate(zz[k], mode);
                 out[t * ldo + i0 + i] = from_float<T>(u * out_scale);
             }
         }
@@ -487,8 +489,51 @@ __global__ void gated_norm_kernel(const float* __restrict__ y, const T* __restri
     for (int i = threadIdx.x; i < part; i += blockDim.x) {
         const float z = to_float(gate[t * ldg + i0 + i]);
         float u = y[t * W + i0 + i];
-        u = mode == 0 ? u * (z * lr_sigmoid(z)) * inv * weight[i0 + i] : u * inv * weight[i0 + i] * lr_sigmoid(z);
+        u = mode == 0 ? u * (z * lr_sigmoid(z)) * inv * weight[i0 + i] : u * inv * weight[i0 + i] * lr_gate(z, mode);
         out[t * ldo + i0 + i] = from_float<T>(u * out_scale);
+    }
+}
+
+// The same for parts that are multiples of four up to 256: a warp a part, up to two vectors of four a lane.
+template <typename T>
+__global__ void gated_norm_vec_kernel(const float* __restrict__ y, const T* __restrict__ gate, int64_t ldg,
+                                      const float* __restrict__ weight, T* __restrict__ out, int64_t ldo, int W, int groups,
+                                      float eps, int mode, float out_scale, int64_t items) {
+    pdl_wait();
+    pdl_trigger();
+    const int64_t item = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (item >= items) return;
+    const int lane = threadIdx.x & 31, part = W / groups;
+    const int64_t t = item / groups;
+    const int i0 = (int)(item - t * groups) * part;
+    float4 u[2], z[2];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        const int i = 4 * (lane + 32 * k);
+        u[k] = z[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (i < part) {
+            u[k] = *reinterpret_cast<const float4*>(y + t * W + i0 + i);
+            z[k] = Vec4<T>::load(gate + t * ldg + i0 + i);
+            if (mode == 0) {
+                u[k].x *= lr_gate(z[k].x, 2); u[k].y *= lr_gate(z[k].y, 2);
+                u[k].z *= lr_gate(z[k].z, 2); u[k].w *= lr_gate(z[k].w, 2);
+            }
+            ss += u[k].x * u[k].x + u[k].y * u[k].y + u[k].z * u[k].z + u[k].w * u[k].w;
+        }
+    }
+    const float inv = rsqrtf(warp_sum(ss) / (float)part + eps);
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        const int i = 4 * (lane + 32 * k);
+        if (i >= part) break;
+        const float4 w = *reinterpret_cast<const float4*>(weight + i0 + i);
+        float4 o = make_float4(u[k].x * inv * w.x, u[k].y * inv * w.y, u[k].z * inv * w.z, u[k].w * inv * w.w);
+        if (mode != 0) {
+            o.x *= lr_gate(z[k].x, mode); o.y *= lr_gate(z[k].y, mode);
+            o.z *= lr_gate(z[k].z, mode); o.w *= lr_gate(z[k].w, mode);
+        }
+        Vec4<T>::store(out + t * ldo + i0 + i, make_float4(o.x * out_scale, o.y * out_scale, o.z * out_scale, o.w * out_scale));
     }
 }
 
@@ -496,8 +541,18 @@ extern "C" int acorn_gated_norm(const float* y, const void* gate, int64_t ldg, c
                                 int tokens, int W, int groups, float eps, int mode, float out_scale, int dtype,
                                 cudaStream_t stream) {
     if (tokens <= 0) return 0;
-    if (groups < 1 || W % groups || groups > 65535 || mode < 0 || mode > 1) return ACORN_ERR_UNSUPPORTED;
+    if (groups < 1 || W % groups || groups > 65535 || mode < 0 || mode > 2) return ACORN_ERR_UNSUPPORTED;
     const int part = W / groups;
+    if (part % 4 == 0 && part <= 256 && ldg % 4 == 0 && ldo % 4 == 0 &&
+        (((uintptr_t)y | (uintptr_t)weight) & 15) == 0 &&
+        (((uintptr_t)gate | (uintptr_t)out) & (dtype == ACORN_DTYPE_BF16 ? 7 : 15)) == 0) {
+        const int64_t items = (int64_t)tokens * groups;
+        const int64_t blocks = (items + 7) / 8;
+        if (blocks > 0x7fffffff) return ACORN_ERR_UNSUPPORTED;
+        ACORN_DISPATCH_DTYPE(dtype, T, return acorn_launch(gated_norm_vec_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, y,
+                                                           (const T*)gate, ldg, weight, (T*)out, ldo, W, groups, eps, mode,
+                                                           out_scale, items));
+    }
     const int threads = part >= 1024 ? 256 : 128;
     ACORN_DISPATCH_DTYPE(dtype, T, return acorn_launch(gated_norm_kernel<T>, dim3(tokens, groups), dim3(threads), 0, stream,
                                                        y, (const T*)gate, ldg, weight, (T*)out, ldo, W, groups, eps, mode,

@@ -1,7 +1,7 @@
 // A routed mixture of experts: the router's choice, the grouping of tokens by expert, a matrix
 // product per expert over its tokens, and the weighted sum.
 //
-//   moe_route     per token: s = softmax(z) over all N router outputs, or sigmoid(z) of each; the choice score is
+//   moe_route     per token: a bias per output on the logits z, if given; then s = softmax(z) over all N router outputs, or sigmoid(z) of each; the choice score is
 //                 s + correction (no correction: z itself, in whose order the scores stand); the outputs form `groups` equal groups of neighbours, a group's score is its largest choice
 //                 score, and only outputs of the `keep` best groups can be chosen; the `top` largest choice
 //                 scores win; their weights are s itself, or with `normalize` s over the chosen's sum
@@ -17,25 +17,27 @@
 #include "mma_helpers.cuh"
 
 // One warp per token.  Ties go to the lower index.
-__device__ __forceinline__ void route_token(const float* __restrict__ z, int64_t ldz, const float* __restrict__ correction,
+__device__ __forceinline__ void route_token(const float* __restrict__ z, int64_t ldz, const float* __restrict__ bias,
+                                            const float* __restrict__ correction,
                                             int* __restrict__ idx, float* __restrict__ wts, int t, int N, int top, int groups,
                                             int keep, int normalize, int scoring, float* s) {
     const int lane = threadIdx.x & 31;
     float* choice = s + N;                              // s[N], choice[N]: this warp's
     const float* zr = z + (int64_t)t * ldz;
     float m = -INFINITY;
-    for (int i = lane; i < N; i += 32) m = fmaxf(m, zr[i]);
+    auto logit = [&](int i) -> float { return bias ? zr[i] + bias[i] : zr[i]; };
+    for (int i = lane; i < N; i += 32) m = fmaxf(m, logit(i));
     m = warp_max(m);
     float sum = 0.f;
     for (int i = lane; i < N; i += 32) {
-        const float e = scoring == 1 ? 1.f / (1.f + expf(-zr[i])) : expf(zr[i] - m);
+        const float e = scoring == 1 ? 1.f / (1.f + expf(-logit(i))) : expf(logit(i) - m);
         s[i] = e;
         sum += e;
     }
     sum = scoring == 1 ? 1.f : warp_sum(sum);
     for (int i = lane; i < N; i += 32) {
         s[i] = s[i] / sum;
-        choice[i] = correction ? s[i] + correction[i] : zr[i];
+        choice[i] = correction ? s[i] + correction[i] : logit(i);
     }
     __syncwarp();
     if (groups > 1 && keep < groups) {
@@ -104,7 +106,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z, int64_t
     }
 }
 
-__global__ void moe_route_kernel(const float* __restrict__ z, int64_t ldz, const float* __restrict__ correction,
+__global__ void moe_route_kernel(const float* __restrict__ z, int64_t ldz, const float* __restrict__ bias, const float* __restrict__ correction,
                                  int* __restrict__ idx, float* __restrict__ wts, int tokens, int N, int top, int groups,
                                  int keep, int normalize, int scoring) {
     extern __shared__ float sm[];
@@ -113,11 +115,11 @@ __global__ void moe_route_kernel(const float* __restrict__ z, int64_t ldz, const
     const int warp = threadIdx.x >> 5;
     const int t = blockIdx.x * (blockDim.x >> 5) + warp;
     if (t >= tokens) return;
-    route_token(z, ldz, correction, idx, wts, t, N, top, groups, keep, normalize, scoring, sm + (size_t)warp * 2 * N);
+    route_token(z, ldz, bias, correction, idx, wts, t, N, top, groups, keep, normalize, scoring, sm + (size_t)warp * 2 * N);
 }
 
-// scoring 0: softmax over the outputs; 1: the sigmoid of each.  correction may be null.
-extern "C" int acorn_moe_route(const float* z, int64_t ldz, const float* correction, int* idx, float* wts, int tokens, int N,
+// scoring 0: softmax over the outputs; 1: the sigmoid of each.  bias (on the logits) and correction may be null.
+extern "C" int acorn_moe_route(const float* z, int64_t ldz, const float* bias, const float* correction, int* idx, float* wts, int tokens, int N,
                                int top, int groups, int keep, int normalize, int scoring, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (scoring < 0 || scoring > 1 || ldz < N) return ACORN_ERR_UNSUPPORTED;
@@ -131,8 +133,8 @@ extern "C" int acorn_moe_route(const float* z, int64_t ldz, const float* correct
         if (e != cudaSuccess) return (int)e;
         configured.mark();
     }
-    return acorn_launch(moe_route_kernel, dim3((tokens + warps - 1) / warps), dim3(32 * warps), smem, stream, z, ldz, correction,
-                        idx, wts, tokens, N, top, groups, keep, normalize, scoring);
+    return acorn_launch(moe_route_kernel, dim3((tokens + warps - 1) / warps), dim3(32 * warps), smem, stream, z, ldz, bias,
+                        correction, idx, wts, tokens, N, top, groups, keep, normalize, scoring);
 }
 
 // One block: histogram of the chosen outputs, exclusive sums, then a slot for every pair.  Within an
@@ -177,7 +179,8 @@ __global__ void moe_plan_kernel(const int* __restrict__ idx, int* __restrict__ o
 #define MOE_SMALL_TOKENS 128
 #define MOE_SMALL_OUTPUTS 160
 
-__global__ void __launch_bounds__(1024) moe_route_plan_kernel(const float* __restrict__ z, int64_t ldz, const float* __restrict__ correction,
+__global__ void __launch_bounds__(1024) moe_route_plan_kernel(const float* __restrict__ z, int64_t ldz, const float* __restrict__ bias,
+                                                              const float* __restrict__ correction,
                                                               int* idx, float* wts, int tokens, int N, int top, int groups, int keep,
                                                               int normalize, int scoring, int* __restrict__ offsets,
                                                               int* __restrict__ slot_of, int* __restrict__ slot_token,
@@ -187,7 +190,7 @@ __global__ void __launch_bounds__(1024) moe_route_plan_kernel(const float* __res
     pdl_trigger();
     const int warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     for (int t = warp; t < tokens; t += warps) {
-        route_token(z, ldz, correction, idx, wts, t, N, top, groups, keep, normalize, scoring, sm + (size_t)warp * 2 * N);
+        route_token(z, ldz, bias, correction, idx, wts, t, N, top, groups, keep, normalize, scoring, sm + (size_t)warp * 2 * N);
         __syncwarp();
     }
     __syncthreads();                                    // what the block's warps wrote to idx and wts is read by all of it
@@ -196,7 +199,7 @@ __global__ void __launch_bounds__(1024) moe_route_plan_kernel(const float* __res
 
 extern "C" int acorn_moe_route_plan_supported(int tokens, int N) { return tokens <= MOE_SMALL_TOKENS && N <= MOE_SMALL_OUTPUTS; }
 
-extern "C" int acorn_moe_route_plan(const float* z, int64_t ldz, const float* correction, int* idx, float* wts, int tokens,
+extern "C" int acorn_moe_route_plan(const float* z, int64_t ldz, const float* bias, const float* correction, int* idx, float* wts, int tokens,
                                     int N, int top, int groups, int keep, int normalize, int scoring, int* offsets,
                                     int* slot_of, int* slot_token, float* slot_wts, cudaStream_t stream) {
     if (tokens <= 0) return 0;
@@ -204,7 +207,7 @@ extern "C" int acorn_moe_route_plan(const float* z, int64_t ldz, const float* co
         groups < 1 || groups > 64 || N % groups || keep < 1 || keep > groups)
         return ACORN_ERR_UNSUPPORTED;
     const int warps = tokens < 8 ? 8 : (tokens > 32 ? 32 : tokens);
-    return acorn_launch(moe_route_plan_kernel, dim3(1), dim3(32 * warps), (size_t)warps * 2 * N * sizeof(float), stream, z, ldz,
+    return acorn_launch(moe_route_plan_kernel, dim3(1), dim3(32 * warps), (size_t)warps * 2 * N * sizeof(float), stream, z, ldz, bias,
                         correction, idx, wts, tokens, N, top, groups, keep, normalize, scoring, offsets, slot_of, slot_token,
                         slot_wts);
 }

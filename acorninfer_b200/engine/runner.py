@@ -249,6 +249,8 @@ class ModelRunner:
             if self._graph_pool is None:
                 self._graph_pool = torch.cuda.graph_pool_handle()
             torch.cuda.synchronize()
+            # what parts derived for the step they just ran (a table of its angles) is made again inside the graph
+            inputs.extra = {name: t for name, t in inputs.extra.items() if name in plan.extra}
             with torch.cuda.graph(graph, pool=self._graph_pool):
                 out = self.decoder.forward(inputs, self.caches)
             launches = ops.LAUNCHES - before

@@ -139,14 +139,14 @@ class _Sigs:
     acorn_conv_state_update = [c_void_p, c_int64, c_void_p, c_int64, c_int64, c_void_p, c_void_p, c_int, c_int, c_int,
                                c_int, c_int, c_void_p, c_void_p]
     acorn_delta_rule = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p,
-                        c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p,
-                        c_void_p]
+                        c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p,
+                        c_void_p, c_void_p]
     acorn_delta_fold = [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]
     acorn_delta_out = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p]
-    acorn_moe_route = [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+    acorn_moe_route = [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                        c_void_p]
     acorn_moe_plan = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p]
-    acorn_moe_route_plan = [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+    acorn_moe_route_plan = [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                             c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]
     acorn_moe_route_plan_supported = [c_int, c_int]
     acorn_grouped_gemm = [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int,
@@ -163,6 +163,20 @@ class _Sigs:
     acorn_min_gru = [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int,
                      c_int, c_int, c_void_p, c_int, c_void_p]
     acorn_min_gru_scratch = [c_int, c_int, c_int]
+    acorn_hyper_norm = [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                        c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
+    acorn_qk_row_norm = [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                         c_void_p, c_int64, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                         c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p]
+    acorn_delta_heads_prep = [c_void_p, c_int64, c_int, c_int, c_void_p, c_int, c_void_p, c_int64, c_int64, c_void_p, c_void_p,
+                              c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                              c_int, c_int, c_int, c_int, c_void_p]
+    acorn_linear_heads_prep = [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p,
+                               c_int, c_int, c_int, c_int, c_int, c_void_p]
+    acorn_recurrent_step = [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64,
+                            c_void_p, c_float, c_void_p, c_int64, c_void_p, c_float, c_float, c_void_p, c_int64, c_void_p,
+                            c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
+    acorn_recurrent_step_supported = [c_int, c_int]
     acorn_diff_combine = [c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_int,
                           c_void_p]
     acorn_pair_rows = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
@@ -549,6 +563,57 @@ def qk_rope_kv(qkv: torch.Tensor, q_weight32: torch.Tensor | None, k_weight32: t
                                1 if norm_after else 0, float(q_temp[0]) if q_temp is not None else 0.0,
                                int(q_temp[1]) if q_temp is not None else 0, _stream()),
         "qk_rope_kv")
+
+
+def qk_row_norm(proj: torch.Tensor, q_weight32: torch.Tensor | None, k_weight32: torch.Tensor | None, cos_sin: torch.Tensor | None,
+                positions: torch.Tensor, token_row: torch.Tensor, block_table: torch.Tensor, page_base: torch.Tensor,
+                k_pages: torch.Tensor, v_pages: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int,
+                interleaved: bool, eps: float, q_out: torch.Tensor, bias32: torch.Tensor | None = None,
+                conv: "ShortConv | None" = None, q_count: int | None = None, k_count: int | None = None,
+                v_scale: float = 1.0) -> None:
+    """Projected rows ``[q | k | v | ...]`` (a row stride is allowed) with a bias and a short convolution over time per channel,
+    q and k normed over all their heads at once (weights [nq d] and [nkv d]; ``q_count`` / ``k_count``: how many of a row's
+    entries count, where heads are padded with zeros), rotated by the step's table (``rope_table``; its width is the
+    rotated part of a head), q to ``q_out``, k and v (times ``v_scale``) into the cache pages."""
+    _rows2(proj, "proj")
+    _rows2(q_out, "q_out", proj.dtype)
+    T = proj.shape[0]
+    channels = (num_heads + num_kv_heads) * head_dim + num_kv_heads * value_dim
+    if proj.shape[1] < channels or q_out.shape != (T, num_heads * head_dim):
+        raise KernelError(f"qk_row_norm: rows {tuple(proj.shape)} / queries {tuple(q_out.shape)} do not fit {channels} channels")
+    _check(k_pages, "k_pages", proj.dtype, 4)
+    _check(v_pages, "v_pages", proj.dtype, 4)
+    if k_pages.shape[1] != num_kv_heads or k_pages.shape[3] != head_dim or tuple(v_pages.shape) != (*k_pages.shape[:3], value_dim):
+        raise KernelError(f"qk_row_norm: cache pages {tuple(k_pages.shape)} / {tuple(v_pages.shape)} do not fit")
+    for w, n, name in ((q_weight32, num_heads * head_dim, "q_norm weight"), (k_weight32, num_kv_heads * head_dim, "k_norm weight"),
+                       (bias32, channels, "bias")):
+        if w is not None:
+            _check(w, name, torch.float32, 1)
+            if w.numel() != n:
+                raise KernelError(f"qk_row_norm: {name} must have {n} entries")
+    rot = 0
+    if cos_sin is not None:
+        _check(cos_sin, "cos_sin", torch.float32, 2)
+        rot = cos_sin.shape[1]
+        if cos_sin.shape[0] != T or rot > head_dim:
+            raise KernelError("qk_row_norm: the table of cosines and sines does not fit")
+    taps = 0
+    if conv is not None:
+        _check(conv.weight32, "conv weight", torch.float32, 2)
+        taps = conv.weight32.shape[1]
+        if conv.weight32.shape[0] != channels or (taps > 1 and conv.state.shape[1] < conv.offset + (taps - 1) * channels):
+            raise KernelError("qk_row_norm: convolution weights or memory do not fit")
+    _check(block_table, "block_table", torch.int32, 2)
+    _ok(lib().acorn_qk_row_norm(proj.data_ptr(), proj.stride(0), q_out.data_ptr(), q_out.stride(0), k_pages.data_ptr(),
+                                v_pages.data_ptr(), _ptr(q_weight32), _ptr(k_weight32), _ptr(conv.weight32) if conv else None, taps,
+                                _ptr(bias32), _ptr(conv.state) if conv else None, conv.state.stride(0) if conv else 0,
+                                conv.offset if conv else 0, _ptr(conv.row_start) if conv else None,
+                                _ptr(conv.row_slot) if conv else None, 1 if conv and conv.update_single else 0,
+                                token_row.data_ptr(), positions.data_ptr(), block_table.data_ptr(), page_base.data_ptr(),
+                                block_table.stride(0), _ptr(cos_sin), T, num_heads, num_kv_heads, head_dim, value_dim,
+                                k_pages.shape[2], rot, 1 if interleaved else 0, int(q_count or num_heads * head_dim),
+                                int(k_count or num_kv_heads * head_dim), float(eps), float(v_scale), dtype_code(proj.dtype), _stream()),
+        "qk_row_norm")
 
 
 class ShortConv:
@@ -1435,7 +1500,7 @@ DELTA_WAVE_BLOCKS = 296             # blocks of the segmented passes that run at
 
 
 def delta_segments(longest_row: int, num_rows: int, heads: int, dim: int, vdim: int) -> tuple[int, int]:
-    """(tokens a segment, segments a row) for the form of ``delta_rule`` that reads the state first; (0, 1): rows in
+    """(tokens a segment, segments a row) for the forms of ``delta_rule`` without the delta correction; (0, 1): rows in
     one piece.  Rows run side by side with heads and tiles of columns; where those are too few to fill the device
     and a row is long, rows are cut into segments that run side by side, at the price of a second pass: as many
     as still run at once (a second wave of blocks would wait for the first)."""
@@ -1447,19 +1512,24 @@ def delta_segments(longest_row: int, num_rows: int, heads: int, dim: int, vdim: 
     return -(-longest_row // nseg), nseg
 
 
+DELTA_FORMS = {"rule": 0, "pre": 1, "linear": 2}
+
+
 def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Tensor | None, g: torch.Tensor,
                state: torch.Tensor, row_start: torch.Tensor, row_slot: torch.Tensor, num_rows: int,
-               bonus32: torch.Tensor | None = None, longest_row: int | None = None) -> torch.Tensor:
-    """The recurrence over every row's tokens from the state in its slot (updated in place): float32
-    o [T, H, vdim].  With ``bonus32`` (float32 [H, dim]) and no ``beta`` the form without the delta correction
-    whose output reads the state before the token's decay and write and sees the token itself through the
-    bonus: ``o = S^T q + (sum_d q_d bonus_d k_d) v;  S = diag(g) S + k v^T``.  In that form, with ``longest_row``
-    (the most tokens a row of the step brings, a host value), long rows of a step with few rows run in segments
-    side by side (``delta_segments``)."""
+               bonus32: torch.Tensor | None = None, longest_row: int | None = None, state_off: int = 0) -> torch.Tensor:
+    """The recurrence over every row's tokens from the state in its slot (at ``state_off``, updated in place): float32
+    o [T, H, vdim].  Three forms: with ``beta`` the delta rule; with ``bonus32`` (float32 [H, dim]) and no ``beta`` the form
+    without the correction whose output reads the state before the token's decay and write and sees the token itself
+    through the bonus: ``o = S^T q + (sum_d q_d bonus_d k_d) v;  S = diag(g) S + k v^T``; with neither gated linear
+    attention: ``S = diag(g) S + k v^T;  o = S^T q``.  Decays ``g``: [T, H, dim], or [T, H], one per head.  In the forms
+    without correction, with ``longest_row`` (the most tokens a row of the step brings, a host value), long rows of a
+    step with few rows run in segments side by side (``delta_segments``)."""
     T, H, vdim = v.shape
     KH, dim = q.shape[1], q.shape[2]
-    if (beta is None) == (bonus32 is None):
-        raise KernelError("delta_rule: give beta (the delta rule) or bonus32 (the form that reads the state first)")
+    if beta is not None and bonus32 is not None:
+        raise KernelError("delta_rule: beta (the delta rule) and bonus32 (the form that reads the state first) exclude one another")
+    form = DELTA_FORMS["rule" if beta is not None else ("pre" if bonus32 is not None else "linear")]
     if bonus32 is not None:
         _check(bonus32, "bonus", torch.float32, 2)
         if bonus32.shape != (H, dim):
@@ -1467,16 +1537,18 @@ def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Te
     for t, n in ((q, "q"), (k, "k"), (v, "v"), (g, "g")) + (((beta, "beta"),) if beta is not None else ()):
         _check(t, n, torch.float32)
     _check(state, "state", torch.float32, 2)
-    if state.shape[1] < H * dim * vdim or g.shape != (T, H, dim) or dim > 256:
-        raise KernelError(f"delta_rule: sizes do not fit (state {tuple(state.shape)}, H={H}, dim={dim}, vdim={vdim})")
+    per_head = g.dim() == 2
+    if state.shape[1] < state_off + H * dim * vdim or g.shape != ((T, H) if per_head else (T, H, dim)) or dim > 256:
+        raise KernelError(f"delta_rule: sizes do not fit (state {tuple(state.shape)}, g {tuple(g.shape)}, H={H}, dim={dim}, vdim={vdim})")
     out = torch.empty((T, H, vdim), dtype=torch.float32, device=v.device)
-    seg_len, nseg = delta_segments(longest_row, num_rows, H, dim, vdim) if (bonus32 is not None and longest_row) else (0, 1)
+    seg_len, nseg = delta_segments(longest_row, num_rows, H, dim, vdim) if (beta is None and longest_row) else (0, 1)
+    s_ptr = state.data_ptr() + 4 * int(state_off)
 
     def run(pass_, seg_state=None, seg_decay=None):
-        _ok(lib().acorn_delta_rule(q.data_ptr(), k.data_ptr(), v.data_ptr(), _ptr(beta), g.data_ptr(), state.data_ptr(),
+        _ok(lib().acorn_delta_rule(q.data_ptr(), k.data_ptr(), v.data_ptr(), _ptr(beta), g.data_ptr(), s_ptr,
                                    state.stride(0), row_start.data_ptr(), row_slot.data_ptr(), out.data_ptr(), num_rows, H,
-                                   KH, dim, vdim, _ptr(bonus32), pass_, nseg, max(seg_len, 1), _ptr(seg_state),
-                                   _ptr(seg_decay), _stream()), "delta_rule", f"pass {pass_}")
+                                   KH, dim, vdim, _ptr(bonus32), form, 1 if per_head else 0, pass_, nseg, max(seg_len, 1),
+                                   _ptr(seg_state), _ptr(seg_decay), _stream()), "delta_rule", f"pass {pass_}")
 
     if nseg == 1:
         run(0)
@@ -1484,7 +1556,7 @@ def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Te
     seg_state = torch.empty((num_rows * nseg, H, dim, vdim), dtype=torch.float32, device=v.device)
     seg_decay = torch.empty((num_rows * nseg, H, dim), dtype=torch.float32, device=v.device)
     run(1, seg_state, seg_decay)
-    _ok(lib().acorn_delta_fold(state.data_ptr(), state.stride(0), row_slot.data_ptr(), seg_state.data_ptr(),
+    _ok(lib().acorn_delta_fold(s_ptr, state.stride(0), row_slot.data_ptr(), seg_state.data_ptr(),
                                seg_decay.data_ptr(), num_rows, nseg, H, dim, vdim, _stream()), "delta_fold")
     run(2, seg_state, seg_decay)
     return out
@@ -1503,6 +1575,100 @@ def delta_out(o32: torch.Tensor, gate32: torch.Tensor, weight32: torch.Tensor, e
     _ok(lib().acorn_delta_out(o32.data_ptr(), gate32.data_ptr(), weight32.data_ptr(), y.data_ptr(), T, H, vdim, float(eps),
                               dtype_code(dtype), 1 if (weight32.numel() == H * vdim and H > 1) else 0, _stream()), "delta_out")
     return y
+
+
+# ------------------------------------------------------------------ recurrent heads: before, after, and a token at once
+
+
+def delta_heads_prep(proj: torch.Tensor, beta_col: int, decay_col: int, conv_w32: torch.Tensor | None, state: torch.Tensor | None,
+                     conv_off: int, a_log32: torch.Tensor, dt_bias32: torch.Tensor, token_row: torch.Tensor,
+                     row_start: torch.Tensor, row_slot: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int,
+                     update_single: bool = False):
+    """For a gated delta rule with one decay per head, of projected rows ``[q | k | v | ...]`` (a row stride is allowed; the
+    write strengths' columns start at ``beta_col``, the decays' at ``decay_col``): convolution over time + silu of the q, k,
+    v channels, unit norms of q and k (q also times dim^-1/2), ``sigmoid``, ``exp(-exp(A_log) softplus(. + dt_bias))``.  Float32
+    (q [T, KH, dim], k, v [T, H, vdim], beta [T, H], g [T, H]).  ``update_single``: the convolution's memory of rows of one
+    token is shifted here (``conv_state_update(skip_single=True)`` does the longer rows)."""
+    _rows2(proj, "proj")
+    T, C = proj.shape[0], 2 * kv_heads * dim + heads * vdim
+    if max(C, beta_col + heads, decay_col + heads) > proj.shape[1] or a_log32.numel() != heads or dt_bias32.numel() != heads:
+        raise KernelError(f"delta_heads_prep: proj {tuple(proj.shape)} or the decay parameters do not fit")
+    taps = 0
+    if conv_w32 is not None:
+        _check(conv_w32, "conv weights", torch.float32, 2)
+        taps = conv_w32.shape[1]
+        if conv_w32.shape[0] != C or (taps > 1 and (state is None or state.shape[1] < conv_off + (taps - 1) * C)):
+            raise KernelError("delta_heads_prep: convolution weights or memory do not fit")
+    f = lambda *shape: torch.empty(shape, dtype=torch.float32, device=proj.device)
+    q, k, v, beta, g = f(T, kv_heads, dim), f(T, kv_heads, dim), f(T, heads, vdim), f(T, heads), f(T, heads)
+    _ok(lib().acorn_delta_heads_prep(proj.data_ptr(), proj.stride(0), int(beta_col), int(decay_col), _ptr(conv_w32), taps, _ptr(state),
+                                     state.stride(0) if state is not None else 0, int(conv_off), a_log32.data_ptr(),
+                                     dt_bias32.data_ptr(), token_row.data_ptr(), row_start.data_ptr(), row_slot.data_ptr(),
+                                     1 if update_single else 0, q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(),
+                                     g.data_ptr(), T, heads, kv_heads, dim, vdim, dtype_code(proj.dtype), _stream()),
+        "delta_heads_prep")
+    return q, k, v, beta, g
+
+
+def linear_heads_prep(proj: torch.Tensor, z32: torch.Tensor, bias32: torch.Tensor, tau: float, heads: int, dim: int, vdim: int):
+    """For gated linear attention, of projected rows ``[q | k | v | ...]``: float32 q (times dim^-1/2), k [T, H, dim], v [T, H, vdim]
+    and the decay per key channel ``sigmoid(z + bias)^(1 / tau)`` [T, H, dim]."""
+    _rows2(proj, "proj")
+    _rows2(z32, "z", torch.float32)
+    _check(bias32, "bias", torch.float32, 1)
+    T = proj.shape[0]
+    if proj.shape[1] < heads * (2 * dim + vdim) or z32.shape != (T, heads * dim) or bias32.numel() != heads * dim:
+        raise KernelError(f"linear_heads_prep: proj {tuple(proj.shape)}, z {tuple(z32.shape)} do not fit")
+    f = lambda *shape: torch.empty(shape, dtype=torch.float32, device=proj.device)
+    q, k, v, g = f(T, heads, dim), f(T, heads, dim), f(T, heads, vdim), f(T, heads, dim)
+    _ok(lib().acorn_linear_heads_prep(proj.data_ptr(), proj.stride(0), z32.data_ptr(), z32.stride(0), bias32.data_ptr(),
+                                      1.0 / float(tau), q.data_ptr(), k.data_ptr(), v.data_ptr(), g.data_ptr(), T, heads, dim, vdim,
+                                      dtype_code(proj.dtype), _stream()), "linear_heads_prep")
+    return q, k, v, g
+
+
+def recurrent_step_ok(dim: int, vdim: int, f32_aligned: tuple = (), rows: tuple = ()) -> bool:
+    """Whether ``recurrent_step`` takes these heads and operands (tensors and offsets in floats of the state)."""
+    if not lib().acorn_recurrent_step_supported(dim, vdim):
+        return False
+    if any((t % 4 if isinstance(t, int) else t.data_ptr() % 16) for t in f32_aligned):
+        return False
+    return all(t.stride(0) % 4 == 0 and t.data_ptr() % (8 if t.dtype == torch.bfloat16 else 16) == 0 for t in rows)
+
+
+def recurrent_step(state: torch.Tensor, state_off: int, row_slot: torch.Tensor, gate: torch.Tensor, norm_w32: torch.Tensor,
+                   eps: float, out: torch.Tensor, heads: int, dim: int, vdim: int, out_scale: float = 1.0, delta=None,
+                   linear=None) -> torch.Tensor:
+    """A step of single-token rows (row r brings token r) through a recurrence and what follows it, in one kernel: the state
+    of every head read and written once, the read-out over its root mean square (per head) times ``norm_w32`` [vdim] times
+    ``silu(gate)`` times ``out_scale``, into ``out`` [T, H vdim].  ``delta`` = (q, k, v, beta, g) of ``delta_heads_prep``: the
+    delta rule; ``linear`` = (proj, z32, bias32, tau) as ``linear_heads_prep`` takes them: gated linear attention."""
+    _check(state, "state", torch.float32, 2)
+    _rows2(gate, "gate")
+    _rows2(out, "out", gate.dtype)
+    T, C = out.shape
+    if C != heads * vdim or gate.shape != out.shape or norm_w32.numel() != vdim or (delta is None) == (linear is None) \
+            or state.shape[1] < state_off + heads * dim * vdim:
+        raise KernelError(f"recurrent_step: out {tuple(out.shape)}, gate {tuple(gate.shape)}, state {tuple(state.shape)} do not fit")
+    q = k = v = beta = g = proj = z = bias = None
+    kv_heads, tau = heads, 1.0
+    if delta is not None:
+        q, k, v, beta, g = delta
+        kv_heads = q.shape[1]
+        if q.shape != (T, kv_heads, dim) or v.shape != (T, heads, vdim) or g.shape != (T, heads):
+            raise KernelError("recurrent_step: the delta rule's inputs do not fit")
+    else:
+        proj, z, bias, tau = linear
+        _rows2(proj, "proj", gate.dtype)
+        if proj.shape[0] != T or proj.shape[1] < heads * (2 * dim + vdim) or z.shape != (T, heads * dim):
+            raise KernelError("recurrent_step: the linear attention's inputs do not fit")
+    _ok(lib().acorn_recurrent_step(1 if delta is not None else 0, _ptr(q), _ptr(k), _ptr(v), _ptr(beta), _ptr(g), _ptr(proj),
+                                   proj.stride(0) if proj is not None else 0, _ptr(z), z.stride(0) if z is not None else 0, _ptr(bias),
+                                   1.0 / float(tau), gate.data_ptr(), gate.stride(0), norm_w32.data_ptr(), float(eps), float(out_scale),
+                                   state.data_ptr() + 4 * int(state_off), state.stride(0), row_slot.data_ptr(), out.data_ptr(),
+                                   out.stride(0), T, heads, kv_heads, dim, vdim, dtype_code(gate.dtype), _stream()),
+        "recurrent_step", "delta" if delta is not None else "linear")
+    return out
 
 
 # ------------------------------------------------------------------ time mixing with a matrix state
@@ -1662,13 +1828,14 @@ class DeltaPair:
 
 @dataclass
 class ExpertsPending:
-    """A routed feed-forward's result before its sum: ``sum_k y[slot_of[t, k]] (+ sigmoid(extra_z[t]) extra[t])``, every
-    choice counted once (its weight went into the expert)."""
+    """A routed feed-forward's result before its sum: ``sum_k wts[t, k] y[slot_of[t, k]] (+ sigmoid(extra_z[t]) extra[t])``; no
+    ``wts``: every choice counts once (its weight went into the expert)."""
 
     y: torch.Tensor                          # [slots, width]
     slot_of: torch.Tensor                    # [tokens, choices] int32
     extra: torch.Tensor | None = None        # [tokens, width]
     extra_z: torch.Tensor | None = None      # [tokens, 1] float32
+    wts: torch.Tensor | None = None          # [tokens, choices] float32
 
 
 class NormedStream:
@@ -1694,6 +1861,8 @@ def stream_norm(x32: torch.Tensor, delta=None, norms=(), out_dtype: torch.dtype 
     a, b, scale = (delta.a, delta.b, delta.scale) if isinstance(delta, DeltaPair) else (delta, None, 1.0)
     experts = b if isinstance(b, ExpertsPending) else None
     if experts is not None:
+        if experts.wts is not None:
+            raise KernelError("stream_norm: a pending result of experts counts every choice once")
         b = None
     results = [t for t in (a, b, experts.y if experts is not None else None, experts.extra if experts is not None else None)
                if t is not None]
@@ -1746,6 +1915,81 @@ def stream_norm(x32: torch.Tensor, delta=None, norms=(), out_dtype: torch.dtype 
         _ptr(w[0]), _ptr(o[0]), _ptr(w[1]), _ptr(o[1]), count, H, groups, eps, dtype_code(dtype), _stream()), "stream_norm",
         f"{n} earlier" if n else "")
     return outs
+
+
+class StreamBundle:
+    """Several residual streams: ``x32`` [n, T, W] float32, or [1, T, W] while all ``n`` are still the same rows; and what the
+    sublayer before still has to write to them (``pending``: its result y [T, W] or ``ExpertsPending``, the matrix ``mix`` [from,
+    to] and the factors ``put`` with which the new streams are made, ``x_t <- sum_s mix[s, t] x_s + scale put[t] y``)."""
+
+    def __init__(self, x32: torch.Tensor, n: int, pending=None):
+        self.x32, self.n, self.pending = x32, int(n), pending
+
+    def read(self, take32: torch.Tensor | None, norm_w32: torch.Tensor, eps: float, dtype: torch.dtype,
+             rows: torch.Tensor | None = None) -> torch.Tensor:
+        """The streams brought up to date and the RMS norm of ``sum_t take32[t] x_t`` (None: of the plain sum) in one kernel.
+        With ``rows`` the norm of those rows only, and the streams are left as they are."""
+        x_out = None
+        if rows is None and self.pending is not None:
+            x_out = self.x32 if self.x32.shape[0] == self.n else torch.empty((self.n, *self.x32.shape[1:]), dtype=torch.float32,
+                                                                              device=self.x32.device)
+        out = hyper_norm(self.x32, self.n, self.pending, take32, norm_w32, eps, dtype, rows=rows, x_out=x_out)
+        if rows is None and self.pending is not None:
+            self.x32, self.pending = x_out, None
+        return out
+
+
+def hyper_norm(x32: torch.Tensor, n: int, pending, take32: torch.Tensor | None, norm_w32: torch.Tensor, eps: float,
+               dtype: torch.dtype, rows: torch.Tensor | None = None, x_out: torch.Tensor | None = None) -> torch.Tensor:
+    """See ``StreamBundle``.  ``pending``: None or (y [T, W] or ``ExpertsPending``, mix32 [n, n], put32 [n], scale); the new streams
+    go to ``x_out`` [n, T, W] (``x32`` itself is allowed when it holds all n)."""
+    _check(x32, "streams", torch.float32, 3)
+    _, T, W = x32.shape
+    if x32.shape[0] not in (1, n):
+        raise KernelError(f"hyper_norm: {x32.shape[0]} rows of streams for {n} streams")
+    _check(norm_w32, "norm weight", torch.float32, 1)
+    if norm_w32.numel() != W or (take32 is not None and take32.numel() != n):
+        raise KernelError("hyper_norm: norm weight or read-out factors do not fit")
+    a = experts = mix = put = None
+    scale = 1.0
+    if pending is not None:
+        y, mix, put, scale = pending
+        _check(mix, "mix", torch.float32, 2)
+        _check(put, "put", torch.float32, 1)
+        if mix.shape != (n, n) or put.numel() != n:
+            raise KernelError(f"hyper_norm: mix {tuple(mix.shape)} / put {put.numel()} for {n} streams")
+        if isinstance(y, ExpertsPending):
+            experts = y
+            _check(y.y, "expert outputs", dtype, 2)
+            _check(y.slot_of, "slot_of", torch.int32, 2)
+            if y.extra_z is not None or y.slot_of.shape[0] != T or y.y.shape[1] != W or y.y.shape[0] < y.slot_of.numel():
+                raise KernelError("hyper_norm: the experts' pending result does not fit")
+            if y.extra is not None:
+                _check(y.extra, "extra", dtype, 2)
+            if y.wts is not None:
+                _check(y.wts, "weights", torch.float32, 2)
+        else:
+            a = y
+            _check(a, "pending result", dtype, 2)
+            if a.shape != (T, W):
+                raise KernelError(f"hyper_norm: a pending result {tuple(a.shape)} does not fit the streams {tuple(x32.shape)}")
+    count = T
+    if rows is not None:
+        _check(rows, "rows", torch.int32, 1)
+        count = rows.numel()
+    if x_out is not None:
+        _check(x_out, "x_out", torch.float32, 3)
+        if x_out.shape != (n, T, W):
+            raise KernelError("hyper_norm: x_out does not fit")
+    out = torch.empty((count, W), dtype=dtype, device=x32.device)
+    _ok(lib().acorn_hyper_norm(x32.data_ptr(), T * W if x32.shape[0] > 1 else 0, _ptr(x_out), T * W, _ptr(rows), _ptr(a),
+                               _ptr(experts.y) if experts is not None else None, _ptr(experts.slot_of) if experts is not None else None,
+                               _ptr(experts.wts) if experts is not None else None,
+                               experts.slot_of.shape[1] if experts is not None else 1,
+                               _ptr(experts.extra) if experts is not None else None, _ptr(mix), _ptr(put), float(scale),
+                               _ptr(take32), norm_w32.data_ptr(), float(eps), out.data_ptr(), count, W, n, dtype_code(dtype),
+                               _stream()), "hyper_norm")
+    return out
 
 
 def add_into(resid32: torch.Tensor, delta: torch.Tensor) -> None:
@@ -1899,9 +2143,10 @@ def linear_scan(b: torch.Tensor, c: torch.Tensor, x: torch.Tensor, decay: torch.
 
 
 def gated_norm(y32: torch.Tensor, gate: torch.Tensor, weight32: torch.Tensor, eps: float, groups: int, gate_first: bool,
-               out: torch.Tensor, out_scale: float = 1.0) -> torch.Tensor:
+               out: torch.Tensor, out_scale: float = 1.0, silu: bool = False) -> torch.Tensor:
     """RMS norm of ``y32`` [T, W] in ``groups`` equal parts times ``weight32``, with a gate ``z`` [T, W]:
-    ``gate_first``: ``norm(y silu(z))``; else ``norm(y) sigmoid(z)``.  Times ``out_scale``, rounded once into ``out``
+    ``gate_first``: ``norm(y silu(z))``; else ``norm(y) sigmoid(z)``, with
+    ``silu`` ``norm(y) silu(z)``.  Times ``out_scale``, rounded once into ``out``
     [T, W] (a column slice of a wider buffer is allowed, as for ``gate``)."""
     _check(y32, "y", torch.float32, 2)
     _rows2(gate, "gate")
@@ -1911,7 +2156,7 @@ def gated_norm(y32: torch.Tensor, gate: torch.Tensor, weight32: torch.Tensor, ep
     if gate.shape != (T, W) or out.shape != (T, W) or weight32.numel() != W or W % groups:
         raise KernelError(f"gated_norm: y {tuple(y32.shape)}, gate {tuple(gate.shape)}, out {tuple(out.shape)}, groups {groups}")
     _ok(lib().acorn_gated_norm(y32.data_ptr(), gate.data_ptr(), gate.stride(0), weight32.data_ptr(), out.data_ptr(),
-                               out.stride(0), T, W, groups, float(eps), 0 if gate_first else 1, float(out_scale),
+                               out.stride(0), T, W, groups, float(eps), 0 if gate_first else (2 if silu else 1), float(out_scale),
                                dtype_code(gate.dtype), _stream()), "gated_norm")
     return out
 
@@ -1959,10 +2204,17 @@ def min_gru(proj: torch.Tensor, bias32: torch.Tensor, state: torch.Tensor, state
 MOE_SCORINGS = {"softmax": 0, "sigmoid": 1}
 
 
+def _check_router_bias(bias32: torch.Tensor | None, n: int) -> None:
+    if bias32 is not None:
+        _check(bias32, "router bias", torch.float32, 1)
+        if bias32.numel() != n:
+            raise KernelError("moe_route: the bias must have one entry per router output")
+
+
 def moe_route(z32: torch.Tensor, correction32: torch.Tensor | None, top: int, groups: int, keep: int, normalize: bool = False,
-              scoring: str = "softmax"):
+              scoring: str = "softmax", bias32: torch.Tensor | None = None):
     """(chosen [T, top] int32, weights [T, top] float32) from router logits z [T, N] (columns of a wider product are
-    allowed).  ``scoring``: an output's score is its softmax, or the sigmoid of its logit.  Outputs are ranked by score +
+    allowed), ``bias32`` [N] added to them if given.  ``scoring``: an output's score is its softmax, or the sigmoid of its logit.  Outputs are ranked by score +
     correction; without a correction by the logits, in whose order the scores stand.  ``normalize``: the
     chosen outputs' scores are divided by their sum (+ 1e-20)."""
     _rows2(z32, "router logits", torch.float32)
@@ -1971,11 +2223,12 @@ def moe_route(z32: torch.Tensor, correction32: torch.Tensor | None, top: int, gr
         _check(correction32, "correction", torch.float32, 1)
         if correction32.numel() != N:
             raise KernelError("moe_route: correction must have one entry per router output")
+    _check_router_bias(bias32, N)
     if scoring not in MOE_SCORINGS:
         raise KernelError(f"moe_route: scoring must be one of {sorted(MOE_SCORINGS)}, got {scoring!r}")
     idx = torch.empty((T, top), dtype=torch.int32, device=z32.device)
     wts = torch.empty((T, top), dtype=torch.float32, device=z32.device)
-    _ok(lib().acorn_moe_route(z32.data_ptr(), z32.stride(0), _ptr(correction32), idx.data_ptr(), wts.data_ptr(), T, N, int(top),
+    _ok(lib().acorn_moe_route(z32.data_ptr(), z32.stride(0), _ptr(bias32), _ptr(correction32), idx.data_ptr(), wts.data_ptr(), T, N, int(top),
                               int(groups), int(keep), 1 if normalize else 0, MOE_SCORINGS[scoring], _stream()), "moe_route")
     return idx, wts
 
@@ -2001,12 +2254,12 @@ def moe_plan(idx: torch.Tensor, num_outputs: int, wts: torch.Tensor | None = Non
 
 
 def moe_route_plan(z32: torch.Tensor, correction32: torch.Tensor | None, top: int, groups: int, keep: int,
-                   normalize: bool = False, scoring: str = "softmax", by_slot: bool = False):
+                   normalize: bool = False, scoring: str = "softmax", by_slot: bool = False, bias32: torch.Tensor | None = None):
     """``moe_route`` followed by ``moe_plan``: (chosen, weights, offsets, slot_of, slot_token, weights by slot if ``by_slot``
     else None); one kernel for steps of few tokens."""
     T, N = z32.shape
     if not lib().acorn_moe_route_plan_supported(T, N):
-        idx, wts = moe_route(z32, correction32, top, groups, keep, normalize, scoring)
+        idx, wts = moe_route(z32, correction32, top, groups, keep, normalize, scoring, bias32)
         offsets, slot_of, slot_token, *rest = moe_plan(idx, N, wts if by_slot else None)
         return idx, wts, offsets, slot_of, slot_token, (rest[0] if by_slot else None)
     _rows2(z32, "router logits", torch.float32)
@@ -2014,11 +2267,12 @@ def moe_route_plan(z32: torch.Tensor, correction32: torch.Tensor | None, top: in
         _check(correction32, "correction", torch.float32, 1)
         if correction32.numel() != N:
             raise KernelError("moe_route: correction must have one entry per router output")
+    _check_router_bias(bias32, N)
     i32 = lambda *shape: torch.empty(shape, dtype=torch.int32, device=z32.device)
     f32 = lambda *shape: torch.empty(shape, dtype=torch.float32, device=z32.device)
     idx, wts, offsets, slot_of, slot_token = i32(T, top), f32(T, top), i32(N + 1), i32(T, top), i32(T * top)
     slot_wts = f32(T * top) if by_slot else None
-    _ok(lib().acorn_moe_route_plan(z32.data_ptr(), z32.stride(0), _ptr(correction32), idx.data_ptr(), wts.data_ptr(), T, N, int(top),
+    _ok(lib().acorn_moe_route_plan(z32.data_ptr(), z32.stride(0), _ptr(bias32), _ptr(correction32), idx.data_ptr(), wts.data_ptr(), T, N, int(top),
                                    int(groups), int(keep), 1 if normalize else 0, MOE_SCORINGS[scoring], offsets.data_ptr(),
                                    slot_of.data_ptr(), slot_token.data_ptr(), _ptr(slot_wts), _stream()), "moe_route_plan")
     return idx, wts, offsets, slot_of, slot_token, slot_wts

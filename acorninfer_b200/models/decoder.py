@@ -76,6 +76,13 @@ class Decoder:
                 raise ValueError("a stream mix does not go with schedule entries that take the token rows in again")
             self.stream_mix = build_part(STREAM_MIXES, spec.stream_mix, self.ctx)
             self._named_parts.append((spec.stream_mix.prefix, self.stream_mix))
+        if spec.streams is not None:
+            if spec.streams < 1 or self.stream_mix is not None or any(e.opens_pass is not None or e.add_embedding for e in spec.schedule):
+                raise ValueError("several residual streams do not go with a stream mix or schedule entries that take the token rows in again")
+            if not all(getattr(b, "takes_streams", False) for b in self.blocks) or not hasattr(self.final_norm, "eps"):
+                raise ValueError("several residual streams need layers in an arrangement that takes them, and an RMS norm at the end")
+        elif any(getattr(b, "takes_streams", False) for b in self.blocks):
+            raise ValueError("an arrangement with several residual streams needs ModelSpec.streams")
         for i, e in enumerate(spec.schedule):
             if e.opens_pass is not None and self.pass_entry is None:
                 raise ValueError(f"schedule entry {i} opens a pass, but the model names no pass_entry part")
@@ -185,6 +192,13 @@ class Decoder:
             return self._head(h, inputs) if h is not None else None
         delta = None
         sched = self.spec.schedule
+        if self.spec.streams is not None:
+            streams = ops.StreamBundle(resid32[None], self.spec.streams)       # all streams start as the token rows
+            for i, e in enumerate(sched):
+                streams, _ = self.blocks[e.layer].forward(streams, None, inputs, caches[i])
+            if inputs.num_logits == 0:
+                return None
+            return self._head(streams.read(None, self.final_norm.weight32, self.final_norm.eps, self.dtype, rows=inputs.logit_tokens), inputs)
         # a run that takes the tokens in again adds the stream as it was here
         def reenters(e):
             return e.add_embedding or e.opens_pass is not None

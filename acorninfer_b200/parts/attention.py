@@ -23,7 +23,12 @@ without weights (``qk_norm_weights`` false: the heads are only brought to unit r
 head, a term ``exp(sink_h)`` in the softmax denominator that has no key and no value (``sink``); a cap on the scaled
 scores, ``cap tanh(score / cap)`` (``softcap``); a query temperature, the finished query of position p times
 ``1 + coef ln(floor((p + 1) / every) + 1)`` (``q_temp`` = (coef, every)).  A position encoding's factor on cos and sin
-(``magnitude``) is applied.
+(``magnitude``) is applied.  With ``qk_norm_rows`` the q/k norm goes over the whole projected row of q (of k), all heads at
+once, with weights of that size.  ``unit_sink``: one is added to the softmax denominator (a sink fixed at zero).
+
+Under a bfloat16 engine heads whose key and value rows differ in width, or whose width is no multiple of 16, can be padded
+with zeros to one such width when the weights are bound (``pad_heads``): padded entries of q and k add nothing to a score,
+padded value entries are zero and meet zero columns of the output matrix; the tensor-core attention kernels then take them.
 
 All sizes are parameters.  The q, k, v (and gate) matrices are concatenated when bound so that one
 matrix product yields a token's whole row.  A run that reads another run's
@@ -44,6 +49,9 @@ _NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o":
           "q_conv": "q_conv.weight", "k_conv": "k_conv.weight", "v_conv": "v_conv.weight", "sink": "sink"}
 
 
+ATTENTION_TC_MAX_HEAD = 128       # head sizes the tensor-core attention kernels take for prompts and decoded tokens alike
+
+
 @MIXERS.register("attention")
 class Attention(Mixer):
     graph_safe = True
@@ -56,7 +64,8 @@ class Attention(Mixer):
                  value_dim: int | None = None, values_from_keys: bool = False, head_gate: bool = False,
                  names: dict | None = None, bias: bool = False, conv_taps: int | None = None,
                  slope_exponent: float | None = None, norm_after_rotation: bool = False, qk_norm_weights: bool = True,
-                 sink: bool = False, softcap: float | None = None, q_temp: tuple[float, int] | None = None):
+                 sink: bool = False, softcap: float | None = None, q_temp: tuple[float, int] | None = None,
+                 qk_norm_rows: bool = False, unit_sink: bool = False, pad_heads: bool = False):
         """``names``: the tensors' names relative to the part's prefix (keys q, k, v, o, q_norm, k_norm, gate,
         q_bias, k_bias, v_bias, q_conv, k_conv, v_conv, sink)."""
         if (norm_after_rotation or not qk_norm_weights) and (qk_norm_eps is None or conv_taps or bias):
@@ -70,6 +79,12 @@ class Attention(Mixer):
         self.q_temp = None if q_temp is None else (float(q_temp[0]), int(q_temp[1]))
         if conv_taps is not None and (conv_taps < 1 or values_from_keys):
             raise ValueError("conv_taps must be >= 1 or None, and needs value columns of their own")
+        if qk_norm_rows and (qk_norm_eps is None or values_from_keys or head_gate or q_temp is not None or slope_exponent is not None
+                             or norm_after_rotation or not qk_norm_weights):
+            raise ValueError("a q/k norm over whole rows needs qk_norm_eps and value columns of their own, and goes with windows, "
+                             "biases, convolutions, rotations, sinks and caps only")
+        if unit_sink and sink:
+            raise ValueError("a sink per head and a sink fixed at zero exclude one another")
         if num_heads % num_kv_heads:
             raise ValueError(f"num_heads ({num_heads}) must be a multiple of num_kv_heads ({num_kv_heads})")
         for what, n in (("window", window), ("chunk", chunk)):
@@ -91,6 +106,13 @@ class Attention(Mixer):
         self.position = ctx.positions[position] if position is not None else None
         if self.position is not None and self.position.head_dim != head_dim:
             raise ValueError("position encoding was built for another head size")
+        self.norm_rows, self.unit_sink = bool(qk_norm_rows), bool(unit_sink)
+        self.d_own, self.dv_own = self.d, self.dv                  # the sizes of the checkpoint's heads
+        if pad_heads and self.norm_rows and ctx.dtype == torch.bfloat16:
+            width = -(-max(self.d, self.dv) // 16) * 16
+            if width <= ATTENTION_TC_MAX_HEAD:
+                self.d = self.dv = width
+        head_dim = self.d
         # the plain arrangement [q | k | v] of equal head sizes, which the fused products take
         self.bias, self.taps = bool(bias), conv_taps
         self.slopes32 = None
@@ -103,28 +125,29 @@ class Attention(Mixer):
         self.sink32 = None
         magnitude = getattr(self.position, "magnitude", 1.0) if self.position is not None else 1.0
         self.plain = (not (values_from_keys or head_gate or bias or conv_taps or self.norm_after or self.sink or softcap
-                           or q_temp is not None)
+                           or q_temp is not None or self.norm_rows or self.unit_sink)
                       and self.norm_weights and magnitude == 1.0 and self.dv == head_dim)
         self.gate_col = (self.nq + self.nkv) * self.d + (0 if values_from_keys else self.nkv * self.dv)
         self.w_qkv = self.w_o = self.q_norm32 = self.k_norm32 = None
 
     def tensor_specs(self):
         n = self.names
+        d, dv = self.d_own, self.dv_own
         specs = {
-            n["q"]: TensorSpec((self.nq * self.d, self.hidden_size)),
-            n["k"]: TensorSpec((self.nkv * self.d, self.hidden_size)),
-            n["o"]: TensorSpec((self.hidden_size, self.nq * self.dv)),
+            n["q"]: TensorSpec((self.nq * d, self.hidden_size)),
+            n["k"]: TensorSpec((self.nkv * d, self.hidden_size)),
+            n["o"]: TensorSpec((self.hidden_size, self.nq * dv)),
         }
         if not self.values_from_keys:
-            specs[n["v"]] = TensorSpec((self.nkv * self.dv, self.hidden_size))
+            specs[n["v"]] = TensorSpec((self.nkv * dv, self.hidden_size))
         if self.head_gate:
             specs[n["gate"]] = TensorSpec((self.nq, self.hidden_size))
         if self.qk_norm_eps is not None and self.norm_weights:
-            specs[n["q_norm"]] = TensorSpec((self.d,), "norm")
-            specs[n["k_norm"]] = TensorSpec((self.d,), "norm")
+            specs[n["q_norm"]] = TensorSpec((self.nq * d if self.norm_rows else d,), "norm")
+            specs[n["k_norm"]] = TensorSpec((self.nkv * d if self.norm_rows else d,), "norm")
         if self.sink:
             specs[n["sink"]] = TensorSpec((self.nq,), "sink")
-        rows = {"q": self.nq * self.d, "k": self.nkv * self.d, **({} if self.values_from_keys else {"v": self.nkv * self.dv})}
+        rows = {"q": self.nq * d, "k": self.nkv * d, **({} if self.values_from_keys else {"v": self.nkv * dv})}
         for which, size in rows.items():
             if self.bias:
                 specs[n[which + "_bias"]] = TensorSpec((size,), "bias")
@@ -132,8 +155,27 @@ class Attention(Mixer):
                 specs[n[which + "_conv"]] = TensorSpec((size, self.taps), "conv")
         return specs
 
+    def _padded(self, tensors):
+        """The tensors with every head padded with zeros to the width the kernels see."""
+        if (self.d, self.dv) == (self.d_own, self.dv_own):
+            return tensors
+        n, out = self.names, dict(tensors)
+
+        def pad(t, heads, own, to):          # rows of `heads` heads
+            v = t.new_zeros((heads, to, *t.shape[1:]))
+            v[:, :own] = t.view(heads, own, *t.shape[1:])
+            return v.reshape(heads * to, *t.shape[1:])
+
+        for w, heads, own, to in (("q", self.nq, self.d_own, self.d), ("k", self.nkv, self.d_own, self.d), ("v", self.nkv, self.dv_own, self.dv)):
+            for name in (n[w], n[w + "_bias"], n[w + "_conv"], n.get(w + "_norm")):
+                if name in out:
+                    out[name] = pad(out[name], heads, own, to)
+        out[n["o"]] = pad(out[n["o"]].t().contiguous(), self.nq, self.dv_own, self.dv).t().contiguous()
+        return out
+
     def bind(self, tensors):
         n = self.names
+        tensors = self._padded(tensors)
         parts = [tensors[n["q"]], tensors[n["k"]]]
         if not self.values_from_keys:
             parts.append(tensors[n["v"]])
@@ -148,6 +190,13 @@ class Attention(Mixer):
         if self.qk_norm_eps is not None and self.norm_weights:
             self.q_norm32 = tensors[n["q_norm"]].to(torch.float32).contiguous()
             self.k_norm32 = tensors[n["k_norm"]].to(torch.float32).contiguous()
+        if self.norm_rows:                    # rows up to a multiple of 8, so that another mixer's may stand beside them
+            pad = (-self.w_qkv.shape[0]) % 8
+            if pad:
+                self.w_qkv = torch.cat([self.w_qkv, self.w_qkv.new_zeros((pad, self.w_qkv.shape[1]))], dim=0).contiguous()
+            self.w_in = self.w_qkv
+        if self.unit_sink:
+            self.sink32 = torch.zeros(self.nq, dtype=torch.float32, device=self.w_o.device)
         if self.sink:
             self.sink32 = tensors[n["sink"]].to(torch.float32).contiguous()
         which = ("q", "k") + (() if self.values_from_keys else ("v",))
@@ -170,16 +219,46 @@ class Attention(Mixer):
 
     def fusable(self, num_rows):
         # (the options only change what runs between the two products, which take the fused forms either way)
-        return (self._rows_fuse(num_rows) and self.w_qkv.dtype == torch.bfloat16
+        return (not self.norm_rows and self._rows_fuse(num_rows) and self.w_qkv.dtype == torch.bfloat16
                 and self.w_o.dtype == torch.bfloat16 and self.hidden_size % 8 == 0 and (self.nq * self.d) % 8 == 0)
 
     def _rows_fuse(self, num_rows):
         widths = ((self.nq + 2 * self.nkv) * self.d, self.hidden_size)         # of the q/k/v product and of the o product
         return ops.fused_rows_ok(num_rows, self.ctx.dtype, widths, ops.device_sms(self.ctx.device))
 
-    def inner(self, x, inputs, cache, out_scale: float = 1.0, out=None):
+    def _inner_norm_rows(self, x, inputs, cache, out_scale, out, proj):
+        g, pos = inputs.groups[cache.group], self.position
+        if not cache.write:
+            raise ValueError("attention: a q/k norm over whole rows needs a cache of the run's own")
+        if proj is None:
+            proj = ops.linear(x, self.w_qkv, out_dtype=self.ctx.dtype)
+        q = torch.empty((proj.shape[0], self.nq * self.d), dtype=self.ctx.dtype, device=proj.device)
+        conv = None
+        if self.taps:
+            conv = ops.ShortConv(self.conv32, cache.state if self.taps > 1 else proj.new_zeros((1, 0), dtype=torch.float32),
+                                 self.state_base, inputs.row_start, inputs.row_slot, update_single=True)
+        rotates = pos is not None and pos.rotary_dim > 0
+        # the factor on the result goes in with the values, which the heads' outputs are linear in
+        ops.qk_row_norm(proj, self.q_norm32, self.k_norm32, pos.table(inputs) if rotates else None, inputs.positions,
+                        inputs.token_row, g.block_table, g.page_base, cache.k_pages, cache.v_pages, self.nq, self.nkv, self.d,
+                        self.dv, pos.interleaved if rotates else False, self.qk_norm_eps, q, bias32=self.bias32, conv=conv,
+                        q_count=self.nq * self.d_own, k_count=self.nkv * self.d_own, v_scale=out_scale)
+        if self.taps and self.taps > 1 and inputs.plan.max_q_len > 1:     # rows of one token shifted their memory above
+            ops.conv_state_update(proj, cache.state, self.state_base, inputs.row_start, inputs.row_slot, inputs.num_rows,
+                                  self.channels, self.taps, bias32=self.bias32, skip_single=True)
+        heads = attn_kernels.paged_attention(q, inputs, g, cache, self.nq, self.nkv, self.d, self.scale, self.window,
+                                             chunk=self.chunk, keep_first=self.keep_first, value_dim=self.dv,
+                                             sink32=self.sink32, softcap=self.softcap)
+        return heads if out is None else ops.head_gate(heads, None, self.nq, 1.0, out=out)
+
+    state_base = 0
+    w_in = None            # the projection of x where its product may be made by the caller (``inner(proj=...)``)
+
+    def inner(self, x, inputs, cache, out_scale: float = 1.0, out=None, proj=None):
         """Everything before the output projection: the heads' outputs [T, nq * dv] (gated, times ``out_scale``),
-        into ``out`` if given (rows of a wider buffer)."""
+        into ``out`` if given (rows of a wider buffer).  ``proj``: the rows of ``w_in``'s product, if the caller made it."""
+        if self.norm_rows:
+            return self._inner_norm_rows(x, inputs, cache, out_scale, out, proj)
         g = inputs.groups[cache.group]
         pos = self.position
         rows = x.x.shape[0] if isinstance(x, ops.NormedRows) else x.shape[0]
@@ -203,7 +282,7 @@ class Attention(Mixer):
             conv = None
             if self.taps:
                 conv = ops.ShortConv(self.conv32, cache.state if self.taps > 1 else proj.new_zeros((1, 0), dtype=torch.float32),
-                                     0, inputs.row_start, inputs.row_slot, update_single=True)
+                                     self.state_base, inputs.row_start, inputs.row_slot, update_single=True)
             ops.qk_rope_kv(proj, self.q_norm32, self.k_norm32,
                            pos.inv_freq if pos is not None else _no_freq(self.ctx.device),
                            inputs.positions, inputs.token_row, g.block_table, g.page_base,
@@ -213,7 +292,7 @@ class Attention(Mixer):
                            value_dim=self.dv, bias32=self.bias32, conv=conv, q_out=qkv,
                            magnitude=getattr(pos, "magnitude", 1.0) if pos is not None else 1.0, q_temp=self.q_temp)
             if self.taps and self.taps > 1 and inputs.plan.max_q_len > 1:     # rows of one token shifted their memory above
-                ops.conv_state_update(proj, cache.state, 0, inputs.row_start, inputs.row_slot, inputs.num_rows,
+                ops.conv_state_update(proj, cache.state, self.state_base, inputs.row_start, inputs.row_slot, inputs.num_rows,
                                       self.channels, self.taps, bias32=self.bias32, skip_single=True)
         else:
             qkv = ops.linear(x, self.w_qkv, out_dtype=self.ctx.dtype)

@@ -107,6 +107,7 @@ class ModelSpec:
     embedding_scale: float = 1.0                  # factor on the token rows as they enter the stream (not on a tied head)
     pass_entry: PartSpec | None = None            # kind of the PASS_ENTRIES registry: runs before entries with ``opens_pass``
     stream_mix: PartSpec | None = None            # kind of the STREAM_MIXES registry: runs after every layer run
+    streams: int | None = None                    # number of residual streams (arrangements that take them); their sum ends the model
     ignorable: tuple[str, ...] = ()               # tensors a folder may hold although the model does not read them
     logit_scale: float = 1.0                      # factor on the logits
 

@@ -24,6 +24,12 @@ after every sublayer (norms ``mixer_in``, ``mixer_out``, ``feed_forward_in``, ``
 float32 in the kernel that norms a sublayer's output, which where it can also applies the norm the next
 sublayer reads the stream through.  A layer may have no feed-forward; an extra named ``side`` (a sublayer that
 adds to the stream itself, such as a token's side rows) runs last.
+
+``hyper``: several residual streams x_1 .. x_n (``ModelSpec.streams``).  Sublayer q (1: mixer, 2: feed-forward) reads
+``norm(sum_s in_q[s] x_s)``; its result y goes back as ``x_t <- sum_s mix_q[s, t] x_s + m out_q[t] y``, all streams at once
+from the old ones (tensors ``hc<q>.in``, ``hc<q>.mix``, ``hc<q>.out``; m is ``residual_scale``).  The streams are float32; the new
+streams, what the next sublayer reads of them and its norm are one kernel (``ops.StreamBundle``), which also takes the sum
+over a routed feed-forward's experts.  A layer may have no feed-forward.
 """
 
 from __future__ import annotations
@@ -31,7 +37,7 @@ from __future__ import annotations
 import torch
 
 from ..kernels import ops
-from .base import BLOCKS, Block
+from .base import BLOCKS, Block, TensorSpec
 from .norms import take_stream_norms
 
 
@@ -217,3 +223,56 @@ class SandwichBlock(Block):
         if self.side is not None:
             return resid32, self.side.forward(resid32, rounded if rounded is not None else resid32, inputs, defer=True)
         return resid32, None
+
+
+@BLOCKS.register("hyper")
+class HyperBlock(Block):
+    graph_safe = True
+    takes_streams = True           # ``resid32`` is an ``ops.StreamBundle``
+
+    def __init__(self, ctx, mixer, feed_forward, norms, streams: int, residual_scale: float = 1.0, learned: bool = True):
+        """``learned`` false: one stream, read and added to as it is (``x += m mixer(norm(x))``), without tensors."""
+        super().__init__(mixer, feed_forward, norms)
+        self.ctx, self.n, self.scale, self.learned = ctx, int(streams), float(residual_scale), bool(learned)
+        if not learned and self.n != 1:
+            raise ValueError("a hyper block without tensors has one stream")
+        self.sublayers = ("mixer",) + (("feed_forward",) if feed_forward is not None else ())
+        missing = set(self.sublayers) - {k for k, v in norms.items() if hasattr(v, "tensor_specs")}
+        if missing:
+            raise ValueError(f"hyper block needs norms named {list(self.sublayers)}; missing {sorted(missing)}")
+        self.take32, self.mix32, self.put32 = {}, {}, {}
+
+    def tensor_specs(self):
+        n = self.n
+        specs = {}
+        if not self.learned:
+            return specs
+        for q, _ in enumerate(self.sublayers, 1):
+            specs.update({f"hc{q}.in": TensorSpec((n,), "stream_in"), f"hc{q}.out": TensorSpec((n,), "stream_out"),
+                          f"hc{q}.mix": TensorSpec((n, n), "stream_mix")})
+        return specs
+
+    def bind(self, tensors):
+        if not self.learned:
+            one = torch.ones(1, dtype=torch.float32, device=self.ctx.device)
+            for which in self.sublayers:
+                self.take32[which], self.put32[which], self.mix32[which] = one, one, one.view(1, 1)
+            return
+        f32 = lambda name: tensors[name].to(torch.float32).contiguous()
+        for q, which in enumerate(self.sublayers, 1):
+            self.take32[which], self.put32[which], self.mix32[which] = f32(f"hc{q}.in"), f32(f"hc{q}.out"), f32(f"hc{q}.mix")
+
+    def _read(self, streams, which):
+        norm = self.norms[which]
+        return streams.read(self.take32[which], norm.weight32, norm.eps, self.ctx.dtype)
+
+    def forward(self, resid32, delta, inputs, cache, next_norm=None):
+        streams = resid32
+        y = self.mixer.forward(self._read(streams, "mixer"), inputs, cache)
+        streams.pending = (y, self.mix32["mixer"], self.put32["mixer"], self.scale)
+        if self.feed_forward is not None:
+            h = self._read(streams, "feed_forward")
+            more = {"defer": True} if getattr(self.feed_forward, "defers_weighted", False) else {}
+            y = self.feed_forward.forward(h, inputs, **more)
+            streams.pending = (y, self.mix32["feed_forward"], self.put32["feed_forward"], self.scale)
+        return streams, None

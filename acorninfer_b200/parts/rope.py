@@ -17,7 +17,8 @@ from .base import POSITION_ENCODINGS, BuildContext, PositionEncoding
 @POSITION_ENCODINGS.register("rope")
 class Rope(PositionEncoding):
     def __init__(self, ctx: BuildContext, head_dim: int, theta: float, rotary_dim: int | None = None,
-                 pairing: str = "half"):
+                 pairing: str = "half", exact: bool = False):
+        """``exact``: the frequencies are evaluated in float64 and rounded once."""
         rotary_dim = head_dim if rotary_dim is None else rotary_dim
         if pairing not in ("half", "interleaved"):
             raise ValueError(f"rope pairing must be 'half' or 'interleaved', got {pairing!r}")
@@ -30,6 +31,10 @@ class Rope(PositionEncoding):
         self.interleaved = pairing == "interleaved"
         self.magnitude = 1.0                  # factor on cos and sin
         self._inv_freq_cpu = 1.0 / (self.theta ** (torch.arange(0, rotary_dim, 2, dtype=torch.float32) / rotary_dim))
+        if exact:
+            self._inv_freq_cpu = torch.tensor([self.theta ** (-2.0 * i / rotary_dim) for i in range(rotary_dim // 2)],
+                                              dtype=torch.float64).to(torch.float32)
+        self.exact = bool(exact)
         self._inv_freq_dev: torch.Tensor | None = None
 
     @property
@@ -42,7 +47,7 @@ class Rope(PositionEncoding):
         """cos and sin of every token's angles, [tokens, rotary_dim] float32 (cos, then sin): computed by
         the first layer of a step that asks and kept with the step's inputs for the others."""
         from ..kernels import ops
-        key = ("rope.table", self.theta, self.rotary_dim)
+        key = ("rope.table", self.theta, self.rotary_dim, self.exact)
         if key not in inputs.extra:
             inputs.extra[key] = ops.rope_table(inputs.positions, self.inv_freq)
         return inputs.extra[key]

@@ -15,7 +15,7 @@ the same form (``shared_size``, ``shared_limit``; tensors ``shared.gate`` / ``up
 takes, added to the weighted sum; scores ``sigmoid(z)`` of each output instead of the softmax (``scoring="sigmoid"``);
 the chosen outputs' weights on the experts' *inputs* instead of their outputs (``weight_on="input"``: the sum over the
 chosen of ``expert(s h)``); the shared expert's result times ``sigmoid(W_sg h)``, one number per token (``shared_gate``;
-tensor ``shared.sg``).
+tensor ``shared.sg``); a bias per output on the router's logits (``router_bias``; tensor ``router.b``).
 
 On the device: the router's choice and the (token, choice) pairs grouped by expert (a kernel each, one for both in
 steps of few tokens), one product per expert over its own rows for gate/up (SwiGLU in its epilogue on the tensor-core
@@ -44,7 +44,7 @@ class RoutedExperts(FeedForward):
                  top: int, groups: int = 1, keep: int = 1, correction: bool = True, normalize: bool = False,
                  activation: str = "silu", limit: float = 0.0, shared_size: int | None = None,
                  shared_limit: float | None = None, scoring: str = "softmax", weight_on: str = "output",
-                 shared_gate: bool = False):
+                 shared_gate: bool = False, router_bias: bool = False):
         if scoring not in ops.MOE_SCORINGS:
             raise ValueError(f"scoring must be one of {sorted(ops.MOE_SCORINGS)}, got {scoring!r}")
         if weight_on not in ("output", "input") or (weight_on == "input" and (num_identity or num_experts < 1)):
@@ -52,15 +52,16 @@ class RoutedExperts(FeedForward):
         if shared_gate and not shared_size:
             raise ValueError("shared_gate needs a shared expert")
         self.scoring, self.weight_on, self.shared_gate = scoring, weight_on, bool(shared_gate)
+        self.router_bias, self.bias32 = bool(router_bias), None
         self.defers = weight_on == "input"      # ``forward(..., defer=True)`` leaves the sum over the choices undone
+        self.defers_weighted = weight_on == "output" and not num_identity and num_experts > 0 and not shared_gate   # ... with its weights
         if activation not in ("silu", "capped_swish"):
             raise ValueError(f"expert activation must be 'silu' or 'capped_swish', got {activation!r}")
         self.correction, self.normalize, self.activation, self.limit = bool(correction), bool(normalize), activation, float(limit)
         self.shared_size, self.shared_limit = shared_size, float(shared_limit if shared_limit is not None else limit)
-        self.w_shared_gu = self.w_shared_down = None
-        # a shared expert of the uncapped form is a gated feed-forward like any other
-        self.shared_ff = SwiGLU(ctx, hidden_size, shared_size, "silu", {"gate": "gate", "up": "up", "down": "down"}) \
-            if shared_size and activation == "silu" else None
+        # a shared expert is a gated feed-forward like any other
+        self.shared_ff = SwiGLU(ctx, hidden_size, shared_size, activation, {"gate": "gate", "up": "up", "down": "down"},
+                                limit=self.shared_limit) if shared_size else None
         n = num_experts + num_identity
         if n < 1 or n % groups or not (1 <= keep <= groups) or top > keep * (n // groups):
             raise ValueError(f"{n} router outputs do not split into {groups} groups of which {keep} hold {top} choices")
@@ -74,6 +75,8 @@ class RoutedExperts(FeedForward):
         specs = {"router": TensorSpec((n, self.hidden_size))}
         if self.correction:
             specs["correction"] = TensorSpec((n,), "bias")
+        if self.router_bias:
+            specs["router.b"] = TensorSpec((n,), "bias")
         if self.shared_gate:
             specs["shared.sg"] = TensorSpec((1, self.hidden_size))
         if self.shared_size:
@@ -97,14 +100,9 @@ class RoutedExperts(FeedForward):
             dtype = sg.dtype if sg.dtype == self.w_router.dtype else torch.float32
             self.w_router = torch.cat([self.w_router.to(dtype), sg.to(dtype)], dim=0).contiguous()
         self.correction32 = t["correction"].to(torch.float32).contiguous() if self.correction else None
-        if self.shared_size:
-            g, u = t["shared.gate"], t["shared.up"]
-            dtype = g.dtype if g.dtype == u.dtype else torch.float32
-            if self.shared_ff is not None:
-                self.shared_ff.bind({n: t["shared." + n] for n in ("gate", "up", "down")})
-            else:
-                self.w_shared_gu = torch.cat([g.to(dtype), u.to(dtype)], dim=0).contiguous()       # [gate | up]
-                self.w_shared_down = t["shared.down"].contiguous()
+        self.bias32 = t["router.b"].to(torch.float32).contiguous() if self.router_bias else None
+        if self.shared_ff is not None:
+            self.shared_ff.bind({n: t["shared." + n] for n in ("gate", "up", "down")})
         if self.E:
             mats = [t[f"e{e}.{n}"] for e in range(self.E) for n in ("gate", "up", "down")]
             dtype = mats[0].dtype if all(m.dtype == mats[0].dtype for m in mats) else torch.float32
@@ -122,7 +120,7 @@ class RoutedExperts(FeedForward):
         z = ops.linear(x, self.w_router, out_dtype=torch.float32)
         idx, wts, offsets, slot_of, slot_token, slot_wts = ops.moe_route_plan(
             z[:, :n], self.correction32, self.top, self.groups, self.keep, self.normalize, self.scoring,
-            by_slot=self.weight_on == "input")
+            by_slot=self.weight_on == "input", bias32=self.bias32)
         if self.weight_on == "input":
             wts = None                       # the weights go in with the rows: the choices are summed as they are
         slots = T * self.top
@@ -134,16 +132,10 @@ class RoutedExperts(FeedForward):
             y = ops.grouped_gemm(hidden, None, w_dn, offsets, slots)
         else:
             y = x
-        shared = None
-        if self.shared_ff is not None:
-            shared = beside.join()
-        elif self.shared_size:
-            gu = ops.linear(x, self.w_shared_gu, out_dtype=self.ctx.dtype)
-            shared = ops.linear(ops.swiglu(gu, activation=self.activation, limit=self.shared_limit), self.w_shared_down,
-                                out_dtype=self.ctx.dtype)
+        shared = beside.join() if beside is not None else None
         shared_z = z[:, n:n + 1] if self.shared_gate else None
-        if defer and self.defers:
-            return ops.ExpertsPending(y, slot_of, shared, shared_z)
+        if defer and (self.defers or self.defers_weighted):
+            return ops.ExpertsPending(y, slot_of, shared, shared_z, wts)
         if add_normed is not None:
             resid32, norm = add_normed
             return ops.moe_combine(y, x, slot_of, idx, wts, self.E, resid32=resid32, weight32=norm.weight32, eps=norm.eps,

@@ -179,6 +179,20 @@ def _depth_average(d: Draw) -> torch.Tensor:
 
 
 INIT_KINDS.register("depth_average", _depth_average)
+INIT_KINDS.register("stream_in", lambda d: d.normal(0.3, 1.0 / d.shape[0]))    # what a sublayer reads of each residual stream
+INIT_KINDS.register("stream_out", lambda d: d.normal(0.3, 1.0))                  # what it writes to each
+
+
+def _stream_mix(d: Draw) -> torch.Tensor:
+    """A matrix between residual streams around the identity."""
+    t = d.normal(0.15)
+    first = d.rows[0] if d.rows is not None else 0
+    for i in range(t.shape[0]):
+        t[i, first + i] += 0.8
+    return t
+
+
+INIT_KINDS.register("stream_mix", _stream_mix)
 INIT_KINDS.register("blend", lambda d: d.normal(0.2, 0.5))             # shares of the row before in a blend of two rows
 
 
