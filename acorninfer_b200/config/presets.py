@@ -159,6 +159,33 @@ PRESETS.update({
 })
 
 
+def _badepel(width: int, vocab: int, heads: int, kv_heads: int, ff: int, window: int, experts: int, top: int, streams: int) -> dict:
+    """Layers in the pattern delta rule with a dense feed-forward, attention beside linear attention with routed experts, the
+    same again, delta rule with routed experts, twice; heads of 128 (key channels of the linear attention 64); the
+    routed layers' active width (the chosen experts and the shared one) is ``ff``."""
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": ff // (2 * top), "limit": 7.0}, "router": {"experts": experts, "top": top},
+           "shared": {"ff": ff // 2, "limit": 7.0}}
+    delta = {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}
+    both = {"left": {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0, "conv": 4,
+                     "mask": {"size": window}, "rot": {"base": 5e5, "dims": 64}},
+            "right": {"heads": heads, "dim": 64, "vdim": 128, "tau": 16.0, "decay_rank": 16}, "left_scale": 0.8, "right_scale": 1.1}
+    layers = []
+    for _ in range(2):
+        layers.append({"type": "delta", "mixer": dict(delta), "mlp": dense})
+        layers.append({"type": "parallel", "mixer": dict(both), "mlp": moe})
+        layers.append({"type": "parallel", "mixer": dict(both), "mlp": moe})
+        layers.append({"type": "delta", "mixer": dict(delta), "mlp": moe})
+    return {"architecture": "Badepel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "streams": streams,
+            "residual_mult": 0.6, "layers": layers}
+
+
+PRESETS.update({
+    "badepel-w1024": _badepel(1024, 32768, heads=8, kv_heads=2, ff=3072, window=1024, experts=16, top=2, streams=4),
+    "badepel-w2048": _badepel(2048, 65536, heads=16, kv_heads=4, ff=6144, window=1024, experts=16, top=2, streams=4),
+})
+
+
 def preset(name: str) -> dict:
     try:
         import copy

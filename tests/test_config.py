@@ -102,6 +102,8 @@ def test_presets_of_the_family_are_valid_configurations():
             assert len(spec_for(cfg).schedule) == 8          # layers 1 and 2 twice among six
         elif name.startswith("zusolix"):
             assert [l.type for l in cfg.layers[:4]] == ["attention", "attention", "mingru", "attention"]
+        elif name.startswith("badepel"):
+            assert [l.type for l in cfg.layers[:4]] == ["delta", "parallel", "parallel", "delta"] and cfg.streams == 4
         else:
             assert name.startswith("tedenex") and [l.type for l in cfg.layers[:3]] == ["wkv", "attention", "latent_attention"]
             assert len(spec_for(cfg).schedule) == 9          # the first three layers twice, then the other three
