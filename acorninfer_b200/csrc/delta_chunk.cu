@@ -1,0 +1,436 @@
+// The gated delta rule with one decay per head, over chunks of 64 tokens (float32 throughout):
+//     S_i = g_i S_(i-1) + k_i u_i^T,   u_i = beta_i (v_i - g_i S_(i-1)^T k_i),   o_i = S_i^T q_i.
+// Within a chunk that starts from S_0, with b_i the sum of the log decays up to i and G_ij = exp(b_i - b_j) (at most one for
+// j <= i), the u_i solve a unit lower triangular system, so what hangs on S_0 can be split off:
+//     (1 + A) U = diag(beta) V - diag(beta exp(b)) K S_0,   A_ij = beta_i G_ij (k_i . k_j) for j < i
+//     U = Ubar - W S_0,   O = diag(exp(b)) Q S_0 + P U,   P_ij = G_ij (q_i . k_j) for j <= i
+//     S_end = exp(b_n) S_0 + sum_j G_nj k_j u_j^T
+// (the form known from Yang, Kautz, Hatamizadeh, "Gated Delta Networks: Improving Mamba2 with Delta Rule").  Three kernels:
+//   delta_chunk_solve   all chunks side by side: b, A, P, and W and Ubar by forward substitution, a column a thread
+//   delta_chunk_state   a row's chunks one after the other, heads and tiles of 16 value columns side by side: U and the state
+//                       every chunk starts from; the row's end state into its slot
+//   delta_chunk_out     all chunks side by side: O
+// A row's chunks are counted from its first token of the step; chunk c of row r is number row_start[r] / 64 + r + c of the
+// step (distinct for all chunks; some numbers stay unused).
+#include "common.cuh"
+
+#define DC 64                       // tokens a chunk
+#define DC_VT 16                    // value columns a block of delta_chunk_state
+#define DC_OT 64                    // value columns a block of delta_chunk_out
+#define DC_PAD 4                    // floats between rows in shared memory (16-byte reads of neighbouring rows hit distinct banks)
+
+struct DeltaChunkParams {
+    const float* q;                 // [T, KH, dim]
+    const float* k;
+    const float* v;                 // [T, H, vdim]
+    const float* beta;              // [T, H]
+    const float* log_g;             // [T, H]
+    float* state;                   // slots: [H, dim, vdim]
+    int64_t slot_stride;
+    const int* row_start;
+    const int* row_slot;
+    float* w;                       // scratch: [T, H, dim]
+    float* u;                       // [T, H, vdim]: Ubar, then U
+    float* p;                       // [T, H, DC]
+    float* b;                       // [T, H]
+    float* s0;                      // [chunk numbers, H, dim, vdim]
+    float* out;                     // [T, H, vdim]
+    int rows, H, KH, dim, vdim;
+};
+
+// The row and chunk of a chunk number, or false for an unused one.
+__device__ __forceinline__ bool chunk_of(int id, const int* __restrict__ row_start, int rows, int& r, int& first, int& n) {
+    int lo = 0, hi = rows - 1;
+    while (lo < hi) {
+        const int mid = (lo + hi + 1) >> 1;
+        if (row_start[mid] / DC + mid <= id) lo = mid;
+        else hi = mid - 1;
+    }
+    r = lo;
+    const int start = row_start[lo], c = id - (start / DC + lo);
+    first = start + c * DC;
+    n = min(DC, row_start[lo + 1] - first);
+    return n > 0;
+}
+
+__device__ __forceinline__ void dc_cp16(float* dst, const float* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src));
+}
+
+// n rows of `width` floats (a multiple of 4), ld apart, into DC rows of DP + DC_PAD; the rest zeros
+template <int DP> __device__ __forceinline__ void load_rows(float* dst, const float* src, int64_t ld, int n, int width) {
+    for (int e = threadIdx.x; e < DC * (DP / 4); e += blockDim.x) {
+        const int i = e / (DP / 4), c = (e % (DP / 4)) * 4;
+        float* d = dst + i * (DP + DC_PAD) + c;
+        if (i < n && c < width) dc_cp16(d, src + (int64_t)i * ld + c);
+        else *reinterpret_cast<float4*>(d) = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+}
+
+__device__ __forceinline__ float dot4(const float4& a, const float4& b, float acc) {
+    return fmaf(a.w, b.w, fmaf(a.z, b.z, fmaf(a.y, b.y, fmaf(a.x, b.x, acc))));
+}
+
+template <int DP>
+__global__ void __launch_bounds__(256, 2) delta_chunk_solve_kernel(const DeltaChunkParams p) {
+    constexpr int LD = DP + DC_PAD, LA = DC + DC_PAD;
+    extern __shared__ __align__(16) float sm[];
+    float* sK = sm;                                     // [DC][LD]
+    float* sQ = sK + DC * LD;                           // [DC][LD]
+    float* sA = sQ + DC * LD;                           // [DC][LA]
+    __shared__ float sb[DC], sbeta[DC];
+    pdl_wait();
+    pdl_trigger();
+    const int h = blockIdx.y, kh = h / (p.H / p.KH), tid = threadIdx.x;
+    int r, first, n;
+    if (!chunk_of(blockIdx.x, p.row_start, p.rows, r, first, n)) return;
+    load_rows<DP>(sK, p.k + ((int64_t)first * p.KH + kh) * p.dim, (int64_t)p.KH * p.dim, n, p.dim);
+    load_rows<DP>(sQ, p.q + ((int64_t)first * p.KH + kh) * p.dim, (int64_t)p.KH * p.dim, n, p.dim);
+    asm volatile("cp.async.commit_group;\n" ::);
+    if (tid < 32) {                                     // sums of the log decays: two tokens a lane
+        const int i = 2 * tid;
+        const float a = i < n ? p.log_g[(int64_t)(first + i) * p.H + h] : 0.f;
+        const float c = i + 1 < n ? p.log_g[(int64_t)(first + i + 1) * p.H + h] : 0.f;
+        float run = a + c;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float before = __shfl_up_sync(0xffffffffu, run, o);
+            if (tid >= o) run += before;
+        }
+        sb[i] = run - c;
+        sb[i + 1] = run;
+        if (i < n) p.b[(int64_t)(first + i) * p.H + h] = run - c;
+        if (i + 1 < n) p.b[(int64_t)(first + i + 1) * p.H + h] = run;
+    } else if (tid < 32 + DC) {
+        const int i = tid - 32;
+        sbeta[i] = i < n ? p.beta[(int64_t)(first + i) * p.H + h] : 0.f;
+    }
+    asm volatile("cp.async.wait_group 0;\n" ::);
+    __syncthreads();
+    // k . k and q . k of rows ty + 16 ii and columns tx + 16 jj, the blocks on and below the diagonal
+    const int tx = tid & 15, ty = tid >> 4;
+    float kk[4][4], qk[4][4];
+#pragma unroll
+    for (int ii = 0; ii < 4; ++ii)
+#pragma unroll
+        for (int jj = 0; jj < 4; ++jj) kk[ii][jj] = qk[ii][jj] = 0.f;
+#pragma unroll 2
+    for (int d = 0; d < DP; d += 4) {
+        float4 kj[4];
+#pragma unroll
+        for (int jj = 0; jj < 4; ++jj) kj[jj] = *reinterpret_cast<const float4*>(sK + (tx + 16 * jj) * LD + d);
+#pragma unroll
+        for (int ii = 0; ii < 4; ++ii) {
+            const float4 ki = *reinterpret_cast<const float4*>(sK + (ty + 16 * ii) * LD + d);
+            const float4 qi = *reinterpret_cast<const float4*>(sQ + (ty + 16 * ii) * LD + d);
+#pragma unroll
+            for (int jj = 0; jj <= ii; ++jj) {
+                kk[ii][jj] = dot4(ki, kj[jj], kk[ii][jj]);
+                qk[ii][jj] = dot4(qi, kj[jj], qk[ii][jj]);
+            }
+        }
+    }
+#pragma unroll
+    for (int ii = 0; ii < 4; ++ii) {
+        const int i = ty + 16 * ii;
+#pragma unroll
+        for (int jj = 0; jj <= ii; ++jj) {
+            const int j = tx + 16 * jj;
+            const float G = j <= i ? expf(sb[i] - sb[j]) : 0.f;
+            sA[i * LA + j] = j < i ? sbeta[i] * G * kk[ii][jj] : 0.f;
+            if (i < n) p.p[((int64_t)(first + i) * p.H + h) * DC + j] = G * qk[ii][jj];
+        }
+    }
+    __syncthreads();
+    // forward substitution: a thread a column of [W | Ubar], its 64 entries in registers
+    for (int c0 = 0; c0 < p.dim + p.vdim; c0 += 256) {
+        const int col = c0 + tid;
+        if (col >= p.dim + p.vdim) break;
+        const bool is_w = col < p.dim;
+        float x[DC];
+        if (is_w) {
+#pragma unroll
+            for (int i = 0; i < DC; ++i) x[i] = sbeta[i] * expf(sb[i]) * sK[i * LD + col];
+        } else {
+            const float* v = p.v + ((int64_t)first * p.H + h) * p.vdim + col - p.dim;
+#pragma unroll
+            for (int i = 0; i < DC; ++i) x[i] = i < n ? v[(int64_t)i * p.H * p.vdim] : 0.f;
+#pragma unroll
+            for (int i = 0; i < DC; ++i) x[i] *= sbeta[i];
+        }
+#pragma unroll
+        for (int i = 1; i < DC; ++i) {
+            float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+            for (int j = 0; j < i; j += 4) {            // entries from j = i on are zeros in A
+                const float4 a = *reinterpret_cast<const float4*>(sA + i * LA + j);
+                s0 = fmaf(a.x, x[j], s0);
+                if (j + 1 < i) s1 = fmaf(a.y, x[j + 1], s1);
+                if (j + 2 < i) s0 = fmaf(a.z, x[j + 2], s0);
+                if (j + 3 < i) s1 = fmaf(a.w, x[j + 3], s1);
+            }
+            x[i] -= s0 + s1;
+        }
+        float* dst = is_w ? p.w + ((int64_t)first * p.H + h) * p.dim + col : p.u + ((int64_t)first * p.H + h) * p.vdim + col - p.dim;
+        const int64_t ld = (int64_t)p.H * (is_w ? p.dim : p.vdim);
+#pragma unroll
+        for (int i = 0; i < DC; ++i)
+            if (i < n) dst[i * ld] = x[i];
+    }
+}
+
+template <int DP>
+__global__ void __launch_bounds__(256) delta_chunk_state_kernel(const DeltaChunkParams p) {
+    constexpr int LD = DP + DC_PAD, HALF = DP / 2;
+    extern __shared__ __align__(16) float sm[];
+    float* sW = sm;                                     // [2][DC][LD]
+    float* sK = sW + 2 * DC * LD;                       // [2][DC][LD]
+    float* sS = sK + 2 * DC * LD;                       // [DC_VT][LD]: the state's columns
+    float2* sU = reinterpret_cast<float2*>(sS + DC_VT * LD);      // [DC][8]: columns c and c + 8 of a token's u, times G_nj
+    float* part = reinterpret_cast<float*>(sU + DC * 8);          // [8][128] the upper half's sums
+    pdl_wait();
+    pdl_trigger();
+    const int h = blockIdx.y, r = blockIdx.z, kh = h / (p.H / p.KH), v0 = blockIdx.x * DC_VT, tid = threadIdx.x;
+    const int start = p.row_start[r], L = p.row_start[r + 1] - start;
+    const int chunks = (L + DC - 1) / DC, id0 = start / DC + r;
+    const int cp = tid & 7;                             // this thread's columns: cp and cp + 8 of the tile
+    const int col0 = v0 + cp, col1 = v0 + cp + 8;
+    const bool on0 = col0 < p.vdim, on1 = col1 < p.vdim;
+    const int dg = tid >> 3;                            // its state entries: key channels 4 dg .. 4 dg + 3
+    const bool holds = 4 * dg < DP;
+    float* slot = p.state + (int64_t)p.row_slot[r] * p.slot_stride + (int64_t)h * p.dim * p.vdim;
+    float S0[4], S1[4];
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+        const int d = 4 * dg + q;
+        S0[q] = holds && d < p.dim && on0 ? slot[(int64_t)d * p.vdim + col0] : 0.f;
+        S1[q] = holds && d < p.dim && on1 ? slot[(int64_t)d * p.vdim + col1] : 0.f;
+    }
+    auto publish = [&]() {
+        if (holds) {
+            *reinterpret_cast<float4*>(sS + cp * LD + 4 * dg) = make_float4(S0[0], S0[1], S0[2], S0[3]);
+            *reinterpret_cast<float4*>(sS + (cp + 8) * LD + 4 * dg) = make_float4(S1[0], S1[1], S1[2], S1[3]);
+        }
+    };
+    publish();
+    auto fetch = [&](int c) {
+        const int first = start + c * DC, n = min(DC, L - c * DC);
+        load_rows<DP>(sW + (c & 1) * DC * LD, p.w + ((int64_t)first * p.H + h) * p.dim, (int64_t)p.H * p.dim, n, p.dim);
+        load_rows<DP>(sK + (c & 1) * DC * LD, p.k + ((int64_t)first * p.KH + kh) * p.dim, (int64_t)p.KH * p.dim, n, p.dim);
+    };
+    if (chunks > 0) fetch(0);
+    asm volatile("cp.async.commit_group;\n" ::);
+    const int half = tid >> 7, ig = (tid & 127) >> 3;   // rows ig + 16 rr over key channels half * HALF ..
+    for (int c = 0; c < chunks; ++c) {
+        const int first = start + c * DC, n = min(DC, L - c * DC);
+        float ub0[4], ub1[4], bj[4];
+        const float bn = p.b[(int64_t)(first + n - 1) * p.H + h];
+        if (half == 0) {
+#pragma unroll
+            for (int rr = 0; rr < 4; ++rr) {
+                const int i = ig + 16 * rr;
+                const int64_t t = (int64_t)(first + min(i, n - 1)) * p.H + h;
+                ub0[rr] = i < n && on0 ? p.u[t * p.vdim + col0] : 0.f;
+                ub1[rr] = i < n && on1 ? p.u[t * p.vdim + col1] : 0.f;
+                bj[rr] = p.b[t];
+            }
+        }
+        if (c + 1 < chunks) fetch(c + 1);
+        asm volatile("cp.async.commit_group;\n" ::);
+        float* keep = p.s0 + ((int64_t)(id0 + c) * p.H + h) * p.dim * p.vdim;      // the state this chunk starts from
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+            const int d = 4 * dg + q;
+            if (holds && d < p.dim) {
+                if (on0) keep[(int64_t)d * p.vdim + col0] = S0[q];
+                if (on1) keep[(int64_t)d * p.vdim + col1] = S1[q];
+            }
+        }
+        asm volatile("cp.async.wait_group 1;\n" ::);
+        __syncthreads();                                // this chunk's rows and the state's columns are there
+        const float* W = sW + (c & 1) * DC * LD;
+        const float* K = sK + (c & 1) * DC * LD;
+        float a0[4] = {0.f, 0.f, 0.f, 0.f}, a1[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+        for (int d = half * HALF; d < half * HALF + HALF; d += 4) {
+            const float4 s0 = *reinterpret_cast<const float4*>(sS + cp * LD + d);
+            const float4 s1 = *reinterpret_cast<const float4*>(sS + (cp + 8) * LD + d);
+#pragma unroll
+            for (int rr = 0; rr < 4; ++rr) {
+                const float4 w = *reinterpret_cast<const float4*>(W + (ig + 16 * rr) * LD + d);
+                a0[rr] = dot4(w, s0, a0[rr]);
+                a1[rr] = dot4(w, s1, a1[rr]);
+            }
+        }
+        if (half == 1) {
+#pragma unroll
+            for (int rr = 0; rr < 4; ++rr) {
+                part[rr * 128 + (tid & 127)] = a0[rr];
+                part[(4 + rr) * 128 + (tid & 127)] = a1[rr];
+            }
+        }
+        __syncthreads();
+        if (half == 0) {
+#pragma unroll
+            for (int rr = 0; rr < 4; ++rr) {
+                const int i = ig + 16 * rr;
+                const float u0 = ub0[rr] - (a0[rr] + part[rr * 128 + tid]), u1 = ub1[rr] - (a1[rr] + part[(4 + rr) * 128 + tid]);
+                const float G = i < n ? expf(bn - bj[rr]) : 0.f;
+                sU[i * 8 + cp] = make_float2(u0 * G, u1 * G);
+                if (i < n) {
+                    const int64_t t = ((int64_t)(first + i) * p.H + h) * p.vdim;
+                    if (on0) p.u[t + col0] = u0;
+                    if (on1) p.u[t + col1] = u1;
+                }
+            }
+        }
+        __syncthreads();
+        if (holds) {
+            const float gn = expf(bn);
+#pragma unroll
+            for (int q = 0; q < 4; ++q) {
+                S0[q] *= gn;
+                S1[q] *= gn;
+            }
+#pragma unroll 8
+            for (int j = 0; j < DC; ++j) {
+                const float4 k = *reinterpret_cast<const float4*>(K + j * LD + 4 * dg);
+                const float2 u = sU[j * 8 + cp];
+                S0[0] = fmaf(k.x, u.x, S0[0]); S1[0] = fmaf(k.x, u.y, S1[0]);
+                S0[1] = fmaf(k.y, u.x, S0[1]); S1[1] = fmaf(k.y, u.y, S1[1]);
+                S0[2] = fmaf(k.z, u.x, S0[2]); S1[2] = fmaf(k.z, u.y, S1[2]);
+                S0[3] = fmaf(k.w, u.x, S0[3]); S1[3] = fmaf(k.w, u.y, S1[3]);
+            }
+        }
+        publish();                                      // (the last reads of the columns lie two barriers back)
+        __syncthreads();                                // this chunk's rows may be overwritten
+    }
+    asm volatile("cp.async.wait_group 0;\n" ::);
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+        const int d = 4 * dg + q;
+        if (holds && d < p.dim) {
+            if (on0) slot[(int64_t)d * p.vdim + col0] = S0[q];
+            if (on1) slot[(int64_t)d * p.vdim + col1] = S1[q];
+        }
+    }
+}
+
+template <int DP>
+__global__ void __launch_bounds__(256, 2) delta_chunk_out_kernel(const DeltaChunkParams p) {
+    constexpr int LD = DP + DC_PAD, LO = DC_OT + DC_PAD, LA = DC + DC_PAD;
+    extern __shared__ __align__(16) float sm[];
+    float* sQ = sm;                                     // [DC][LD]
+    float* sS = sQ + DC * LD;                           // [DP][LO]
+    float* sU = sS + DP * LO;                           // [DC][LO]
+    float* sP = sU + DC * LO;                           // [DC][LA]
+    __shared__ float sb[DC];
+    pdl_wait();
+    pdl_trigger();
+    const int h = blockIdx.y, kh = h / (p.H / p.KH), v0 = blockIdx.z * DC_OT, tid = threadIdx.x;
+    int r, first, n;
+    if (!chunk_of(blockIdx.x, p.row_start, p.rows, r, first, n)) return;
+    load_rows<DP>(sQ, p.q + ((int64_t)first * p.KH + kh) * p.dim, (int64_t)p.KH * p.dim, n, p.dim);
+    const float* S = p.s0 + ((int64_t)blockIdx.x * p.H + h) * p.dim * p.vdim + v0;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int e = tid; e < DP * (DC_OT / 4); e += 256) {
+        const int d = e / (DC_OT / 4), c = (e % (DC_OT / 4)) * 4;
+        if (d < p.dim && v0 + c < p.vdim) dc_cp16(sS + d * LO + c, S + (int64_t)d * p.vdim + c);
+        else *reinterpret_cast<float4*>(sS + d * LO + c) = zero;
+    }
+    for (int e = tid; e < DC * (DC_OT / 4); e += 256) {
+        const int j = e / (DC_OT / 4), c = (e % (DC_OT / 4)) * 4;
+        if (j < n && v0 + c < p.vdim) dc_cp16(sU + j * LO + c, p.u + ((int64_t)(first + j) * p.H + h) * p.vdim + v0 + c);
+        else *reinterpret_cast<float4*>(sU + j * LO + c) = zero;
+    }
+    for (int e = tid; e < DC * (DC / 4); e += 256) {
+        const int i = e / (DC / 4), j = (e % (DC / 4)) * 4;
+        if (i < n && j / 16 <= i / 16) dc_cp16(sP + i * LA + j, p.p + ((int64_t)(first + i) * p.H + h) * DC + j);
+        else *reinterpret_cast<float4*>(sP + i * LA + j) = zero;
+    }
+    asm volatile("cp.async.commit_group;\n" ::);
+    if (tid < DC) sb[tid] = p.b[(int64_t)(first + min(tid, n - 1)) * p.H + h];
+    asm volatile("cp.async.wait_group 0;\n" ::);
+    __syncthreads();
+    const int tx = tid & 15, ty = tid >> 4;             // rows ty + 16 ii, columns 4 tx .. 4 tx + 3
+    float4 acc[4];
+#pragma unroll
+    for (int ii = 0; ii < 4; ++ii) acc[ii] = zero;
+    auto axpy = [](float a, const float4& x, float4& y) {
+        y.x = fmaf(a, x.x, y.x); y.y = fmaf(a, x.y, y.y); y.z = fmaf(a, x.z, y.z); y.w = fmaf(a, x.w, y.w);
+    };
+#pragma unroll 2
+    for (int d = 0; d < DP; d += 4) {
+        float4 s[4];
+#pragma unroll
+        for (int q = 0; q < 4; ++q) s[q] = *reinterpret_cast<const float4*>(sS + (d + q) * LO + 4 * tx);
+#pragma unroll
+        for (int ii = 0; ii < 4; ++ii) {
+            const float4 q4 = *reinterpret_cast<const float4*>(sQ + (ty + 16 * ii) * LD + d);
+            axpy(q4.x, s[0], acc[ii]); axpy(q4.y, s[1], acc[ii]); axpy(q4.z, s[2], acc[ii]); axpy(q4.w, s[3], acc[ii]);
+        }
+    }
+#pragma unroll
+    for (int ii = 0; ii < 4; ++ii) {
+        const float g = expf(sb[ty + 16 * ii]);
+        acc[ii] = make_float4(acc[ii].x * g, acc[ii].y * g, acc[ii].z * g, acc[ii].w * g);
+    }
+#pragma unroll
+    for (int jb = 0; jb < 4; ++jb) {                    // blocks of 16 keys; rows before the block see none of it
+#pragma unroll
+        for (int j = 16 * jb; j < 16 * jb + 16; j += 4) {
+            float4 u[4];
+#pragma unroll
+            for (int q = 0; q < 4; ++q) u[q] = *reinterpret_cast<const float4*>(sU + (j + q) * LO + 4 * tx);
+#pragma unroll
+            for (int ii = jb; ii < 4; ++ii) {
+                const float4 p4 = *reinterpret_cast<const float4*>(sP + (ty + 16 * ii) * LA + j);
+                axpy(p4.x, u[0], acc[ii]); axpy(p4.y, u[1], acc[ii]); axpy(p4.z, u[2], acc[ii]); axpy(p4.w, u[3], acc[ii]);
+            }
+        }
+    }
+#pragma unroll
+    for (int ii = 0; ii < 4; ++ii) {
+        const int i = ty + 16 * ii;
+        if (i < n && v0 + 4 * tx < p.vdim)
+            *reinterpret_cast<float4*>(p.out + ((int64_t)(first + i) * p.H + h) * p.vdim + v0 + 4 * tx) = acc[ii];
+    }
+}
+
+template <int DP> static int launch_delta_chunk(const DeltaChunkParams& p, int ids, cudaStream_t stream) {
+    constexpr int LD = DP + DC_PAD;
+    const size_t solve = (size_t)(2 * DC * LD + DC * (DC + DC_PAD)) * sizeof(float);
+    const size_t walk = (size_t)(4 * DC * LD + DC_VT * LD + DC * 16 + 8 * 128) * sizeof(float);
+    const size_t out = (size_t)(DC * LD + DP * (DC_OT + DC_PAD) + DC * (DC_OT + DC_PAD) + DC * (DC + DC_PAD)) * sizeof(float);
+    static AcornPerDevice configured;
+    if (!configured.seen()) {
+        cudaError_t e = cudaFuncSetAttribute(delta_chunk_solve_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)solve);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_chunk_state_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)walk);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_chunk_out_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)out);
+        if (e != cudaSuccess) return (int)e;
+        configured.mark();
+    }
+    int rc = acorn_launch(delta_chunk_solve_kernel<DP>, dim3(ids, p.H), dim3(256), solve, stream, p);
+    if (rc) return rc;
+    rc = acorn_launch(delta_chunk_state_kernel<DP>, dim3((p.vdim + DC_VT - 1) / DC_VT, p.H, p.rows), dim3(256), walk, stream, p);
+    if (rc) return rc;
+    return acorn_launch(delta_chunk_out_kernel<DP>, dim3(ids, p.H, (p.vdim + DC_OT - 1) / DC_OT), dim3(256), out, stream, p);
+}
+
+extern "C" int acorn_delta_chunk_supported(int dim, int vdim) { return dim >= 4 && dim <= 128 && dim % 4 == 0 && vdim >= 4 && vdim % 4 == 0; }
+
+// chunk numbers of a step (what s0 must have room for)
+extern "C" int acorn_delta_chunk_ids(int tokens, int rows) { return tokens / DC + rows; }
+
+extern "C" int acorn_delta_chunk(const float* q, const float* k, const float* v, const float* beta, const float* log_g, float* state,
+                                 int64_t slot_stride, const int* row_start, const int* row_slot, float* w, float* u, float* pp, float* b,
+                                 float* s0, float* out, int tokens, int rows, int H, int KH, int dim, int vdim, cudaStream_t stream) {
+    if (tokens <= 0 || rows <= 0) return 0;
+    const uintptr_t all = (uintptr_t)q | (uintptr_t)k | (uintptr_t)w | (uintptr_t)u | (uintptr_t)pp | (uintptr_t)s0 | (uintptr_t)out;
+    if (!acorn_delta_chunk_supported(dim, vdim) || KH < 1 || H < 1 || H % KH || H > 65535 || rows > 65535 || (all & 15)) return ACORN_ERR_UNSUPPORTED;
+    DeltaChunkParams p = {q, k, v, beta, log_g, state, slot_stride, row_start, row_slot, w, u, pp, b, s0, out, rows, H, KH, dim, vdim};
+    const int ids = acorn_delta_chunk_ids(tokens, rows);
+    if (dim <= 32) return launch_delta_chunk<32>(p, ids, stream);
+    if (dim <= 64) return launch_delta_chunk<64>(p, ids, stream);
+    return launch_delta_chunk<128>(p, ids, stream);
+}

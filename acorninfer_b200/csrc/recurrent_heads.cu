@@ -4,7 +4,7 @@
 //   delta_heads_prep   gated delta rule with one decay per head, per token: the short causal convolution over time of the
 //                      q, k, v channels with silu (inputs before the step's first token from the request's state, whose
 //                      rows of a single token it shifts), unit norms x / sqrt(sum x^2 + 1e-6) of q and k (q also times
-//                      dim^-1/2), beta = sigmoid(.), g = exp(-exp(A_log) softplus(. + dt_bias)); float32 out
+//                      dim^-1/2), beta = sigmoid(.), log g = -exp(A_log) softplus(. + dt_bias) and g; float32 out
 //   linear_heads_prep  gated linear attention, per token: q times dim^-1/2, k, v as they are, and the decay per key channel
 //                      sigmoid(z + bias)^(1 / tau); float32 out
 //   recurrent_step     rows of one token: a block a (row, head) reads the head's state once, decays it, corrects and writes
@@ -41,6 +41,7 @@ template <typename T> struct DeltaHeadsParams {
     float* vv;
     float* beta;
     float* g;
+    float* log_g;
     int tokens, H, KH, dim, vdim, taps, update_single;
 };
 
@@ -134,7 +135,9 @@ __global__ void delta_heads_prep_vec_kernel(const DeltaHeadsParams<T> p, int lph
                 dst = p.vv + (t * p.H + vh) * p.vdim;
                 if (l == 0) {
                     p.beta[t * p.H + vh] = rh_sigmoid(to_float(p.in[t * p.ld + p.beta0 + vh]));
-                    p.g[t * p.H + vh] = expf(-A * rh_softplus(to_float(p.in[t * p.ld + p.decay0 + vh]) + bias));
+                    const float lg = -A * rh_softplus(to_float(p.in[t * p.ld + p.decay0 + vh]) + bias);
+                    p.g[t * p.H + vh] = expf(lg);
+                    p.log_g[t * p.H + vh] = lg;
                 }
             } else {
                 const bool is_q = h < p.KH;
@@ -189,7 +192,9 @@ __global__ void delta_heads_prep_kernel(const DeltaHeadsParams<T> p) {
     if (is_v) {
         if (lane == 0) {
             p.beta[(int64_t)t * p.H + vh] = rh_sigmoid(to_float(p.in[(int64_t)t * p.ld + p.beta0 + vh]));
-            p.g[(int64_t)t * p.H + vh] = expf(-expf(p.A_log[vh]) * rh_softplus(to_float(p.in[(int64_t)t * p.ld + p.decay0 + vh]) + p.dt_bias[vh]));
+            const float lg = -expf(p.A_log[vh]) * rh_softplus(to_float(p.in[(int64_t)t * p.ld + p.decay0 + vh]) + p.dt_bias[vh]);
+            p.g[(int64_t)t * p.H + vh] = expf(lg);
+            p.log_g[(int64_t)t * p.H + vh] = lg;
         }
         return;
     }
@@ -229,7 +234,7 @@ template <typename T> static int launch_delta_heads(const DeltaHeadsParams<T>& p
 extern "C" int acorn_delta_heads_prep(const void* in, int64_t ld, int beta0, int decay0, const float* conv_w, int taps, float* state,
                                       int64_t slot_stride, int64_t conv_off, const float* A_log, const float* dt_bias,
                                       const int* token_row, const int* row_start, const int* row_slot, int update_single,
-                                      float* qn, float* kn, float* vv, float* beta, float* g, int tokens, int H, int KH, int dim,
+                                      float* qn, float* kn, float* vv, float* beta, float* g, float* log_g, int tokens, int H, int KH, int dim,
                                       int vdim, int dtype, cudaStream_t stream) {
     if (tokens <= 0) return 0;
     if (KH < 1 || H < 1 || H % KH || dim < 1 || vdim < 1 || (conv_w && (taps < 1 || taps > RH_MAX_TAPS)) ||
@@ -240,7 +245,7 @@ extern "C" int acorn_delta_heads_prep(const void* in, int64_t ld, int beta0, int
         p.in = (const T*)in; p.ld = ld; p.beta0 = beta0; p.decay0 = decay0; p.conv_w = conv_w; p.taps = taps; p.state = state;
         p.slot_stride = slot_stride; p.conv_off = conv_off; p.A_log = A_log; p.dt_bias = dt_bias; p.token_row = token_row;
         p.row_start = row_start; p.row_slot = row_slot; p.update_single = update_single; p.qn = qn; p.kn = kn; p.vv = vv;
-        p.beta = beta; p.g = g; p.tokens = tokens; p.H = H; p.KH = KH; p.dim = dim; p.vdim = vdim;
+        p.beta = beta; p.g = g; p.log_g = log_g; p.tokens = tokens; p.H = H; p.KH = KH; p.dim = dim; p.vdim = vdim;
         return launch_delta_heads<T>(p, stream);
     });
     return ACORN_ERR_UNSUPPORTED;

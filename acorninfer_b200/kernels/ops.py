@@ -169,8 +169,12 @@ class _Sigs:
                          c_void_p, c_int64, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                          c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p]
     acorn_delta_heads_prep = [c_void_p, c_int64, c_int, c_int, c_void_p, c_int, c_void_p, c_int64, c_int64, c_void_p, c_void_p,
-                              c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                              c_int, c_int, c_int, c_int, c_void_p]
+                              c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                              c_int, c_int, c_int, c_int, c_int, c_void_p]
+    acorn_delta_chunk = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p,
+                         c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
+    acorn_delta_chunk_supported = [c_int, c_int]
+    acorn_delta_chunk_ids = [c_int, c_int]
     acorn_linear_heads_prep = [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p,
                                c_int, c_int, c_int, c_int, c_int, c_void_p]
     acorn_recurrent_step = [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64,
@@ -361,7 +365,7 @@ class _TimedLib:
 
     def __getattr__(self, name):
         fn = getattr(self._library, name)
-        if not name.startswith("acorn_") or name.endswith(("_supported", "_error", "_merges", "_scratch")):
+        if not name.startswith("acorn_") or name.endswith(("_supported", "_error", "_merges", "_scratch", "_ids")):
             return fn
 
         def timed(*args):
@@ -1512,19 +1516,48 @@ def delta_segments(longest_row: int, num_rows: int, heads: int, dim: int, vdim: 
     return -(-longest_row // nseg), nseg
 
 
+DELTA_CHUNK_MIN_ROW = 64            # tokens: shorter rows are walked one by one
+DELTA_CHUNK_SCRATCH_BYTES = 4 << 30
+
+
+def delta_chunk(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Tensor, log_g: torch.Tensor, state: torch.Tensor,
+                row_start: torch.Tensor, row_slot: torch.Tensor, num_rows: int, state_off: int = 0) -> torch.Tensor:
+    """The gated delta rule with one decay per head (``log_g`` [T, H], logarithms) over chunks of 64 tokens: what a chunk adds
+    whatever state it starts from is worked out for all chunks side by side, then the states are carried from chunk to
+    chunk, then all outputs are read out side by side.  Arguments and result as for ``delta_rule``."""
+    T, H, vdim = v.shape
+    KH, dim = q.shape[1], q.shape[2]
+    for t, n in ((q, "q"), (k, "k"), (v, "v"), (beta, "beta"), (log_g, "log_g")):
+        _check(t, n, torch.float32)
+    _check(state, "state", torch.float32, 2)
+    if log_g.shape != (T, H) or beta.shape != (T, H) or state.shape[1] < state_off + H * dim * vdim:
+        raise KernelError(f"delta_chunk: log_g {tuple(log_g.shape)}, state {tuple(state.shape)} do not fit")
+    f = lambda *shape: torch.empty(shape, dtype=torch.float32, device=v.device)
+    w, u, p, b, out = f(T, H, dim), f(T, H, vdim), f(T, H, 64), f(T, H), f(T, H, vdim)
+    s0 = f(lib().acorn_delta_chunk_ids(T, num_rows), H, dim, vdim)
+    _ok(lib().acorn_delta_chunk(q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(), log_g.data_ptr(),
+                                state.data_ptr() + 4 * int(state_off), state.stride(0), row_start.data_ptr(), row_slot.data_ptr(),
+                                w.data_ptr(), u.data_ptr(), p.data_ptr(), b.data_ptr(), s0.data_ptr(), out.data_ptr(), T, num_rows, H,
+                                KH, dim, vdim, _stream()), "delta_chunk")
+    return out
+
+
 DELTA_FORMS = {"rule": 0, "pre": 1, "linear": 2}
 
 
 def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Tensor | None, g: torch.Tensor,
                state: torch.Tensor, row_start: torch.Tensor, row_slot: torch.Tensor, num_rows: int,
-               bonus32: torch.Tensor | None = None, longest_row: int | None = None, state_off: int = 0) -> torch.Tensor:
+               bonus32: torch.Tensor | None = None, longest_row: int | None = None, state_off: int = 0,
+               log_g: torch.Tensor | None = None) -> torch.Tensor:
     """The recurrence over every row's tokens from the state in its slot (at ``state_off``, updated in place): float32
     o [T, H, vdim].  Three forms: with ``beta`` the delta rule; with ``bonus32`` (float32 [H, dim]) and no ``beta`` the form
     without the correction whose output reads the state before the token's decay and write and sees the token itself
     through the bonus: ``o = S^T q + (sum_d q_d bonus_d k_d) v;  S = diag(g) S + k v^T``; with neither gated linear
     attention: ``S = diag(g) S + k v^T;  o = S^T q``.  Decays ``g``: [T, H, dim], or [T, H], one per head.  In the forms
     without correction, with ``longest_row`` (the most tokens a row of the step brings, a host value), long rows of a
-    step with few rows run in segments side by side (``delta_segments``)."""
+    step with few rows run in segments side by side (``delta_segments``).  The delta rule with decays per head runs over
+    chunks of tokens (``delta_chunk``) where a step has a row of ``DELTA_CHUNK_MIN_ROW`` tokens and the decays' logarithms
+    ``log_g`` [T, H] are given."""
     T, H, vdim = v.shape
     KH, dim = q.shape[1], q.shape[2]
     if beta is not None and bonus32 is not None:
@@ -1540,6 +1573,10 @@ def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Te
     per_head = g.dim() == 2
     if state.shape[1] < state_off + H * dim * vdim or g.shape != ((T, H) if per_head else (T, H, dim)) or dim > 256:
         raise KernelError(f"delta_rule: sizes do not fit (state {tuple(state.shape)}, g {tuple(g.shape)}, H={H}, dim={dim}, vdim={vdim})")
+    if (beta is not None and log_g is not None and (longest_row or 0) >= DELTA_CHUNK_MIN_ROW
+            and lib().acorn_delta_chunk_supported(dim, vdim)
+            and 4 * lib().acorn_delta_chunk_ids(T, num_rows) * H * dim * vdim <= DELTA_CHUNK_SCRATCH_BYTES):
+        return delta_chunk(q, k, v, beta, log_g, state, row_start, row_slot, num_rows, state_off)
     out = torch.empty((T, H, vdim), dtype=torch.float32, device=v.device)
     seg_len, nseg = delta_segments(longest_row, num_rows, H, dim, vdim) if (beta is None and longest_row) else (0, 1)
     s_ptr = state.data_ptr() + 4 * int(state_off)
@@ -1586,8 +1623,8 @@ def delta_heads_prep(proj: torch.Tensor, beta_col: int, decay_col: int, conv_w32
                      update_single: bool = False):
     """For a gated delta rule with one decay per head, of projected rows ``[q | k | v | ...]`` (a row stride is allowed; the
     write strengths' columns start at ``beta_col``, the decays' at ``decay_col``): convolution over time + silu of the q, k,
-    v channels, unit norms of q and k (q also times dim^-1/2), ``sigmoid``, ``exp(-exp(A_log) softplus(. + dt_bias))``.  Float32
-    (q [T, KH, dim], k, v [T, H, vdim], beta [T, H], g [T, H]).  ``update_single``: the convolution's memory of rows of one
+    v channels, unit norms of q and k (q also times dim^-1/2), ``sigmoid``, the decays ``exp(-exp(A_log) softplus(. + dt_bias))``.
+    Float32 (q [T, KH, dim], k, v [T, H, vdim], beta [T, H], g [T, H], log g [T, H]).  ``update_single``: the convolution's memory of rows of one
     token is shifted here (``conv_state_update(skip_single=True)`` does the longer rows)."""
     _rows2(proj, "proj")
     T, C = proj.shape[0], 2 * kv_heads * dim + heads * vdim
@@ -1600,14 +1637,14 @@ def delta_heads_prep(proj: torch.Tensor, beta_col: int, decay_col: int, conv_w32
         if conv_w32.shape[0] != C or (taps > 1 and (state is None or state.shape[1] < conv_off + (taps - 1) * C)):
             raise KernelError("delta_heads_prep: convolution weights or memory do not fit")
     f = lambda *shape: torch.empty(shape, dtype=torch.float32, device=proj.device)
-    q, k, v, beta, g = f(T, kv_heads, dim), f(T, kv_heads, dim), f(T, heads, vdim), f(T, heads), f(T, heads)
+    q, k, v, beta, g, log_g = f(T, kv_heads, dim), f(T, kv_heads, dim), f(T, heads, vdim), f(T, heads), f(T, heads), f(T, heads)
     _ok(lib().acorn_delta_heads_prep(proj.data_ptr(), proj.stride(0), int(beta_col), int(decay_col), _ptr(conv_w32), taps, _ptr(state),
                                      state.stride(0) if state is not None else 0, int(conv_off), a_log32.data_ptr(),
                                      dt_bias32.data_ptr(), token_row.data_ptr(), row_start.data_ptr(), row_slot.data_ptr(),
                                      1 if update_single else 0, q.data_ptr(), k.data_ptr(), v.data_ptr(), beta.data_ptr(),
-                                     g.data_ptr(), T, heads, kv_heads, dim, vdim, dtype_code(proj.dtype), _stream()),
+                                     g.data_ptr(), log_g.data_ptr(), T, heads, kv_heads, dim, vdim, dtype_code(proj.dtype), _stream()),
         "delta_heads_prep")
-    return q, k, v, beta, g
+    return q, k, v, beta, g, log_g
 
 
 def linear_heads_prep(proj: torch.Tensor, z32: torch.Tensor, bias32: torch.Tensor, tau: float, heads: int, dim: int, vdim: int):
@@ -1641,7 +1678,7 @@ def recurrent_step(state: torch.Tensor, state_off: int, row_slot: torch.Tensor, 
                    linear=None) -> torch.Tensor:
     """A step of single-token rows (row r brings token r) through a recurrence and what follows it, in one kernel: the state
     of every head read and written once, the read-out over its root mean square (per head) times ``norm_w32`` [vdim] times
-    ``silu(gate)`` times ``out_scale``, into ``out`` [T, H vdim].  ``delta`` = (q, k, v, beta, g) of ``delta_heads_prep``: the
+    ``silu(gate)`` times ``out_scale``, into ``out`` [T, H vdim].  ``delta`` = (q, k, v, beta, g, ...) of ``delta_heads_prep``: the
     delta rule; ``linear`` = (proj, z32, bias32, tau) as ``linear_heads_prep`` takes them: gated linear attention."""
     _check(state, "state", torch.float32, 2)
     _rows2(gate, "gate")
@@ -1653,7 +1690,7 @@ def recurrent_step(state: torch.Tensor, state_off: int, row_slot: torch.Tensor, 
     q = k = v = beta = g = proj = z = bias = None
     kv_heads, tau = heads, 1.0
     if delta is not None:
-        q, k, v, beta, g = delta
+        q, k, v, beta, g = delta[:5]
         kv_heads = q.shape[1]
         if q.shape != (T, kv_heads, dim) or v.shape != (T, heads, vdim) or g.shape != (T, heads):
             raise KernelError("recurrent_step: the delta rule's inputs do not fit")

@@ -122,9 +122,9 @@ class HeadDelta(_HeadsMixer):
         if self._steps(inputs, cache, (gate, out)):
             return ops.recurrent_step(cache.state, self.state_base, inputs.row_slot, gate, self.norm32, self.eps, out, self.H,
                                       self.dim, self.vdim, out_scale, delta=ins)
-        q, k, v, beta, g = ins
+        q, k, v, beta, g, log_g = ins
         o = ops.delta_rule(q, k, v, beta, g, cache.state, inputs.row_start, inputs.row_slot, inputs.num_rows,
-                           longest_row=inputs.plan.max_q_len, state_off=self.state_base)
+                           longest_row=inputs.plan.max_q_len, state_off=self.state_base, log_g=log_g)
         return ops.gated_norm(o.view(o.shape[0], -1), gate, self.norm_heads32, self.eps, self.H, False, out, out_scale, silu=True)
 
 

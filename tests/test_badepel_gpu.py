@@ -567,8 +567,8 @@ def test_delta_rule_across_steps(H, KH, dim, vdim, taps, dtype, tol):
         if max(n) == 1 and o.recurrent_step_ok(dim, vdim, (sd, sd.stride(0), s_off), (gate, y)):
             o.recurrent_step(sd, s_off, slot_t, gate, dv(norm_w), eps, y, H, dim, vdim, 0.9, delta=ins)
         else:
-            q, k, v, beta, dec = ins
-            r = o.delta_rule(q, k, v, beta, dec, sd, starts, slot_t, len(n), longest_row=max(n), state_off=s_off)
+            q, k, v, beta, dec, log_dec = ins
+            r = o.delta_rule(q, k, v, beta, dec, sd, starts, slot_t, len(n), longest_row=max(n), state_off=s_off, log_g=log_dec)
             o.gated_norm(r.view(x.shape[0], -1), gate, dv(norm_w.repeat(H)), eps, H, False, y, 0.9, silu=True)
         return torch.split(y.float().cpu(), n)
 
@@ -619,10 +619,50 @@ def test_delta_rule_long_memory():
         for a, b in (((0, cut), (cut, T)) if cut else ((0, T),)):
             got.append(o.delta_rule(f(q[a:b]), f(k[a:b]), f(v[a:b]), f(beta[a:b]), f(dec[a:b]), state,
                                     torch.tensor([0, b - a], dtype=torch.int32, device=DEV), torch.tensor([1], dtype=torch.int32, device=DEV), 1,
-                                    longest_row=b - a).double().cpu())
+                                    longest_row=b - a, log_g=f(dec[a:b].log())).double().cpu())
         got = torch.cat(got)
         want = beta[0][:, None] * v[0] * (0.9995 ** torch.arange(T, dtype=torch.float64))[:, None, None]
         assert (got - want).abs().max() < 2e-5 * float(want.abs().max()), (T, cut)
+
+
+@pytest.mark.parametrize("H,KH,dim,vdim", [(4, 2, 8, 12), (3, 3, 32, 20), (2, 1, 64, 64), (6, 3, 96, 80), (2, 2, 128, 128), (1, 1, 128, 200)])
+def test_delta_chunks(H, KH, dim, vdim):
+    """The delta rule over chunks of tokens against the loop over tokens and against the kernel that walks them: rows that end
+    on and around a chunk's edge, many and unequal rows in one step, keys that repeat (a system far from the identity),
+    decays from none to those that leave nothing, states that were there before."""
+    o = ops()
+    g = torch.Generator().manual_seed(dim + vdim)
+    for lens in ([64], [65, 1, 63], [1, 200, 2, 128, 129, 5, 64, 192], [330]):
+        T, slots = sum(lens), list(np.random.default_rng(len(lens)).permutation(10)[:len(lens)])
+        base = _rand(g, KH, dim)
+        k = plain.unit((_rand(g, T, KH, dim, scale=0.4) + base).double())          # neighbouring keys are alike
+        q = plain.unit(_rand(g, T, KH, dim).double()) * dim ** -0.5
+        v, beta = _rand(g, T, H, vdim).double(), torch.rand(T, H, generator=g).double()
+        log_g = -torch.exp(_rand(g, T, H, scale=2.0).double() - 3.0)
+        log_g[T // 2] = -90.0
+        state = _rand(g, 10, H * dim * vdim + 4)
+        f = lambda t: t.float().contiguous().to(DEV)
+        starts = torch.tensor(np.cumsum([0] + lens), dtype=torch.int32, device=DEV)
+        slot_t = torch.tensor(slots, dtype=torch.int32, device=DEV)
+        got, ends = {}, {}
+        for how in ("chunks", "walk"):
+            sd = state.to(DEV)
+            if how == "chunks":
+                out = o.delta_chunk(f(q), f(k), f(v), f(beta), f(log_g), sd, starts, slot_t, len(lens), state_off=4)
+            else:
+                out = o.delta_rule(f(q), f(k), f(v), f(beta), f(log_g.exp()), sd, starts, slot_t, len(lens), state_off=4)
+            got[how], ends[how] = out.double().cpu(), sd.double().cpu()
+        group, at = torch.arange(H) // (H // KH), 0
+        for r, n in enumerate(lens):
+            rows = slice(at, at + n)
+            want, S = plain.delta_recurrence(q[rows][:, group], k[rows][:, group], v[rows], beta[rows], log_g[rows].exp(),
+                                             state[slots[r], 4:].double().view(H, dim, vdim))
+            for how in got:
+                assert (got[how][rows] - want).abs().max() < 3e-5 * float(want.abs().max()), (lens, r, how)
+                assert (ends[how][slots[r], 4:].view(H, dim, vdim) - S).abs().max() < 3e-5 * float(S.abs().max()), (lens, r, how)
+            at += n
+        untouched = [s for s in range(10) if s not in slots]
+        assert torch.equal(ends["chunks"][untouched], state[untouched].double()) and torch.equal(ends["chunks"][:, :4], state[:, :4].double())
 
 
 @pytest.mark.parametrize("dtype,tol", [(torch.float32, 2e-5), (torch.bfloat16, 2e-2)])
