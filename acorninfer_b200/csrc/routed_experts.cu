@@ -197,6 +197,133 @@ __global__ void __launch_bounds__(1024) moe_route_plan_kernel(const float* __res
     plan_pairs(idx, offsets, slot_of, slot_token, tokens * top, N, top, wts, slot_wts, reinterpret_cast<int*>(sm));
 }
 
+// The same where outputs form one group: a warp a token, its logits and scores in registers (NV a lane), what was chosen in
+// shared memory until it is grouped.
+#define MOE_SMALL_CHOICES 1024
+
+template <int NV>
+__global__ void __launch_bounds__(1024) moe_route_plan_small_kernel(const float* __restrict__ z, int64_t ldz, const float* __restrict__ bias,
+                                                                    const float* __restrict__ correction, int* __restrict__ idx,
+                                                                    float* __restrict__ wts, int tokens, int N, int top, int normalize,
+                                                                    int scoring, int* __restrict__ offsets, int* __restrict__ slot_of,
+                                                                    int* __restrict__ slot_token, float* __restrict__ slot_wts) {
+    __shared__ int s_idx[MOE_SMALL_CHOICES];
+    __shared__ float s_wts[MOE_SMALL_CHOICES];
+    __shared__ int s_cnt[MOE_SMALL_OUTPUTS], s_cursor[MOE_SMALL_OUTPUTS];
+    for (int i = threadIdx.x; i < N; i += blockDim.x) s_cnt[i] = 0;
+    __syncthreads();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    float add[NV], corr[NV];
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int i = lane + 32 * k;
+        add[k] = bias && i < N ? bias[i] : 0.f;
+        corr[k] = correction && i < N ? correction[i] : 0.f;
+    }
+    pdl_wait();
+    pdl_trigger();
+    for (int t = warp; t < tokens; t += warps) {
+        float s[NV], choice[NV];
+        float m = -INFINITY;
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            const int i = lane + 32 * k;
+            choice[k] = i < N ? z[(int64_t)t * ldz + i] + add[k] : -INFINITY;
+            m = fmaxf(m, choice[k]);
+        }
+        m = warp_max(m);
+        float sum = 0.f;
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            s[k] = lane + 32 * k >= N ? 0.f : (scoring == 1 ? 1.f / (1.f + expf(-choice[k])) : expf(choice[k] - m));
+            sum += s[k];
+        }
+        sum = scoring == 1 ? 1.f : warp_sum(sum);
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            s[k] /= sum;
+            if (correction && lane + 32 * k < N) choice[k] = s[k] + corr[k];
+        }
+        float total = 0.f, mine = 0.f;                  // the chosen's scores; lane k keeps the k-th choice's
+        int mine_i = 0;
+        for (int c = 0; c < top; ++c) {
+            float best = -INFINITY, score = 0.f;
+            int best_i = N;
+#pragma unroll
+            for (int k = 0; k < NV; ++k)
+                if (choice[k] > best) {
+                    best = choice[k];
+                    best_i = lane + 32 * k;
+                    score = s[k];
+                }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ob = __shfl_xor_sync(0xffffffffu, best, o), os = __shfl_xor_sync(0xffffffffu, score, o);
+                const int oi = __shfl_xor_sync(0xffffffffu, best_i, o);
+                if (ob > best || (ob == best && oi < best_i)) {
+                    best = ob;
+                    best_i = oi;
+                    score = os;
+                }
+            }
+#pragma unroll
+            for (int k = 0; k < NV; ++k)
+                if (best_i == lane + 32 * k) choice[k] = -INFINITY;
+            if (best_i >= N) {                          // nothing left to choose
+                best_i = 0;
+                score = 0.f;
+            }
+            total += score;
+            if ((c & 31) == lane) {
+                mine = score;
+                mine_i = best_i;
+            }
+            if ((c & 31) == 31 || c == top - 1) {
+                const int at = t * top + (c & ~31) + lane;
+                if ((c & ~31) + lane <= c) {
+                    s_idx[at] = mine_i;
+                    s_wts[at] = mine;
+                    atomicAdd(&s_cnt[mine_i], 1);
+                }
+            }
+        }
+        __syncwarp();
+        const float by = normalize ? total + 1e-20f : 1.f;
+        for (int c = lane; c < top; c += 32) {
+            const float w = s_wts[t * top + c] / by;
+            s_wts[t * top + c] = w;
+            idx[(int64_t)t * top + c] = s_idx[t * top + c];
+            wts[(int64_t)t * top + c] = w;
+        }
+    }
+    __syncthreads();
+    if (warp == 0) {                                    // exclusive sums over the outputs
+        int run = 0;
+        for (int base = 0; base < N; base += 32) {
+            const int i = base + lane, n = i < N ? s_cnt[i] : 0;
+            int inc = n;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int before = __shfl_up_sync(0xffffffffu, inc, o);
+                if (lane >= o) inc += before;
+            }
+            if (i < N) {
+                offsets[i] = run + inc - n;
+                s_cursor[i] = run + inc - n;
+            }
+            run += __shfl_sync(0xffffffffu, inc, 31);
+        }
+        if (lane == 0) offsets[N] = run;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < tokens * top; i += blockDim.x) {
+        const int slot = atomicAdd(&s_cursor[s_idx[i]], 1);
+        slot_of[i] = slot;
+        slot_token[slot] = i / top;
+        if (slot_wts) slot_wts[slot] = s_wts[i];
+    }
+}
+
 extern "C" int acorn_moe_route_plan_supported(int tokens, int N) { return tokens <= MOE_SMALL_TOKENS && N <= MOE_SMALL_OUTPUTS; }
 
 extern "C" int acorn_moe_route_plan(const float* z, int64_t ldz, const float* bias, const float* correction, int* idx, float* wts, int tokens,
@@ -207,6 +334,14 @@ extern "C" int acorn_moe_route_plan(const float* z, int64_t ldz, const float* bi
         groups < 1 || groups > 64 || N % groups || keep < 1 || keep > groups)
         return ACORN_ERR_UNSUPPORTED;
     const int warps = tokens < 8 ? 8 : (tokens > 32 ? 32 : tokens);
+    if (groups == 1 && tokens * top <= MOE_SMALL_CHOICES) {
+#define SMALL(NV) return acorn_launch(moe_route_plan_small_kernel<NV>, dim3(1), dim3(32 * (tokens > 32 ? 32 : tokens)), 0, stream, z, ldz, bias, \
+                                      correction, idx, wts, tokens, N, top, normalize, scoring, offsets, slot_of, slot_token, slot_wts)
+        if (N <= 32) SMALL(1);
+        if (N <= 64) SMALL(2);
+        SMALL(5);
+#undef SMALL
+    }
     return acorn_launch(moe_route_plan_kernel, dim3(1), dim3(32 * warps), (size_t)warps * 2 * N * sizeof(float), stream, z, ldz, bias,
                         correction, idx, wts, tokens, N, top, groups, keep, normalize, scoring, offsets, slot_of, slot_token,
                         slot_wts);
@@ -336,7 +471,7 @@ __global__ void __launch_bounds__(256) grouped_gemm_kernel(const T* __restrict__
 // weight rows; eight warps; operand tiles of 64 along K through a ring of cp.async stages.  BM = 128 or 64
 // (warps 2 x 4, 64 x 32 or 32 x 32 each) for steps with many rows an expert, BM = 16 (warps 1 x 8, 16 x 16 each) for
 // decode steps, where the kernel is bound by reading every chosen expert's matrix once.  An output
-// element is the same chain of products in both, so a row's bits do not depend on the step it is in.
+// element is the same chain of products in both.
 #define GT_BN 128
 #define GT_BK 64
 #define GT_LDS (GT_BK + 8)
@@ -477,6 +612,109 @@ __global__ void __launch_bounds__(256) grouped_gemm_tc_kernel(const bf16* __rest
     }
 }
 
+// Few rows an expert (a decode step): what counts is that all of a chosen expert's matrix is on its way at once.  A block: 8 slots
+// of one expert by 16 weight rows (the rows are the 16-row side of mma.sync m16n8k16, the slots its 8 columns); eight warps
+// share K in turns of 32 entries and add up through shared memory.  Operands go from memory straight into fragments: the k
+// entries of a fragment may stand in any order as long as both operands agree, so a lane takes 16 bytes of a row, which
+// are its entries for two k-steps.
+#define GR_AHEAD 8
+
+__global__ void __launch_bounds__(256) grouped_rows_kernel(const bf16* __restrict__ A, int64_t lda, const int* __restrict__ a_rows,
+                                                           const bf16* __restrict__ W, bf16* __restrict__ C, int64_t ldc,
+                                                           const int* __restrict__ offsets, int E, int N, int K, int swiglu,
+                                                           float glu_limit, const float* __restrict__ slot_scale) {
+    __shared__ float red[8][8][17];
+    pdl_wait();
+    pdl_trigger();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    // the expert and slots of tile blockIdx.y, found by every warp for itself
+    int e = -1, first = 0, end = 0;
+    for (int base = 0, run = 0; base < E && e < 0; base += 32) {
+        const int i = base + lane;
+        const int o0 = i < E ? offsets[i] : 0, o1 = i < E ? offsets[i + 1] : 0;
+        const int tiles = (o1 - o0 + 7) / 8;
+        int inc = tiles;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int before = __shfl_up_sync(0xffffffffu, inc, o);
+            if (lane >= o) inc += before;
+        }
+        const int tile = (int)blockIdx.y - run;
+        const unsigned hit = __ballot_sync(0xffffffffu, tile < inc);
+        if (hit) {
+            const int l = __ffs(hit) - 1;
+            e = base + l;
+            const int at = tile - (__shfl_sync(0xffffffffu, inc, l) - __shfl_sync(0xffffffffu, tiles, l));
+            first = __shfl_sync(0xffffffffu, o0, l) + at * 8;
+            end = __shfl_sync(0xffffffffu, o1, l);
+        }
+        run += __shfl_sync(0xffffffffu, inc, 31);
+    }
+    if (e < 0) return;
+    const int g = lane >> 2, t = lane & 3, n0 = blockIdx.x * 16;
+    const bf16* We = W + (int64_t)e * N * K;
+    const bf16* w0 = We + (int64_t)min(n0 + g, N - 1) * K + 8 * t;
+    const bf16* w1 = We + (int64_t)min(n0 + g + 8, N - 1) * K + 8 * t;
+    const int mine = min(first + g, end - 1);           // columns beyond the last slot repeat it and are not stored
+    const bf16* x = A + (a_rows ? (int64_t)a_rows[mine] : (int64_t)mine) * lda + 8 * t;
+    float acc[4] = {};
+    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+    for (int k0 = 32 * warp; k0 < K; k0 += 256 * GR_AHEAD) {
+        uint4 a0[GR_AHEAD], a1[GR_AHEAD], xb[GR_AHEAD];
+#pragma unroll
+        for (int q = 0; q < GR_AHEAD; ++q) {
+            const int k = k0 + 256 * q;
+            const bool in = k + 8 * t < K;
+            a0[q] = in ? *reinterpret_cast<const uint4*>(w0 + k) : zero;
+            a1[q] = in ? *reinterpret_cast<const uint4*>(w1 + k) : zero;
+            xb[q] = in ? *reinterpret_cast<const uint4*>(x + k) : zero;
+        }
+#pragma unroll
+        for (int q = 0; q < GR_AHEAD; ++q) {
+            const uint32_t lo[4] = {a0[q].x, a1[q].x, a0[q].y, a1[q].y}, hi[4] = {a0[q].z, a1[q].z, a0[q].w, a1[q].w};
+            mma_bf16_16816(acc, lo, xb[q].x, xb[q].y);
+            mma_bf16_16816(acc, hi, xb[q].z, xb[q].w);
+        }
+    }
+    red[warp][2 * t][g] = acc[0];
+    red[warp][2 * t + 1][g] = acc[1];
+    red[warp][2 * t][g + 8] = acc[2];
+    red[warp][2 * t + 1][g + 8] = acc[3];
+    __syncthreads();
+    auto total = [&](int col, int row) -> float {
+        float v = 0.f;
+#pragma unroll
+        for (int w = 0; w < 8; ++w) v += red[w][col][row];
+        return v;
+    };
+    const int per = swiglu ? 8 : 16;                    // outputs a slot
+    for (int i = threadIdx.x; i < per * 8; i += 256) {
+        const int col = i / per, o = i % per, slot = first + col;
+        if (slot >= end) continue;
+        const float f = slot_scale ? slot_scale[slot] : 1.f;
+        if (!swiglu) {
+            if (n0 + o < N) C[(int64_t)slot * ldc + n0 + o] = __float2bfloat16_rn(total(col, o) * f);
+            continue;
+        }
+        float gt = total(col, 2 * o) * f, u = total(col, 2 * o + 1) * f, zz = gt;
+        if (glu_limit > 0.f) {                          // the capped form
+            gt = fminf(gt, glu_limit);
+            u = fminf(fmaxf(u, -glu_limit), glu_limit) + 1.f;
+            zz = 1.702f * gt;
+        }
+        if (n0 + 2 * o + 1 < N) C[(int64_t)slot * ldc + (n0 >> 1) + o] = __float2bfloat16_rn(gt / (1.f + expf(-zz)) * u);
+    }
+}
+
+static int grouped_rows_launch(const bf16* A, int64_t lda, const int* a_rows, const bf16* W, bf16* C, int64_t ldc, const int* offsets,
+                               int slots, int E, int N, int K, int swiglu, float glu_limit, const float* slot_scale, cudaStream_t stream) {
+    int64_t tiles = (slots + 7) / 8 + E;
+    if (tiles > slots) tiles = slots;                   // an expert of n slots has at most n tiles
+    if (tiles > 65535) return ACORN_ERR_UNSUPPORTED;
+    return acorn_launch(grouped_rows_kernel, dim3((N + 15) / 16, (unsigned)tiles), dim3(256), 0, stream, A, lda, a_rows, W, C, ldc,
+                        offsets, E, N, K, swiglu, glu_limit, slot_scale);
+}
+
 template <int BM>
 static int grouped_gemm_tc_launch(const bf16* A, int64_t lda, const int* a_rows, const bf16* W, bf16* C, int64_t ldc,
                                   const int* offsets, int slots, int E, int N, int K, int swiglu, float glu_limit,
@@ -510,7 +748,9 @@ extern "C" int acorn_grouped_gemm(const void* A, int64_t lda, const int* a_rows,
     if (swiglu && !(acorn_grouped_gemm_fuses_swiglu(N, K, lda, dtype) && ((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0))
         return ACORN_ERR_UNSUPPORTED;
     if (dtype == ACORN_DTYPE_BF16 && K % 8 == 0 && lda % 8 == 0 && ((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0) {
-        // few rows an expert on average: the small tile (a decode step); else the large one
+        // few rows an expert on average (a decode step): fragments straight from memory; then the small tile; else the large one
+        if ((int64_t)slots <= (int64_t)2 * E)
+            return grouped_rows_launch((const bf16*)A, lda, a_rows, (const bf16*)W, (bf16*)C, ldc, offsets, slots, E, N, K, swiglu, glu_limit, slot_scale, stream);
         if ((int64_t)slots <= (int64_t)16 * E)
             return grouped_gemm_tc_launch<16>((const bf16*)A, lda, a_rows, (const bf16*)W, (bf16*)C, ldc, offsets, slots, E, N, K, swiglu, glu_limit, slot_scale, stream);
         if ((int64_t)slots >= (int64_t)256 * E)          // several full tiles an expert: the tall tile (64 x 32 a warp)

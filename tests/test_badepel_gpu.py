@@ -801,7 +801,7 @@ def test_router_bias_and_weights_over_the_chosen(T, N, top):
     off = offsets.cpu().long()
     assert torch.equal(off[1:] - off[:-1], torch.bincount(best.indices.flatten(), minlength=N))
     idx2, wts2 = o.moe_route(z.to(DEV), None, top, 1, 1, True, "softmax", bias32=bias.to(DEV))
-    assert torch.equal(idx2, idx) and torch.equal(wts2, wts)
+    assert torch.equal(idx2, idx) and (wts2 - wts).abs().max() < 1e-6
 
 
 def test_gated_norm_with_silu():
