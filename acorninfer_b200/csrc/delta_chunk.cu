@@ -1,4 +1,6 @@
-// The gated delta rule with one decay per head, over chunks of 64 tokens (float32 throughout):
+// Two recurrences over chunks of 64 tokens (float32 throughout).
+//
+// The gated delta rule with one decay per head:
 //     S_i = g_i S_(i-1) + k_i u_i^T,   u_i = beta_i (v_i - g_i S_(i-1)^T k_i),   o_i = S_i^T q_i.
 // Within a chunk that starts from S_0, with b_i the sum of the log decays up to i and G_ij = exp(b_i - b_j) (at most one for
 // j <= i), the u_i solve a unit lower triangular system, so what hangs on S_0 can be split off:
@@ -10,6 +12,17 @@
 //   delta_chunk_state   a row's chunks one after the other, heads and tiles of 16 value columns side by side: U and the state
 //                       every chunk starts from; the row's end state into its slot
 //   delta_chunk_out     all chunks side by side: O
+//
+// Gated linear attention, S_i = diag(a_i) S_(i-1) + k_i v_i^T, o_i = S_i^T q_i, with a decay per key channel: with b_i the sums of
+// the logarithms per channel up to i,
+//     O = Q' S_0 + P V,   Q'_i = q_i exp(b_i),   P_ij = sum_d q_id k_jd exp(b_id - b_jd) for j <= i
+//     S_end = diag(exp(b_n)) S_0 + sum_j (k_j exp(b_n - b_j)) v_j^T
+// No exponent is positive: entries of P between two blocks of 16 tokens take the sums at the later block's start as reference,
+// those within a block are evaluated one by one.
+//   linear_chunk_local  all chunks side by side, from the projected rows: b, Q', P, the chunk's own sum over k v^T, v in float32
+//   linear_chunk_fold   per state entry along a row's chunks: the state every chunk starts from, the end state into the slot
+//   delta_chunk_out     as above, with Q' and v in place of q and U
+//
 // A row's chunks are counted from its first token of the step; chunk c of row r is number row_start[r] / 64 + r + c of the
 // step (distinct for all chunks; some numbers stay unused).
 #include "common.cuh"
@@ -36,6 +49,22 @@ struct DeltaChunkParams {
     float* s0;                      // [chunk numbers, H, dim, vdim]
     float* out;                     // [T, H, vdim]
     int rows, H, KH, dim, vdim;
+};
+
+template <typename T> struct LinearChunkParams {
+    const T* in;                    // [tokens, ld]: q (H dim), k (H dim), v (H vdim) as projected
+    int64_t ld;
+    const float* z;                 // [tokens, ldz] the decays' pre-activations (H dim)
+    int64_t ldz;
+    const float* bias;              // [H dim]
+    float inv_tau, q_scale;
+    const int* row_start;
+    float* q;                       // [T, H, dim]: Q'
+    float* v;                       // [T, H, vdim]
+    float* p;                       // [T, H, DC]
+    float* s0;                      // [chunk numbers, H, dim, vdim]: the chunk's own sum
+    float* decay;                   // [chunk numbers, H, dim]
+    int rows, H, dim, vdim;
 };
 
 // The row and chunk of a chunk number, or false for an unused one.
@@ -316,7 +345,8 @@ __global__ void __launch_bounds__(256) delta_chunk_state_kernel(const DeltaChunk
     }
 }
 
-template <int DP>
+// SCALED: q already holds exp(b) (and b is not read)
+template <int DP, bool SCALED>
 __global__ void __launch_bounds__(256, 2) delta_chunk_out_kernel(const DeltaChunkParams p) {
     constexpr int LD = DP + DC_PAD, LO = DC_OT + DC_PAD, LA = DC + DC_PAD;
     extern __shared__ __align__(16) float sm[];
@@ -349,7 +379,7 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_out_kernel(const DeltaChun
         else *reinterpret_cast<float4*>(sP + i * LA + j) = zero;
     }
     asm volatile("cp.async.commit_group;\n" ::);
-    if (tid < DC) sb[tid] = p.b[(int64_t)(first + min(tid, n - 1)) * p.H + h];
+    if (!SCALED && tid < DC) sb[tid] = p.b[(int64_t)(first + min(tid, n - 1)) * p.H + h];
     asm volatile("cp.async.wait_group 0;\n" ::);
     __syncthreads();
     const int tx = tid & 15, ty = tid >> 4;             // rows ty + 16 ii, columns 4 tx .. 4 tx + 3
@@ -370,10 +400,12 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_out_kernel(const DeltaChun
             axpy(q4.x, s[0], acc[ii]); axpy(q4.y, s[1], acc[ii]); axpy(q4.z, s[2], acc[ii]); axpy(q4.w, s[3], acc[ii]);
         }
     }
+    if (!SCALED) {
 #pragma unroll
-    for (int ii = 0; ii < 4; ++ii) {
-        const float g = expf(sb[ty + 16 * ii]);
-        acc[ii] = make_float4(acc[ii].x * g, acc[ii].y * g, acc[ii].z * g, acc[ii].w * g);
+        for (int ii = 0; ii < 4; ++ii) {
+            const float g = expf(sb[ty + 16 * ii]);
+            acc[ii] = make_float4(acc[ii].x * g, acc[ii].y * g, acc[ii].z * g, acc[ii].w * g);
+        }
     }
 #pragma unroll
     for (int jb = 0; jb < 4; ++jb) {                    // blocks of 16 keys; rows before the block see none of it
@@ -406,7 +438,7 @@ template <int DP> static int launch_delta_chunk(const DeltaChunkParams& p, int i
     if (!configured.seen()) {
         cudaError_t e = cudaFuncSetAttribute(delta_chunk_solve_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)solve);
         if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_chunk_state_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)walk);
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_chunk_out_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)out);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_chunk_out_kernel<DP, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)out);
         if (e != cudaSuccess) return (int)e;
         configured.mark();
     }
@@ -414,7 +446,257 @@ template <int DP> static int launch_delta_chunk(const DeltaChunkParams& p, int i
     if (rc) return rc;
     rc = acorn_launch(delta_chunk_state_kernel<DP>, dim3((p.vdim + DC_VT - 1) / DC_VT, p.H, p.rows), dim3(256), walk, stream, p);
     if (rc) return rc;
-    return acorn_launch(delta_chunk_out_kernel<DP>, dim3(ids, p.H, (p.vdim + DC_OT - 1) / DC_OT), dim3(256), out, stream, p);
+    return acorn_launch(delta_chunk_out_kernel<DP, false>, dim3(ids, p.H, (p.vdim + DC_OT - 1) / DC_OT), dim3(256), out, stream, p);
+}
+
+// ---------------------------------------------------------------- gated linear attention
+
+__device__ __forceinline__ float dc_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+
+template <typename T, int DP>
+__global__ void __launch_bounds__(256) linear_chunk_local_kernel(const LinearChunkParams<T> p) {
+    constexpr int LD = DP + DC_PAD, LO = DC_OT + DC_PAD, DQ = DP / 4;
+    extern __shared__ __align__(16) float sm[];
+    float* sQ = sm;                                     // [DC][LD]
+    float* sK = sQ + DC * LD;                           // [DC][LD]
+    float* sB = sK + DC * LD;                           // [DC][LD] sums of the logarithms (to base 2)
+    float* sR = sB + DC * LD;                           // [48][LD] keys of the blocks before one, at its reference
+    float* sV = sR + 48 * LD;                           // [DC][LO]
+    pdl_wait();
+    pdl_trigger();
+    const int h = blockIdx.y, tid = threadIdx.x;
+    int r, first, n;
+    if (!chunk_of(blockIdx.x, p.row_start, p.rows, r, first, n)) return;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    const int Hd = p.H * p.dim;
+    const float to_log2 = -1.4426950408889634f * p.inv_tau;
+    for (int e = tid; e < DC * DQ; e += 256) {
+        const int i = e / DQ, c = (e % DQ) * 4, at = i * LD + c;
+        float4 q = zero, k = zero, l = zero;
+        if (i < n && c < p.dim) {
+            const T* row = p.in + (int64_t)(first + i) * p.ld + h * p.dim + c;
+            q = Vec4<T>::load(row);
+            k = Vec4<T>::load(row + Hd);
+            const float4 z = *reinterpret_cast<const float4*>(p.z + (int64_t)(first + i) * p.ldz + h * p.dim + c);
+            const float4 b = *reinterpret_cast<const float4*>(p.bias + h * p.dim + c);
+            q = make_float4(q.x * p.q_scale, q.y * p.q_scale, q.z * p.q_scale, q.w * p.q_scale);
+            l = make_float4(dc_softplus(-(z.x + b.x)) * to_log2, dc_softplus(-(z.y + b.y)) * to_log2,
+                            dc_softplus(-(z.z + b.z)) * to_log2, dc_softplus(-(z.w + b.w)) * to_log2);
+        }
+        *reinterpret_cast<float4*>(sQ + at) = q;
+        *reinterpret_cast<float4*>(sK + at) = k;
+        *reinterpret_cast<float4*>(sB + at) = l;
+    }
+    __syncthreads();
+    for (int e = tid; e < 4 * DP; e += 256) {           // sums within blocks of 16 tokens, then over the blocks before
+        float run = 0.f;
+        float* col = sB + (e / DP) * 16 * LD + e % DP;
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            run += col[i * LD];
+            col[i * LD] = run;
+        }
+    }
+    __syncthreads();
+    float before[(4 * DP + 255) / 256];
+#pragma unroll
+    for (int m = 0; m < (4 * DP + 255) / 256; ++m) {
+        const int e = tid + 256 * m;
+        before[m] = 0.f;
+        if (e < 4 * DP)
+            for (int s = 0; s < e / DP; ++s) before[m] += sB[(16 * s + 15) * LD + e % DP];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int m = 0; m < (4 * DP + 255) / 256; ++m) {
+        const int e = tid + 256 * m;
+        if (e < 4 * DP && e >= DP)
+#pragma unroll
+            for (int i = 0; i < 16; ++i) sB[((e / DP) * 16 + i) * LD + e % DP] += before[m];
+    }
+    __syncthreads();
+    auto exp4 = [](const float4& a, const float4& b) -> float4 {       // 2^(a - b)
+        return make_float4(exp2f(a.x - b.x), exp2f(a.y - b.y), exp2f(a.z - b.z), exp2f(a.w - b.w));
+    };
+    auto mul4 = [](const float4& a, const float4& b) -> float4 { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); };
+    // entries within blocks of 16 tokens
+    const int tx = tid & 15, ty = tid >> 4;
+    float* P = p.p + ((int64_t)first * p.H + h) * DC;
+    const int64_t ldp = (int64_t)p.H * DC;
+#pragma unroll
+    for (int I = 0; I < 4; ++I) {
+        const int i = 16 * I + ty, j = 16 * I + tx;
+        float s = 0.f;
+        if (tx <= ty) {
+#pragma unroll 4
+            for (int d = 0; d < DP; d += 4) {
+                const float4 q = *reinterpret_cast<const float4*>(sQ + i * LD + d), k = *reinterpret_cast<const float4*>(sK + j * LD + d);
+                const float4 bi = *reinterpret_cast<const float4*>(sB + i * LD + d), bj = *reinterpret_cast<const float4*>(sB + j * LD + d);
+                s = dot4(mul4(q, k), exp4(bi, bj), s);
+            }
+        }
+        if (i < n) P[i * ldp + j] = s;
+    }
+    __syncthreads();
+    // Q' to memory; in shared memory q at its block's reference
+    for (int e = tid; e < DC * DQ; e += 256) {
+        const int i = e / DQ, c = (e % DQ) * 4, at = i * LD + c;
+        const float4 q = *reinterpret_cast<const float4*>(sQ + at), b = *reinterpret_cast<const float4*>(sB + at);
+        if (i < n && c < p.dim) *reinterpret_cast<float4*>(p.q + ((int64_t)(first + i) * p.H + h) * p.dim + c) = mul4(q, exp4(b, zero));
+        if (i >= 16) *reinterpret_cast<float4*>(sQ + at) = mul4(q, exp4(b, *reinterpret_cast<const float4*>(sB + ((i & ~15) - 1) * LD + c)));
+    }
+    if (tid < DQ && 4 * tid < p.dim)
+        *reinterpret_cast<float4*>(p.decay + ((int64_t)blockIdx.x * p.H + h) * p.dim + 4 * tid) =
+            exp4(*reinterpret_cast<const float4*>(sB + (DC - 1) * LD + 4 * tid), zero);
+#pragma unroll
+    for (int I = 1; I < 4; ++I) {                       // entries against the blocks before
+        for (int e = tid; e < 16 * I * DQ; e += 256) {
+            const int j = e / DQ, c = (e % DQ) * 4;
+            *reinterpret_cast<float4*>(sR + j * LD + c) =
+                mul4(*reinterpret_cast<const float4*>(sK + j * LD + c),
+                     exp4(*reinterpret_cast<const float4*>(sB + (16 * I - 1) * LD + c), *reinterpret_cast<const float4*>(sB + j * LD + c)));
+        }
+        __syncthreads();
+        const int i = 16 * I + ty;
+        float s[3] = {0.f, 0.f, 0.f};
+#pragma unroll 4
+        for (int d = 0; d < DP; d += 4) {
+            const float4 q = *reinterpret_cast<const float4*>(sQ + i * LD + d);
+#pragma unroll
+            for (int J = 0; J < I; ++J) s[J] = dot4(q, *reinterpret_cast<const float4*>(sR + (16 * J + tx) * LD + d), s[J]);
+        }
+        if (i < n)
+#pragma unroll
+            for (int J = 0; J < I; ++J) P[i * ldp + 16 * J + tx] = s[J];
+        __syncthreads();
+    }
+    // the keys at the chunk's end, and their sum with the values
+    for (int e = tid; e < DC * DQ; e += 256) {
+        const int at = (e / DQ) * LD + (e % DQ) * 4;
+        *reinterpret_cast<float4*>(sK + at) = mul4(*reinterpret_cast<const float4*>(sK + at),
+                                                   exp4(*reinterpret_cast<const float4*>(sB + (DC - 1) * LD + (e % DQ) * 4),
+                                                        *reinterpret_cast<const float4*>(sB + at)));
+    }
+    constexpr int ND = DP / 64 > 0 ? DP / 64 : 1;       // groups of 4 key channels a thread
+    for (int v0 = 0; v0 < p.vdim; v0 += DC_OT) {
+        for (int e = tid; e < DC * (DC_OT / 4); e += 256) {
+            const int j = e / (DC_OT / 4), c = (e % (DC_OT / 4)) * 4;
+            float4 v = zero;
+            if (j < n && v0 + c < p.vdim) {
+                v = Vec4<T>::load(p.in + (int64_t)(first + j) * p.ld + 2 * Hd + h * p.vdim + v0 + c);
+                *reinterpret_cast<float4*>(p.v + ((int64_t)(first + j) * p.H + h) * p.vdim + v0 + c) = v;
+            }
+            *reinterpret_cast<float4*>(sV + j * LO + c) = v;
+        }
+        __syncthreads();
+        float4 acc[ND][4];
+#pragma unroll
+        for (int m = 0; m < ND; ++m)
+#pragma unroll
+            for (int q = 0; q < 4; ++q) acc[m][q] = zero;
+        if (4 * ty < DP) {
+#pragma unroll 4
+            for (int j = 0; j < DC; ++j) {
+                const float4 v = *reinterpret_cast<const float4*>(sV + j * LO + 4 * tx);
+#pragma unroll
+                for (int m = 0; m < ND; ++m) {
+                    const float4 k = *reinterpret_cast<const float4*>(sK + j * LD + 4 * ty + 64 * m);
+                    const float kk[4] = {k.x, k.y, k.z, k.w};
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) {
+                        acc[m][q].x = fmaf(kk[q], v.x, acc[m][q].x); acc[m][q].y = fmaf(kk[q], v.y, acc[m][q].y);
+                        acc[m][q].z = fmaf(kk[q], v.z, acc[m][q].z); acc[m][q].w = fmaf(kk[q], v.w, acc[m][q].w);
+                    }
+                }
+            }
+            float* E = p.s0 + ((int64_t)blockIdx.x * p.H + h) * p.dim * p.vdim;
+#pragma unroll
+            for (int m = 0; m < ND; ++m)
+#pragma unroll
+                for (int q = 0; q < 4; ++q) {
+                    const int d = 4 * ty + 64 * m + q;
+                    if (d < p.dim && v0 + 4 * tx < p.vdim) *reinterpret_cast<float4*>(E + (int64_t)d * p.vdim + v0 + 4 * tx) = acc[m][q];
+                }
+        }
+        __syncthreads();
+    }
+}
+
+// A thread four value columns of a key channel's state, along a row's chunks; the chunks' sums are fetched a few ahead.
+__global__ void linear_chunk_fold_kernel(float* __restrict__ state, int64_t slot_stride, const int* __restrict__ row_start,
+                                         const int* __restrict__ row_slot, float* __restrict__ s0, const float* __restrict__ decay,
+                                         int H, int dim, int vdim) {
+    pdl_wait();
+    pdl_trigger();
+    const int r = blockIdx.z, h = blockIdx.y;
+    const int per = dim * (vdim / 4), e = blockIdx.x * blockDim.x + threadIdx.x;
+    if (e >= per) return;
+    const int d = e / (vdim / 4);
+    const int start = row_start[r], chunks = (row_start[r + 1] - start + DC - 1) / DC, id0 = start / DC + r;
+    float4* slot = reinterpret_cast<float4*>(state + (int64_t)row_slot[r] * slot_stride + (int64_t)h * dim * vdim) + e;
+    float4* E = reinterpret_cast<float4*>(s0 + ((int64_t)id0 * H + h) * dim * vdim) + e;
+    const float* a = decay + ((int64_t)id0 * H + h) * dim + d;
+    const int64_t step = (int64_t)H * dim * vdim / 4;
+    float4 cur = *slot;
+    constexpr int AHEAD = 8;
+    for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
+        float4 x[AHEAD];
+        float f[AHEAD];
+#pragma unroll
+        for (int q = 0; q < AHEAD; ++q) {
+            const int c = min(c0 + q, chunks - 1);
+            x[q] = E[c * step];
+            f[q] = a[(int64_t)c * H * dim];
+        }
+#pragma unroll
+        for (int q = 0; q < AHEAD; ++q) {
+            if (c0 + q >= chunks) break;
+            E[(c0 + q) * step] = cur;
+            cur = make_float4(fmaf(f[q], cur.x, x[q].x), fmaf(f[q], cur.y, x[q].y), fmaf(f[q], cur.z, x[q].z), fmaf(f[q], cur.w, x[q].w));
+        }
+    }
+    *slot = cur;
+}
+
+template <typename T, int DP> static int launch_linear_chunk(const LinearChunkParams<T>& p, const DeltaChunkParams& o, int ids, cudaStream_t stream) {
+    constexpr int LD = DP + DC_PAD, LO = DC_OT + DC_PAD;
+    const size_t local = (size_t)(3 * DC * LD + 48 * LD + DC * LO) * sizeof(float);
+    const size_t out = (size_t)(DC * LD + DP * LO + DC * LO + DC * (DC + DC_PAD)) * sizeof(float);
+    static AcornPerDevice configured;
+    if (!configured.seen()) {
+        cudaError_t e = cudaFuncSetAttribute(linear_chunk_local_kernel<T, DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)local);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(delta_chunk_out_kernel<DP, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)out);
+        if (e != cudaSuccess) return (int)e;
+        configured.mark();
+    }
+    int rc = acorn_launch(linear_chunk_local_kernel<T, DP>, dim3(ids, p.H), dim3(256), local, stream, p);
+    if (rc) return rc;
+    rc = acorn_launch(linear_chunk_fold_kernel, dim3((p.dim * (p.vdim / 4) + 255) / 256, p.H, p.rows), dim3(256), 0, stream, o.state,
+                      o.slot_stride, o.row_start, o.row_slot, p.s0, (const float*)p.decay, p.H, p.dim, p.vdim);
+    if (rc) return rc;
+    return acorn_launch(delta_chunk_out_kernel<DP, true>, dim3(ids, p.H, (p.vdim + DC_OT - 1) / DC_OT), dim3(256), out, stream, o);
+}
+
+extern "C" int acorn_linear_chunk(const void* in, int64_t ld, const float* z, int64_t ldz, const float* bias, float inv_tau, float* state,
+                                  int64_t slot_stride, const int* row_start, const int* row_slot, float* q, float* v, float* pp, float* s0,
+                                  float* decay, float* out, int tokens, int rows, int H, int dim, int vdim, int dtype, cudaStream_t stream) {
+    if (tokens <= 0 || rows <= 0) return 0;
+    const uintptr_t all = (uintptr_t)z | (uintptr_t)bias | (uintptr_t)q | (uintptr_t)v | (uintptr_t)s0 | (uintptr_t)out | (uintptr_t)state | (uintptr_t)decay;
+    if (dim < 4 || dim > 128 || dim % 4 || vdim < 4 || vdim % 4 || H < 1 || H > 65535 || rows > 65535 || (all & 15) || ld % 4 || ldz % 4 ||
+        slot_stride % 4 || ((uintptr_t)in & (dtype == ACORN_DTYPE_BF16 ? 7 : 15)))
+        return ACORN_ERR_UNSUPPORTED;
+    const DeltaChunkParams o = {q, nullptr, nullptr, nullptr, nullptr, state, slot_stride, row_start, row_slot, nullptr, v, pp, nullptr, s0, out,
+                                rows, H, H, dim, vdim};
+    const int ids = tokens / DC + rows;
+    ACORN_DISPATCH_DTYPE(dtype, T, {
+        LinearChunkParams<T> p;
+        p.in = (const T*)in; p.ld = ld; p.z = z; p.ldz = ldz; p.bias = bias; p.inv_tau = inv_tau; p.q_scale = (float)(1.0 / sqrt((double)dim));
+        p.row_start = row_start; p.q = q; p.v = v; p.p = pp; p.s0 = s0; p.decay = decay; p.rows = rows; p.H = H; p.dim = dim; p.vdim = vdim;
+        if (dim <= 32) return launch_linear_chunk<T, 32>(p, o, ids, stream);
+        if (dim <= 64) return launch_linear_chunk<T, 64>(p, o, ids, stream);
+        return launch_linear_chunk<T, 128>(p, o, ids, stream);
+    });
+    return ACORN_ERR_UNSUPPORTED;
 }
 
 extern "C" int acorn_delta_chunk_supported(int dim, int vdim) { return dim >= 4 && dim <= 128 && dim % 4 == 0 && vdim >= 4 && vdim % 4 == 0; }

@@ -174,6 +174,8 @@ class _Sigs:
     acorn_delta_chunk = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p,
                          c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
     acorn_delta_chunk_supported = [c_int, c_int]
+    acorn_linear_chunk = [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_float, c_void_p, c_int64, c_void_p, c_void_p, c_void_p,
+                          c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
     acorn_delta_chunk_ids = [c_int, c_int]
     acorn_linear_heads_prep = [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p,
                                c_int, c_int, c_int, c_int, c_int, c_void_p]
@@ -1539,6 +1541,37 @@ def delta_chunk(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.T
                                 state.data_ptr() + 4 * int(state_off), state.stride(0), row_start.data_ptr(), row_slot.data_ptr(),
                                 w.data_ptr(), u.data_ptr(), p.data_ptr(), b.data_ptr(), s0.data_ptr(), out.data_ptr(), T, num_rows, H,
                                 KH, dim, vdim, _stream()), "delta_chunk")
+    return out
+
+
+def linear_chunk_ok(longest_row: int, proj: torch.Tensor, z32: torch.Tensor, state: torch.Tensor, state_off: int, num_rows: int,
+                    heads: int, dim: int, vdim: int) -> bool:
+    """Whether a step of these rows takes ``linear_chunk``: a row long enough to pay for it, and sizes the kernels know."""
+    return (longest_row >= DELTA_CHUNK_MIN_ROW and bool(lib().acorn_delta_chunk_supported(dim, vdim)) and state_off % 4 == 0
+            and state.stride(0) % 4 == 0 and proj.stride(0) % 4 == 0 and proj.data_ptr() % (8 if proj.dtype == torch.bfloat16 else 16) == 0
+            and z32.stride(0) % 4 == 0
+            and 4 * lib().acorn_delta_chunk_ids(proj.shape[0], num_rows) * heads * dim * vdim <= DELTA_CHUNK_SCRATCH_BYTES)
+
+
+def linear_chunk(proj: torch.Tensor, z32: torch.Tensor, bias32: torch.Tensor, tau: float, state: torch.Tensor, row_start: torch.Tensor,
+                 row_slot: torch.Tensor, num_rows: int, heads: int, dim: int, vdim: int, state_off: int = 0) -> torch.Tensor:
+    """Gated linear attention over chunks of 64 tokens, from the projected rows ``[q | k | v | ...]`` (see ``linear_heads_prep``):
+    float32 o [T, H, vdim]; the states in the rows' slots are updated in place."""
+    _rows2(proj, "proj")
+    _rows2(z32, "z", torch.float32)
+    _check(bias32, "bias", torch.float32, 1)
+    _check(state, "state", torch.float32, 2)
+    T = proj.shape[0]
+    if proj.shape[1] < heads * (2 * dim + vdim) or z32.shape != (T, heads * dim) or state.shape[1] < state_off + heads * dim * vdim:
+        raise KernelError(f"linear_chunk: proj {tuple(proj.shape)}, z {tuple(z32.shape)}, state {tuple(state.shape)} do not fit")
+    ids = lib().acorn_delta_chunk_ids(T, num_rows)
+    f = lambda *shape: torch.empty(shape, dtype=torch.float32, device=proj.device)
+    q, v, p, out = f(T, heads, dim), f(T, heads, vdim), f(T, heads, 64), f(T, heads, vdim)
+    s0, decay = f(ids, heads, dim, vdim), f(ids, heads, dim)
+    _ok(lib().acorn_linear_chunk(proj.data_ptr(), proj.stride(0), z32.data_ptr(), z32.stride(0), bias32.data_ptr(), 1.0 / float(tau),
+                                 state.data_ptr() + 4 * int(state_off), state.stride(0), row_start.data_ptr(), row_slot.data_ptr(),
+                                 q.data_ptr(), v.data_ptr(), p.data_ptr(), s0.data_ptr(), decay.data_ptr(), out.data_ptr(), T, num_rows,
+                                 heads, dim, vdim, dtype_code(proj.dtype), _stream()), "linear_chunk")
     return out
 
 

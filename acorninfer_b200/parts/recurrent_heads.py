@@ -14,7 +14,8 @@ its root mean square, times one weight of head size, times silu of a gate, and t
 Everything from the activations (the projections of the second) on is float32, and so is the state: S of every head, and
 behind it the convolution's last ``taps - 1`` inputs, in the request's slot (one float32 vector from ``state_base`` on).
 All projections of h are one matrix product.  Steps of single tokens run recurrence, norm and gate in one kernel
-(``ops.recurrent_step``); longer rows run the recurrence over a row's tokens.  The one host-side value of a step that is
+(``ops.recurrent_step``); steps with rows of ``ops.DELTA_CHUNK_MIN_ROW`` tokens run over chunks of tokens (``ops.delta_chunk``,
+``ops.linear_chunk``); others walk their rows' tokens.  The one host-side value of a step that is
 read is its longest row, which is 1 in every captured step.
 """
 
@@ -165,7 +166,12 @@ class GatedLinearAttention(_HeadsMixer):
         if self._steps(inputs, cache, (proj, gate, out)) and (self.H * self.dim) % 2 == 0 and z.stride(0) % 4 == 0:
             return ops.recurrent_step(cache.state, self.state_base, inputs.row_slot, gate, self.norm32, self.eps, out, self.H,
                                       self.dim, self.vdim, out_scale, linear=(proj, z, self.a2_bias32, self.tau))
-        q, k, v, alpha = ops.linear_heads_prep(proj, z, self.a2_bias32, self.tau, self.H, self.dim, self.vdim)
-        o = ops.delta_rule(q, k, v, None, alpha, cache.state, inputs.row_start, inputs.row_slot, inputs.num_rows,
-                           longest_row=inputs.plan.max_q_len, state_off=self.state_base)
+        longest = inputs.plan.max_q_len
+        if ops.linear_chunk_ok(longest, proj, z, cache.state, self.state_base, inputs.num_rows, self.H, self.dim, self.vdim):
+            o = ops.linear_chunk(proj, z, self.a2_bias32, self.tau, cache.state, inputs.row_start, inputs.row_slot, inputs.num_rows,
+                                 self.H, self.dim, self.vdim, state_off=self.state_base)
+        else:
+            q, k, v, alpha = ops.linear_heads_prep(proj, z, self.a2_bias32, self.tau, self.H, self.dim, self.vdim)
+            o = ops.delta_rule(q, k, v, None, alpha, cache.state, inputs.row_start, inputs.row_slot, inputs.num_rows,
+                               longest_row=longest, state_off=self.state_base)
         return ops.gated_norm(o.view(o.shape[0], -1), gate, self.norm_heads32, self.eps, self.H, False, out, out_scale, silu=True)

@@ -668,7 +668,8 @@ def test_delta_chunks(H, KH, dim, vdim):
 @pytest.mark.parametrize("dtype,tol", [(torch.float32, 2e-5), (torch.bfloat16, 2e-2)])
 @pytest.mark.parametrize("H,dim,vdim,tau", [(3, 5, 7, 1.0), (4, 32, 64, 16.0), (2, 128, 128, 4.0), (2, 140, 20, 8.0), (8, 64, 128, 16.0), (1, 16, 200, 2.0)])
 def test_linear_attention_across_steps(H, dim, vdim, tau, dtype, tol):
-    """Gated linear attention over a long row (cut into segments), a short one and a single token, then tokens one by one."""
+    """Gated linear attention over long rows (over chunks of tokens, or walked in segments), short ones and single tokens in
+    one step, then tokens one by one; decays from none to those that leave nothing between two tokens."""
     o = ops()
     g = torch.Generator().manual_seed(dim + vdim)
     Hd, Hv, eps = H * dim, H * vdim, 1e-5
@@ -676,11 +677,14 @@ def test_linear_attention_across_steps(H, dim, vdim, tau, dtype, tol):
     width = gate_col + Hv + (-Hv) % 8
     S_size, s_off = Hd * vdim, 8
     norm_w, bias = _rand(g, vdim), _rand(g, Hd)
-    for lens, slots in (([400], [2]), ([190, 1, 33], [4, 0, 1])):
+    took = set()
+    for lens, slots, chunks in (([400], [2], False), ([400], [2], True), ([190, 1, 33], [4, 0, 1], True), ([64, 65, 1, 129, 63], [4, 0, 1, 5, 2], True)):
         tail = 4
         state = _rand(g, 6, s_off + S_size + (-S_size) % 4, scale=0.5)
         rows = [_rand(g, n + tail, width, dtype=dtype) for n in lens]
         zs = [_rand(g, n + tail, Hd, scale=2.0) + 2.0 for n in lens]
+        zs[0][20:23] -= 400.0
+        zs[0][::7] += 30.0
         sd = state.to(DEV)
         outs = [torch.empty(n + tail, Hv) for n in lens]
 
@@ -694,8 +698,12 @@ def test_linear_attention_across_steps(H, dim, vdim, tau, dtype, tol):
             if max(n) == 1 and (Hd % 2 == 0) and o.recurrent_step_ok(dim, vdim, (sd, sd.stride(0), s_off), (x, gate, y)):
                 o.recurrent_step(sd, s_off, slot_t, gate, norm_w.to(DEV), eps, y, H, dim, vdim, 1.3, linear=(x, z, bias.to(DEV), tau))
             else:
-                q, k, v, al = o.linear_heads_prep(x, z, bias.to(DEV), tau, H, dim, vdim)
-                r = o.delta_rule(q, k, v, None, al, sd, starts, slot_t, len(n), longest_row=max(n), state_off=s_off)
+                if chunks and o.linear_chunk_ok(max(n), x, z, sd, s_off, len(n), H, dim, vdim):
+                    took.add("chunks")
+                    r = o.linear_chunk(x, z, bias.to(DEV), tau, sd, starts, slot_t, len(n), H, dim, vdim, state_off=s_off)
+                else:
+                    q, k, v, al = o.linear_heads_prep(x, z, bias.to(DEV), tau, H, dim, vdim)
+                    r = o.delta_rule(q, k, v, None, al, sd, starts, slot_t, len(n), longest_row=max(n), state_off=s_off)
                 o.gated_norm(r.view(x.shape[0], -1), gate, norm_w.repeat(H).to(DEV), eps, H, False, y, 1.3, silu=True)
             return torch.split(y.float().cpu(), n)
 
@@ -717,6 +725,7 @@ def test_linear_attention_across_steps(H, dim, vdim, tau, dtype, tol):
             assert (sd[slots[i], s_off:s_off + S_size].double().cpu().view(H, dim, vdim) - S).abs().max() < 2e-5 * max(1.0, float(S.abs().max()))
         untouched = [s for s in range(6) if s not in slots]
         assert torch.equal(sd[untouched].cpu(), state[untouched]) and torch.equal(sd[:, :s_off].cpu(), state[:, :s_off])
+    assert took or dim % 4 or vdim % 4 or dim > 128
 
 
 def test_sink_at_zero_where_one_key_decides():
