@@ -39,19 +39,31 @@ template <typename T> struct HyperParams {
 template <typename T, int N, int NV>
 __global__ void __launch_bounds__(NV == 4 ? 256 : 512) hyper_norm_vec_kernel(const HyperParams<T> p) {
     __shared__ float scratch[32];
-    pdl_wait();
-    pdl_trigger();
     const int r = blockIdx.x;
-    const int64_t row = p.row_idx ? p.row_idx[r] : r;
     const int n4 = p.H >> 2;
     int at[NV];
     bool in[NV];
-    float4 x[N][NV];
+    float4 x[N][NV], nw[NV];
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
         const int i = threadIdx.x + k * blockDim.x;
         in[k] = i < n4;
         at[k] = 4 * min(i, n4 - 1);
+        if (NV <= 2 && p.out) nw[k] = *reinterpret_cast<const float4*>(p.w + at[k]);
+    }
+    float m[N][N], put[N], take[N];                     // (what the model fixes is fetched before the kernel ahead has finished)
+#pragma unroll
+    for (int t = 0; t < N; ++t) {
+        put[t] = p.a || p.y ? p.scale * p.put[t] : 0.f;
+        take[t] = p.take ? p.take[t] : 1.f;
+#pragma unroll
+        for (int s = 0; s < N; ++s) m[s][t] = p.a || p.y ? p.mix[s * N + t] : 0.f;
+    }
+    pdl_wait();
+    pdl_trigger();
+    const int64_t row = p.row_idx ? p.row_idx[r] : r;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
 #pragma unroll
         for (int s = 0; s < N; ++s) x[s][k] = *reinterpret_cast<const float4*>(p.x + s * p.x_stride + row * p.H + at[k]);
     }
@@ -74,13 +86,6 @@ __global__ void __launch_bounds__(NV == 4 ? 256 : 512) hyper_norm_vec_kernel(con
                     d[k].z = fmaf(f, e.z, d[k].z); d[k].w = fmaf(f, e.w, d[k].w);
                 }
             }
-        }
-        float m[N][N], put[N];
-#pragma unroll
-        for (int t = 0; t < N; ++t) {
-            put[t] = p.scale * p.put[t];
-#pragma unroll
-            for (int s = 0; s < N; ++s) m[s][t] = p.mix[s * N + t];
         }
 #pragma unroll
         for (int k = 0; k < NV; ++k) {
@@ -113,7 +118,7 @@ __global__ void __launch_bounds__(NV == 4 ? 256 : 512) hyper_norm_vec_kernel(con
         u[k] = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
         for (int t = 0; t < N; ++t) {
-            const float f = p.take ? p.take[t] : 1.f;
+            const float f = take[t];
             u[k].x = fmaf(f, x[t][k].x, u[k].x); u[k].y = fmaf(f, x[t][k].y, u[k].y);
             u[k].z = fmaf(f, x[t][k].z, u[k].z); u[k].w = fmaf(f, x[t][k].w, u[k].w);
         }
@@ -123,7 +128,7 @@ __global__ void __launch_bounds__(NV == 4 ? 256 : 512) hyper_norm_vec_kernel(con
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
         if (!in[k]) continue;
-        const float4 w = *reinterpret_cast<const float4*>(p.w + at[k]);
+        const float4 w = NV <= 2 ? nw[k] : *reinterpret_cast<const float4*>(p.w + at[k]);
         Vec4<T>::store(p.out + (int64_t)r * p.H + at[k],
                        make_float4(u[k].x * inv * w.x, u[k].y * inv * w.y, u[k].z * inv * w.z, u[k].w * inv * w.w));
     }

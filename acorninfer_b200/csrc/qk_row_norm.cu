@@ -47,114 +47,124 @@ __device__ __forceinline__ void rown_pair_sum(float& a, float& b, float2* scratc
     b = warp_sum(t.y);
 }
 
-// Four channels a lane; a block walks `tpt` consecutive tokens of the step and carries a lane's inputs before the current
-// token along in registers while it stays within a row.  VPT vectors a thread.
-template <typename T, int TAPS, int VPT>
-__global__ void __launch_bounds__(512) qk_row_norm_vec_kernel(const RowNormParams<T> p, int tpt) {
-    __shared__ float2 scratch[2][32];
-    pdl_wait();
-    pdl_trigger();
-    constexpr int PAST = TAPS > 1 ? TAPS - 1 : 1;
+// Four channels a lane, VPT such vectors a thread; a block takes TPT consecutive tokens of the step: their rows and those before
+// them are fetched at once, the convolved values wait in registers for the rows' norms.
+template <typename T, int TAPS, int VPT, int TPT>
+__global__ void __launch_bounds__(VPT == 1 ? 768 : 512) qk_row_norm_vec_kernel(const RowNormParams<T> p) {
+    __shared__ float sums[2 * TPT][32];
+    __shared__ float inv_s[2 * TPT];
+    constexpr int PAST = TAPS > 1 ? TAPS - 1 : 0;
     constexpr int WT = TAPS > 0 ? 4 * TAPS : 1;
     const int qv = p.nq * p.d / 4, kv = p.nkv * p.d / 4, nvec = qv + kv + p.nkv * p.dv / 4;
     const int channels = nvec * 4;
-    int chan[VPT], kind[VPT];                           // kind 0: q, 1: k, 2: v, 3: no vector
-    float4 b[VPT], past[VPT][PAST], raw[VPT];
-    float w[VPT][WT];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+    const int t0 = blockIdx.x * TPT;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-    const int t0 = blockIdx.x * tpt, t_end = min(p.tokens, t0 + tpt);
+    float4 x[VPT][TPT];
+    int chan[VPT], kind[VPT];                           // kind 0: q, 1: k, 2: v, 3: no vector
+    float sq[TPT], sk[TPT];
+#pragma unroll
+    for (int q = 0; q < TPT; ++q) sq[q] = sk[q] = 0.f;
 #pragma unroll
     for (int k = 0; k < VPT; ++k) {
         const int v = threadIdx.x + k * blockDim.x;
         kind[k] = v >= nvec ? 3 : (v >= qv + kv ? 2 : (v >= qv ? 1 : 0));
         chan[k] = 4 * min(v, nvec - 1);
-        b[k] = p.bias ? *reinterpret_cast<const float4*>(p.bias + chan[k]) : zero;
+    }
+    int row[TPT], i0[TPT];
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+        float w[WT];
+        const float4 b = p.bias ? *reinterpret_cast<const float4*>(p.bias + chan[k]) : zero;
 #pragma unroll
         for (int j = 0; j < TAPS; ++j) {
             const float4 u = *reinterpret_cast<const float4*>(p.conv_w + (int64_t)chan[k] * TAPS + 4 * j);
-            w[k][4 * j] = u.x; w[k][4 * j + 1] = u.y; w[k][4 * j + 2] = u.z; w[k][4 * j + 3] = u.w;
+            w[4 * j] = u.x; w[4 * j + 1] = u.y; w[4 * j + 2] = u.z; w[4 * j + 3] = u.w;
         }
-        raw[k] = Vec4<T>::load(p.proj + (int64_t)t0 * p.ld + chan[k]);
+        if (k == 0) {
+            pdl_wait();
+            pdl_trigger();
 #pragma unroll
-        for (int j = 0; j < PAST; ++j) past[k][j] = zero;
-    }
-    for (int t = t0; t < t_end; ++t) {
-        const int r = p.token_row[t];
-        const int pos = p.positions[t];
-        float4 x[VPT];
-        int i0 = 0;
-        bool fresh = false, shift = false;
-        float* cstate = nullptr;
-        if constexpr (TAPS > 1) {
-            const int first = p.row_start[r];
-            i0 = t - first;
-            fresh = t == t0 || i0 == 0;
-            if (fresh) {
-                cstate = p.state + (int64_t)p.row_slot[r] * p.slot_stride + p.conv_off;
-                shift = p.update_single && p.row_start[r + 1] - first == 1;
+            for (int q = 0; q < TPT; ++q) {
+                const int t = min(t0 + q, p.tokens - 1);
+                row[q] = p.token_row[t];
+                i0[q] = PAST ? t - p.row_start[row[q]] : 0;               // the token's index within its row
             }
         }
-        float sq = 0.f, sk = 0.f;
+        float4 in[TPT + PAST];                          // inputs of tokens t0 - PAST .. t0 + TPT - 1
 #pragma unroll
-        for (int k = 0; k < VPT; ++k) {
-            const float4 own = make_float4(raw[k].x + b[k].x, raw[k].y + b[k].y, raw[k].z + b[k].z, raw[k].w + b[k].w);
-            x[k] = own;
+        for (int q = 0; q < TPT + PAST; ++q) {
+            const int t = min(max(t0 + q - PAST, 0), p.tokens - 1);
+            const float4 u = Vec4<T>::load(p.proj + (int64_t)t * p.ld + chan[k]);
+            in[q] = make_float4(u.x + b.x, u.y + b.y, u.z + b.z, u.w + b.w);
+        }
+#pragma unroll
+        for (int q = 0; q < TPT; ++q) {
+            float4 y = in[q + PAST];
             if constexpr (TAPS > 0) {
-                x[k] = zero;
-                if constexpr (TAPS > 1) {
-                    if (fresh) {
+                y = zero;
+                float* cstate = nullptr;
+                if constexpr (PAST > 0)
+                    if (i0[q] < PAST) cstate = p.state + (int64_t)p.row_slot[row[q]] * p.slot_stride + p.conv_off + chan[k];
+                float4 before[PAST > 0 ? PAST : 1];
 #pragma unroll
-                        for (int j = 0; j < TAPS - 1; ++j) {
-                            const int idx = i0 - (TAPS - 1) + j;          // input index within the row; negative: before the step
-                            if (idx >= 0) {
-                                const float4 u = Vec4<T>::load(p.proj + (int64_t)(t + idx - i0) * p.ld + chan[k]);
-                                past[k][j] = make_float4(u.x + b[k].x, u.y + b[k].y, u.z + b[k].z, u.w + b[k].w);
-                            } else {
-                                past[k][j] = *reinterpret_cast<const float4*>(cstate + (int64_t)(TAPS - 1 + idx) * channels + chan[k]);
-                            }
-                        }
-                        if (shift && kind[k] < 3) {                       // the row's only token: a lane alone reads and writes its channels
-#pragma unroll
-                            for (int j = 1; j < TAPS - 1; ++j)
-                                *reinterpret_cast<float4*>(cstate + (int64_t)(j - 1) * channels + chan[k]) = past[k][j];
-                            *reinterpret_cast<float4*>(cstate + (int64_t)(TAPS - 2) * channels + chan[k]) = own;
-                        }
-                    }
-#pragma unroll
-                    for (int j = 0; j < TAPS - 1; ++j) {
-                        x[k].x = fmaf(w[k][j], past[k][j].x, x[k].x);
-                        x[k].y = fmaf(w[k][TAPS + j], past[k][j].y, x[k].y);
-                        x[k].z = fmaf(w[k][2 * TAPS + j], past[k][j].z, x[k].z);
-                        x[k].w = fmaf(w[k][3 * TAPS + j], past[k][j].w, x[k].w);
-                    }
-#pragma unroll
-                    for (int j = 0; j < TAPS - 2; ++j) past[k][j] = past[k][j + 1];
-                    past[k][PAST - 1] = own;
+                for (int j = 0; j < PAST; ++j) {        // index within the row i0 - PAST + j; negative: before the step
+                    float4 u = in[q + j];
+                    if (i0[q] - PAST + j < 0) u = *reinterpret_cast<const float4*>(cstate + (int64_t)(i0[q] + j) * channels);
+                    before[j] = u;
+                    y.x = fmaf(w[j], u.x, y.x);
+                    y.y = fmaf(w[TAPS + j], u.y, y.y);
+                    y.z = fmaf(w[2 * TAPS + j], u.z, y.z);
+                    y.w = fmaf(w[3 * TAPS + j], u.w, y.w);
                 }
-                x[k].x = fmaf(w[k][TAPS - 1], own.x, x[k].x);
-                x[k].y = fmaf(w[k][2 * TAPS - 1], own.y, x[k].y);
-                x[k].z = fmaf(w[k][3 * TAPS - 1], own.z, x[k].z);
-                x[k].w = fmaf(w[k][4 * TAPS - 1], own.w, x[k].w);
-            }
-            const float ss = x[k].x * x[k].x + x[k].y * x[k].y + x[k].z * x[k].z + x[k].w * x[k].w;
-            if (kind[k] == 0) sq += ss;
-            if (kind[k] == 1) sk += ss;
-        }
-        if (t + 1 < t_end) {                                              // the next token's row, on its way during the sums
+                y.x = fmaf(w[TAPS - 1], in[q + PAST].x, y.x);
+                y.y = fmaf(w[2 * TAPS - 1], in[q + PAST].y, y.y);
+                y.z = fmaf(w[3 * TAPS - 1], in[q + PAST].z, y.z);
+                y.w = fmaf(w[4 * TAPS - 1], in[q + PAST].w, y.w);
+                if constexpr (PAST > 0) {
+                    // the row's only token: a lane alone reads and writes its channels
+                    if (p.update_single && kind[k] < 3 && i0[q] == 0 && t0 + q < p.tokens && p.row_start[row[q] + 1] - (t0 + q) == 1) {
 #pragma unroll
-            for (int k = 0; k < VPT; ++k) raw[k] = Vec4<T>::load(p.proj + (int64_t)(t + 1) * p.ld + chan[k]);
+                        for (int j = 1; j < PAST; ++j) *reinterpret_cast<float4*>(cstate + (int64_t)(j - 1) * channels) = before[j];
+                        *reinterpret_cast<float4*>(cstate + (int64_t)(PAST - 1) * channels) = in[q + PAST];
+                    }
+                }
+            }
+            x[k][q] = y;
+            const float ss = y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w;
+            if (kind[k] == 0) sq[q] += ss;
+            if (kind[k] == 1) sk[q] += ss;
         }
-        const int page = p.block_table[(int64_t)r * p.table_stride + (pos / p.P - p.page_base[r])];
-        rown_pair_sum(sq, sk, scratch[(t - t0) & 1]);
-        const float inv_q = rsqrtf(sq / p.q_count + p.eps), inv_k = rsqrtf(sk / p.k_count + p.eps);
+    }
+#pragma unroll
+    for (int q = 0; q < TPT; ++q) {
+        const float a = warp_sum(sq[q]), b = warp_sum(sk[q]);
+        if (lane == 0) {
+            sums[2 * q][warp] = a;
+            sums[2 * q + 1][warp] = b;
+        }
+    }
+    __syncthreads();
+    for (int e = warp; e < 2 * TPT; e += nwarps) {
+        const float total = warp_sum(lane < nwarps ? sums[e][lane] : 0.f);
+        if (lane == 0) inv_s[e] = rsqrtf(total / (e & 1 ? p.k_count : p.q_count) + p.eps);
+    }
+    __syncthreads();
+#pragma unroll
+    for (int q = 0; q < TPT; ++q) {
+        const int t = t0 + q;
+        if (t >= p.tokens) break;
+        const int pos = p.positions[t];
+        const int page = p.block_table[(int64_t)row[q] * p.table_stride + (pos / p.P - p.page_base[row[q]])];
 #pragma unroll
         for (int k = 0; k < VPT; ++k) {
             if (kind[k] == 3) continue;
+            float4 y = x[k][q];
             T* dst;
             if (kind[k] == 2) {
                 const int c = chan[k] - (p.nq + p.nkv) * p.d;
                 const int h = c / p.dv, i = c - h * p.dv;
-                x[k] = make_float4(x[k].x * p.v_scale, x[k].y * p.v_scale, x[k].z * p.v_scale, x[k].w * p.v_scale);
+                y = make_float4(y.x * p.v_scale, y.y * p.v_scale, y.z * p.v_scale, y.w * p.v_scale);
                 dst = p.v_pages + (((int64_t)page * p.nkv + h) * p.P + pos % p.P) * p.dv + i;
             } else {
                 const int c = kind[k] == 0 ? chan[k] : chan[k] - p.nq * p.d;
@@ -162,26 +172,26 @@ __global__ void __launch_bounds__(512) qk_row_norm_vec_kernel(const RowNormParam
                 const float* nw = kind[k] == 0 ? p.q_w : p.k_w;
                 if (nw) {
                     const float4 g = *reinterpret_cast<const float4*>(nw + c);
-                    const float inv = kind[k] == 0 ? inv_q : inv_k;
-                    x[k] = make_float4(x[k].x * inv * g.x, x[k].y * inv * g.y, x[k].z * inv * g.z, x[k].w * inv * g.w);
+                    const float inv = inv_s[2 * q + kind[k]];
+                    y = make_float4(y.x * inv * g.x, y.y * inv * g.y, y.z * inv * g.z, y.w * inv * g.w);
                 }
                 if (i < p.rot) {                                          // two whole pairs, or one where the rotated part ends between them
                     const float* cs = p.cos_sin + (int64_t)t * p.rot + (i >> 1);
                     const int half = p.rot >> 1;
                     const float c0 = cs[0], s0 = cs[half];
-                    const float e = x[k].x, f = x[k].y;
-                    x[k].x = e * c0 - f * s0;
-                    x[k].y = f * c0 + e * s0;
+                    const float e = y.x, f = y.y;
+                    y.x = e * c0 - f * s0;
+                    y.y = f * c0 + e * s0;
                     if (i + 2 < p.rot) {
                         const float c1 = cs[1], s1 = cs[half + 1];
-                        const float m = x[k].z, n = x[k].w;
-                        x[k].z = m * c1 - n * s1;
-                        x[k].w = n * c1 + m * s1;
+                        const float m = y.z, o = y.w;
+                        y.z = m * c1 - o * s1;
+                        y.w = o * c1 + m * s1;
                     }
                 }
                 dst = kind[k] == 0 ? p.q_out + (int64_t)t * p.ld_q + c : p.k_pages + (((int64_t)page * p.nkv + h) * p.P + pos % p.P) * p.d + i;
             }
-            Vec4<T>::store(dst, x[k]);
+            Vec4<T>::store(dst, y);
         }
     }
 }
@@ -254,12 +264,15 @@ __global__ void qk_row_norm_kernel(const RowNormParams<T> p) {
 
 template <typename T, int TAPS> static int launch_row_norm_vec(const RowNormParams<T>& p, int nvec, cudaStream_t stream) {
     const int tpt = p.tokens > 512 ? 4 : 1;             // a step of few tokens: a block a token
-    const dim3 grid((p.tokens + tpt - 1) / tpt);
-    const int vpt = nvec <= 384 ? 1 : (nvec <= 1024 ? 2 : 4);
-    const dim3 block(((nvec + vpt - 1) / vpt + 31) / 32 * 32);
-    if (vpt == 1) return acorn_launch(qk_row_norm_vec_kernel<T, TAPS, 1>, grid, block, 0, stream, p, tpt);
-    if (vpt == 2) return acorn_launch(qk_row_norm_vec_kernel<T, TAPS, 2>, grid, block, 0, stream, p, tpt);
-    return acorn_launch(qk_row_norm_vec_kernel<T, TAPS, 4>, grid, block, 0, stream, p, tpt);
+    const int vpt = nvec <= 768 ? 1 : (nvec <= 1024 ? 2 : 4);
+    const dim3 grid((p.tokens + tpt - 1) / tpt), block(((nvec + vpt - 1) / vpt + 31) / 32 * 32);
+    if (vpt == 1) {
+        if (tpt == 1) return acorn_launch(qk_row_norm_vec_kernel<T, TAPS, 1, 1>, grid, block, 0, stream, p);
+        return acorn_launch(qk_row_norm_vec_kernel<T, TAPS, 1, 4>, grid, block, 0, stream, p);
+    }
+    const dim3 one(p.tokens);
+    if (vpt == 2) return acorn_launch(qk_row_norm_vec_kernel<T, TAPS, 2, 1>, one, block, 0, stream, p);
+    return acorn_launch(qk_row_norm_vec_kernel<T, TAPS, 4, 1>, one, block, 0, stream, p);
 }
 
 template <typename T> static int launch_row_norm(const RowNormParams<T>& p, cudaStream_t stream) {

@@ -45,108 +45,100 @@ template <typename T> struct DeltaHeadsParams {
     int tokens, H, KH, dim, vdim, taps, update_single;
 };
 
-// Four channels a lane, 2^lph_log2 lanes a head; a lane walks tpt tokens and carries the inputs before the current one along.
-template <typename T, int TAPS>
-__global__ void delta_heads_prep_vec_kernel(const DeltaHeadsParams<T> p, int lph_log2, int tpt) {
-    pdl_wait();
-    pdl_trigger();
-    constexpr int PAST = TAPS > 1 ? TAPS - 1 : 1;
+// Four channels a lane, 2^lph_log2 lanes a head; a lane takes TPT consecutive tokens, whose inputs and those before them are
+// fetched at once.
+template <typename T, int TAPS, int TPT>
+__global__ void __launch_bounds__(256) delta_heads_prep_vec_kernel(const DeltaHeadsParams<T> p, int lph_log2) {
+    constexpr int PAST = TAPS > 1 ? TAPS - 1 : 0;
     const int heads = 2 * p.KH + p.H;
     const int64_t gid = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
     const int64_t item = gid >> lph_log2;
     const int l = (int)(gid & ((1 << lph_log2) - 1));
-    const int64_t chunks = ((int64_t)p.tokens + tpt - 1) / tpt;
+    const int64_t chunks = ((int64_t)p.tokens + TPT - 1) / TPT;
     const bool in_range = item < chunks * heads;
     const int64_t it = in_range ? item : 0;
-    const int64_t t_first = (it / heads) * tpt;
-    const int h = (int)(it % heads);
+    const int t0 = (int)(it / heads) * TPT;
+    const int h = (int)(it % heads), vh = h - 2 * p.KH;
     const bool is_v = h >= 2 * p.KH;
     const bool lane_on = in_range && 4 * l < (is_v ? p.vdim : p.dim);
     const int C = 2 * p.KH * p.dim + p.H * p.vdim;
-    const int chan = (is_v ? 2 * p.KH * p.dim + (h - 2 * p.KH) * p.vdim : h * p.dim) + 4 * l;
+    const int chan = lane_on ? (is_v ? 2 * p.KH * p.dim + vh * p.vdim : h * p.dim) + 4 * l : 0;      // idle lanes read channel 0
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
     float w[TAPS > 0 ? 4 * TAPS : 1];
-    if (lane_on) {
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) {
-            const float4 v = *reinterpret_cast<const float4*>(p.conv_w + (int64_t)chan * TAPS + 4 * j);
-            w[4 * j] = v.x; w[4 * j + 1] = v.y; w[4 * j + 2] = v.z; w[4 * j + 3] = v.w;
-        }
+    for (int j = 0; j < TAPS; ++j) {
+        const float4 v = *reinterpret_cast<const float4*>(p.conv_w + (int64_t)chan * TAPS + 4 * j);
+        w[4 * j] = v.x; w[4 * j + 1] = v.y; w[4 * j + 2] = v.z; w[4 * j + 3] = v.w;
     }
+    const bool scalars = is_v && l == 0 && in_range;    // this lane also makes its head's write strength and decay
     float A = 0.f, bias = 0.f;
-    const int vh = h - 2 * p.KH;
-    if (is_v && l == 0 && in_range) {
+    if (scalars) {
         A = expf(p.A_log[vh]);
         bias = p.dt_bias[vh];
     }
-    float4 past[PAST];
+    pdl_wait();
+    pdl_trigger();
+    float4 in[TPT + PAST];                              // inputs of tokens t0 - PAST .. t0 + TPT - 1
 #pragma unroll
-    for (int j = 0; j < PAST; ++j) past[j] = zero;
-    for (int k = 0; k < tpt; ++k) {
-        const int64_t t = t_first + k;
+    for (int q = 0; q < TPT + PAST; ++q) {
+        const int t = min(max(t0 + q - PAST, 0), p.tokens - 1);
+        in[q] = Vec4<T>::load(p.in + (int64_t)t * p.ld + chan);
+    }
+#pragma unroll
+    for (int q = 0; q < TPT; ++q) {
+        const int64_t t = t0 + q;
         const bool active = lane_on && t < p.tokens;
-        float4 x = zero;
-        if (active) {
-            const T* src = p.in + t * p.ld + chan;
-            const float4 own = Vec4<T>::load(src);
-            if constexpr (TAPS == 0) {
-                x = own;
-            } else {
-                if constexpr (TAPS > 1) {
-                    const int r = p.token_row[t];
-                    const int first = p.row_start[r];
-                    const int i0 = (int)t - first;
-                    if (k == 0 || i0 == 0) {
-                        float* cstate = p.state + (int64_t)p.row_slot[r] * p.slot_stride + p.conv_off + chan;
-                        const bool shift = p.update_single && p.row_start[r + 1] - first == 1;
+        float4 x = in[q + PAST];
+        if constexpr (TAPS > 0) {
+            x = zero;
+            if constexpr (PAST > 0) {
+                const int r = p.token_row[min((int)t, p.tokens - 1)];
+                const int first = p.row_start[r], i0 = min((int)t, p.tokens - 1) - first;
+                float* cstate = i0 < PAST ? p.state + (int64_t)p.row_slot[r] * p.slot_stride + p.conv_off + chan : nullptr;
+                float4 before[PAST];
 #pragma unroll
-                        for (int j = 0; j < TAPS - 1; ++j) {
-                            const int idx = i0 - (TAPS - 1) + j;          // negative: before the step
-                            past[j] = idx >= 0 ? Vec4<T>::load(src + (int64_t)(idx - i0) * p.ld)
-                                               : *reinterpret_cast<const float4*>(cstate + (int64_t)(TAPS - 1 + idx) * C);
-                            if (shift && j > 0) *reinterpret_cast<float4*>(cstate + (int64_t)(j - 1) * C) = past[j];
-                        }
-                        if (shift) *reinterpret_cast<float4*>(cstate + (int64_t)(TAPS - 2) * C) = own;
-                    }
-#pragma unroll
-                    for (int j = 0; j < TAPS - 1; ++j) {
-                        x.x = fmaf(w[j], past[j].x, x.x);
-                        x.y = fmaf(w[TAPS + j], past[j].y, x.y);
-                        x.z = fmaf(w[2 * TAPS + j], past[j].z, x.z);
-                        x.w = fmaf(w[3 * TAPS + j], past[j].w, x.w);
-                    }
-#pragma unroll
-                    for (int j = 0; j < TAPS - 2; ++j) past[j] = past[j + 1];
-                    past[PAST - 1] = own;
+                for (int j = 0; j < PAST; ++j) {        // index within the row i0 - PAST + j; negative: before the step
+                    float4 u = in[q + j];
+                    if (i0 - PAST + j < 0) u = *reinterpret_cast<const float4*>(cstate + (int64_t)(i0 + j) * C);
+                    before[j] = u;
+                    x.x = fmaf(w[j], u.x, x.x);
+                    x.y = fmaf(w[TAPS + j], u.y, x.y);
+                    x.z = fmaf(w[2 * TAPS + j], u.z, x.z);
+                    x.w = fmaf(w[3 * TAPS + j], u.w, x.w);
                 }
-                x.x = fmaf(w[TAPS - 1], own.x, x.x);
-                x.y = fmaf(w[2 * TAPS - 1], own.y, x.y);
-                x.z = fmaf(w[3 * TAPS - 1], own.z, x.z);
-                x.w = fmaf(w[4 * TAPS - 1], own.w, x.w);
+                if (active && p.update_single && i0 == 0 && p.row_start[r + 1] - first == 1) {
+                    // the row's only token: a lane alone reads and writes its channels
+#pragma unroll
+                    for (int j = 1; j < PAST; ++j) *reinterpret_cast<float4*>(cstate + (int64_t)(j - 1) * C) = before[j];
+                    *reinterpret_cast<float4*>(cstate + (int64_t)(PAST - 1) * C) = in[q + PAST];
+                }
             }
-            x.x *= rh_sigmoid(x.x); x.y *= rh_sigmoid(x.y); x.z *= rh_sigmoid(x.z); x.w *= rh_sigmoid(x.w);
+            x.x = fmaf(w[TAPS - 1], in[q + PAST].x, x.x);
+            x.y = fmaf(w[2 * TAPS - 1], in[q + PAST].y, x.y);
+            x.z = fmaf(w[3 * TAPS - 1], in[q + PAST].z, x.z);
+            x.w = fmaf(w[4 * TAPS - 1], in[q + PAST].w, x.w);
         }
+        x.x *= rh_sigmoid(x.x); x.y *= rh_sigmoid(x.y); x.z *= rh_sigmoid(x.z); x.w *= rh_sigmoid(x.w);
         // every lane of the warp takes part in the sums, whatever its head is
-        float ss = x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+        float ss = lane_on ? x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w : 0.f;
         for (int o = (1 << lph_log2) >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-        if (active) {
-            float* dst;
-            if (is_v) {
-                dst = p.vv + (t * p.H + vh) * p.vdim;
-                if (l == 0) {
-                    p.beta[t * p.H + vh] = rh_sigmoid(to_float(p.in[t * p.ld + p.beta0 + vh]));
-                    const float lg = -A * rh_softplus(to_float(p.in[t * p.ld + p.decay0 + vh]) + bias);
-                    p.g[t * p.H + vh] = expf(lg);
-                    p.log_g[t * p.H + vh] = lg;
-                }
-            } else {
-                const bool is_q = h < p.KH;
-                const float f = rsqrtf(ss + 1e-6f) * (is_q ? rsqrtf((float)p.dim) : 1.f);
-                x = make_float4(x.x * f, x.y * f, x.z * f, x.w * f);
-                dst = is_q ? p.qn + (t * p.KH + h) * p.dim : p.kn + (t * p.KH + h - p.KH) * p.dim;
+        if (!active) continue;
+        float* dst;
+        if (is_v) {
+            dst = p.vv + (t * p.H + vh) * p.vdim;
+            if (scalars) {
+                p.beta[t * p.H + vh] = rh_sigmoid(to_float(p.in[t * p.ld + p.beta0 + vh]));
+                const float lg = -A * rh_softplus(to_float(p.in[t * p.ld + p.decay0 + vh]) + bias);
+                p.g[t * p.H + vh] = expf(lg);
+                p.log_g[t * p.H + vh] = lg;
             }
-            *reinterpret_cast<float4*>(dst + 4 * l) = x;
+        } else {
+            const bool is_q = h < p.KH;
+            const float f = rsqrtf(ss + 1e-6f) * (is_q ? rsqrtf((float)p.dim) : 1.f);
+            x = make_float4(x.x * f, x.y * f, x.z * f, x.w * f);
+            dst = is_q ? p.qn + (t * p.KH + h) * p.dim : p.kn + (t * p.KH + h - p.KH) * p.dim;
         }
+        *reinterpret_cast<float4*>(dst + 4 * l) = x;
     }
 }
 
@@ -206,11 +198,12 @@ template <typename T, int TAPS> static int launch_delta_heads_vec(const DeltaHea
     const int widest = p.dim > p.vdim ? p.dim : p.vdim;
     int lph_log2 = 0;
     while ((4 << lph_log2) < widest) ++lph_log2;
-    const int tpt = p.tokens > 1024 ? 8 : (p.tokens > 256 ? 4 : 1);
+    const int tpt = p.tokens > 256 ? 4 : 1;
     const int64_t threads = (((int64_t)p.tokens + tpt - 1) / tpt * (2 * p.KH + p.H)) << lph_log2;
     const int block = threads >= 256 ? 256 : 128;
-    return acorn_launch(delta_heads_prep_vec_kernel<T, TAPS>, dim3((unsigned)((threads + block - 1) / block)), dim3(block), 0, stream,
-                        p, lph_log2, tpt);
+    const dim3 grid((unsigned)((threads + block - 1) / block));
+    if (tpt == 1) return acorn_launch(delta_heads_prep_vec_kernel<T, TAPS, 1>, grid, dim3(block), 0, stream, p, lph_log2);
+    return acorn_launch(delta_heads_prep_vec_kernel<T, TAPS, 4>, grid, dim3(block), 0, stream, p, lph_log2);
 }
 
 template <typename T> static int launch_delta_heads(const DeltaHeadsParams<T>& p, cudaStream_t stream) {

@@ -211,7 +211,7 @@ def test_long_requests_over_pages_and_segments(tmp_path):
             check(got, ref, dtype, f"long, {cut}")
 
 
-@pytest.mark.parametrize("seed", [1, 4, 6, 11, 13])
+@pytest.mark.parametrize("seed", [1, 4, 6, 12, 13])
 def test_configurations_drawn_at_random(seed, tmp_path):
     """Models whose sizes are drawn from what real models have, requests of up to 200 tokens, whole, with a decoded
     tail and mixed in a small pool, float32 and bfloat16."""
