@@ -181,7 +181,8 @@ __global__ void __launch_bounds__(512) hyper_norm_kernel(const HyperParams<T> p)
 
 template <typename T, int N> static int launch_hyper_vec(const HyperParams<T>& p, int rows, cudaStream_t stream) {
     const int n4 = p.H / 4;
-    const int most = rows <= 148 ? 512 : 256;            // few rows: more threads a row; many: more rows at a time
+    const int most = rows <= 148 || N >= 3 ? 512 : 256;  // few rows: more threads a row; many: more rows at a time, unless a
+                                                         // thread's vectors of all streams would take too many registers
     const int nv = (n4 + most - 1) / most;
     const int per = nv <= 1 ? 1 : (nv <= 2 ? 2 : 4);
     const int threads = ((n4 + per - 1) / per + 31) / 32 * 32;
