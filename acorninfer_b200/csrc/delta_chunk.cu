@@ -208,37 +208,45 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_solve_kernel(const DeltaCh
     }
 }
 
+// Both products of a chunk have few outputs (64 x 16 and dim x 16) and a long sum, so a warp takes a slice of the sum for large
+// register tiles (8 x 4 a lane: three reads of shared memory for 32 multiply-adds) and the slices are added up through
+// shared memory: U over 8 slices of the key channels, the state over 4 slices of the tokens by 2 halves of the channels.
 template <int DP>
 __global__ void __launch_bounds__(256) delta_chunk_state_kernel(const DeltaChunkParams p) {
-    constexpr int LD = DP + DC_PAD, HALF = DP / 2;
+    constexpr int LD = DP + DC_PAD, LV = DC_VT + DC_PAD, SLICE = DP / 8, ND = DP / 64 > 0 ? DP / 64 : 1;
+    constexpr int PARTS = 8 * DC > 4 * DP ? 8 * DC : 4 * DP;
     extern __shared__ __align__(16) float sm[];
     float* sW = sm;                                     // [2][DC][LD]
     float* sK = sW + 2 * DC * LD;                       // [2][DC][LD]
-    float* sS = sK + 2 * DC * LD;                       // [DC_VT][LD]: the state's columns
-    float2* sU = reinterpret_cast<float2*>(sS + DC_VT * LD);      // [DC][8]: columns c and c + 8 of a token's u, times G_nj
-    float* part = reinterpret_cast<float*>(sU + DC * 8);          // [8][128] the upper half's sums
+    float* sS = sK + 2 * DC * LD;                       // [DP][LV] the state's tile
+    float* sU = sS + DP * LV;                           // [DC][LV] a token's u times G_nj
+    float* part = sU + DC * LV;                         // [PARTS][LV] slices of the sums
     pdl_wait();
     pdl_trigger();
     const int h = blockIdx.y, r = blockIdx.z, kh = h / (p.H / p.KH), v0 = blockIdx.x * DC_VT, tid = threadIdx.x;
+    const int lane = tid & 31, warp = tid >> 5, rg = lane >> 2, cg = lane & 3;
     const int start = p.row_start[r], L = p.row_start[r + 1] - start;
     const int chunks = (L + DC - 1) / DC, id0 = start / DC + r;
-    const int cp = tid & 7;                             // this thread's columns: cp and cp + 8 of the tile
-    const int col0 = v0 + cp, col1 = v0 + cp + 8;
-    const bool on0 = col0 < p.vdim, on1 = col1 < p.vdim;
-    const int dg = tid >> 3;                            // its state entries: key channels 4 dg .. 4 dg + 3
-    const bool holds = 4 * dg < DP;
+    const int c4 = v0 + 4 * (tid & 3);                  // this thread's four columns when sums are collected
+    const bool on = c4 < p.vdim;
     float* slot = p.state + (int64_t)p.row_slot[r] * p.slot_stride + (int64_t)h * p.dim * p.vdim;
-    float S0[4], S1[4];
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    // the state entries this thread keeps: key channels (tid + 256 m) / 4, columns c4 ..
+    float4 S[ND];
 #pragma unroll
-    for (int q = 0; q < 4; ++q) {
-        const int d = 4 * dg + q;
-        S0[q] = holds && d < p.dim && on0 ? slot[(int64_t)d * p.vdim + col0] : 0.f;
-        S1[q] = holds && d < p.dim && on1 ? slot[(int64_t)d * p.vdim + col1] : 0.f;
+    for (int m = 0; m < ND; ++m) {
+        const int d = (tid + 256 * m) >> 2;
+        S[m] = zero;
+        if (d < p.dim && on) {                          // (a slot starts wherever it may: no vector reads)
+            const float* at = slot + (int64_t)d * p.vdim + c4;
+            S[m] = make_float4(at[0], at[1], at[2], at[3]);
+        }
     }
     auto publish = [&]() {
-        if (holds) {
-            *reinterpret_cast<float4*>(sS + cp * LD + 4 * dg) = make_float4(S0[0], S0[1], S0[2], S0[3]);
-            *reinterpret_cast<float4*>(sS + (cp + 8) * LD + 4 * dg) = make_float4(S1[0], S1[1], S1[2], S1[3]);
+#pragma unroll
+        for (int m = 0; m < ND; ++m) {
+            const int d = (tid + 256 * m) >> 2;
+            if (d < DP) *reinterpret_cast<float4*>(sS + d * LV + 4 * (tid & 3)) = S[m];
         }
     };
     publish();
@@ -247,100 +255,103 @@ __global__ void __launch_bounds__(256) delta_chunk_state_kernel(const DeltaChunk
         load_rows<DP>(sW + (c & 1) * DC * LD, p.w + ((int64_t)first * p.H + h) * p.dim, (int64_t)p.H * p.dim, n, p.dim);
         load_rows<DP>(sK + (c & 1) * DC * LD, p.k + ((int64_t)first * p.KH + kh) * p.dim, (int64_t)p.KH * p.dim, n, p.dim);
     };
+    auto axpy = [](float a, const float4& x, float4& y) {
+        y.x = fmaf(a, x.x, y.x); y.y = fmaf(a, x.y, y.y); y.z = fmaf(a, x.z, y.z); y.w = fmaf(a, x.w, y.w);
+    };
+    auto add = [](float4& y, const float4& x) { y.x += x.x; y.y += x.y; y.z += x.z; y.w += x.w; };
     if (chunks > 0) fetch(0);
     asm volatile("cp.async.commit_group;\n" ::);
-    const int half = tid >> 7, ig = (tid & 127) >> 3;   // rows ig + 16 rr over key channels half * HALF ..
+    const int token = tid >> 2;                         // the token whose u this thread collects
     for (int c = 0; c < chunks; ++c) {
         const int first = start + c * DC, n = min(DC, L - c * DC);
-        float ub0[4], ub1[4], bj[4];
         const float bn = p.b[(int64_t)(first + n - 1) * p.H + h];
-        if (half == 0) {
-#pragma unroll
-            for (int rr = 0; rr < 4; ++rr) {
-                const int i = ig + 16 * rr;
-                const int64_t t = (int64_t)(first + min(i, n - 1)) * p.H + h;
-                ub0[rr] = i < n && on0 ? p.u[t * p.vdim + col0] : 0.f;
-                ub1[rr] = i < n && on1 ? p.u[t * p.vdim + col1] : 0.f;
-                bj[rr] = p.b[t];
-            }
-        }
+        const int64_t t = (int64_t)(first + min(token, n - 1)) * p.H + h;
+        const bool live = token < n && on;
+        const float4 ub = live ? *reinterpret_cast<const float4*>(p.u + t * p.vdim + c4) : zero;
+        const float bj = p.b[t];
         if (c + 1 < chunks) fetch(c + 1);
         asm volatile("cp.async.commit_group;\n" ::);
         float* keep = p.s0 + ((int64_t)(id0 + c) * p.H + h) * p.dim * p.vdim;      // the state this chunk starts from
 #pragma unroll
-        for (int q = 0; q < 4; ++q) {
-            const int d = 4 * dg + q;
-            if (holds && d < p.dim) {
-                if (on0) keep[(int64_t)d * p.vdim + col0] = S0[q];
-                if (on1) keep[(int64_t)d * p.vdim + col1] = S1[q];
-            }
+        for (int m = 0; m < ND; ++m) {
+            const int d = (tid + 256 * m) >> 2;
+            if (d < p.dim && on) *reinterpret_cast<float4*>(keep + (int64_t)d * p.vdim + c4) = S[m];
         }
         asm volatile("cp.async.wait_group 1;\n" ::);
-        __syncthreads();                                // this chunk's rows and the state's columns are there
-        const float* W = sW + (c & 1) * DC * LD;
-        const float* K = sK + (c & 1) * DC * LD;
-        float a0[4] = {0.f, 0.f, 0.f, 0.f}, a1[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 4
-        for (int d = half * HALF; d < half * HALF + HALF; d += 4) {
-            const float4 s0 = *reinterpret_cast<const float4*>(sS + cp * LD + d);
-            const float4 s1 = *reinterpret_cast<const float4*>(sS + (cp + 8) * LD + d);
+        __syncthreads();                                // this chunk's rows and the state's tile are there
+        {
+            const float* W = sW + (c & 1) * DC * LD + warp * SLICE;
+            float4 acc[8];
 #pragma unroll
-            for (int rr = 0; rr < 4; ++rr) {
-                const float4 w = *reinterpret_cast<const float4*>(W + (ig + 16 * rr) * LD + d);
-                a0[rr] = dot4(w, s0, a0[rr]);
-                a1[rr] = dot4(w, s1, a1[rr]);
-            }
-        }
-        if (half == 1) {
+            for (int rr = 0; rr < 8; ++rr) acc[rr] = zero;
 #pragma unroll
-            for (int rr = 0; rr < 4; ++rr) {
-                part[rr * 128 + (tid & 127)] = a0[rr];
-                part[(4 + rr) * 128 + (tid & 127)] = a1[rr];
-            }
-        }
-        __syncthreads();
-        if (half == 0) {
+            for (int d = 0; d < SLICE; d += 4) {
+                float4 s[4];
 #pragma unroll
-            for (int rr = 0; rr < 4; ++rr) {
-                const int i = ig + 16 * rr;
-                const float u0 = ub0[rr] - (a0[rr] + part[rr * 128 + tid]), u1 = ub1[rr] - (a1[rr] + part[(4 + rr) * 128 + tid]);
-                const float G = i < n ? expf(bn - bj[rr]) : 0.f;
-                sU[i * 8 + cp] = make_float2(u0 * G, u1 * G);
-                if (i < n) {
-                    const int64_t t = ((int64_t)(first + i) * p.H + h) * p.vdim;
-                    if (on0) p.u[t + col0] = u0;
-                    if (on1) p.u[t + col1] = u1;
+                for (int q = 0; q < 4; ++q) s[q] = *reinterpret_cast<const float4*>(sS + (warp * SLICE + d + q) * LV + 4 * cg);
+#pragma unroll
+                for (int rr = 0; rr < 8; ++rr) {
+                    const float4 w = *reinterpret_cast<const float4*>(W + (rg + 8 * rr) * LD + d);
+                    axpy(w.x, s[0], acc[rr]); axpy(w.y, s[1], acc[rr]); axpy(w.z, s[2], acc[rr]); axpy(w.w, s[3], acc[rr]);
                 }
             }
+#pragma unroll
+            for (int rr = 0; rr < 8; ++rr) *reinterpret_cast<float4*>(part + (warp * DC + rg + 8 * rr) * LV + 4 * cg) = acc[rr];
         }
         __syncthreads();
-        if (holds) {
-            const float gn = expf(bn);
+        {
+            float4 u = zero;
 #pragma unroll
-            for (int q = 0; q < 4; ++q) {
-                S0[q] *= gn;
-                S1[q] *= gn;
-            }
+            for (int q = 0; q < 8; ++q) add(u, *reinterpret_cast<const float4*>(part + (q * DC + token) * LV + 4 * (tid & 3)));
+            u = make_float4(ub.x - u.x, ub.y - u.y, ub.z - u.z, ub.w - u.w);
+            if (live) *reinterpret_cast<float4*>(p.u + t * p.vdim + c4) = u;
+            const float G = token < n ? expf(bn - bj) : 0.f;
+            *reinterpret_cast<float4*>(sU + token * LV + 4 * (tid & 3)) = make_float4(u.x * G, u.y * G, u.z * G, u.w * G);
+        }
+        __syncthreads();
+        {
+            const int jg = warp >> 1, d0 = (warp & 1) * (DP / 2) + 4 * rg;         // key channels d0 + 32 m .. + 3
+            if (4 * rg < DP / 2) {
+                const float* K = sK + (c & 1) * DC * LD + jg * 16 * LD + d0;
+                float4 acc[ND][4];
+#pragma unroll
+                for (int m = 0; m < ND; ++m)
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) acc[m][q] = zero;
 #pragma unroll 8
-            for (int j = 0; j < DC; ++j) {
-                const float4 k = *reinterpret_cast<const float4*>(K + j * LD + 4 * dg);
-                const float2 u = sU[j * 8 + cp];
-                S0[0] = fmaf(k.x, u.x, S0[0]); S1[0] = fmaf(k.x, u.y, S1[0]);
-                S0[1] = fmaf(k.y, u.x, S0[1]); S1[1] = fmaf(k.y, u.y, S1[1]);
-                S0[2] = fmaf(k.z, u.x, S0[2]); S1[2] = fmaf(k.z, u.y, S1[2]);
-                S0[3] = fmaf(k.w, u.x, S0[3]); S1[3] = fmaf(k.w, u.y, S1[3]);
+                for (int j = 0; j < 16; ++j) {
+                    const float4 u = *reinterpret_cast<const float4*>(sU + (jg * 16 + j) * LV + 4 * cg);
+#pragma unroll
+                    for (int m = 0; m < ND; ++m) {
+                        const float4 k = *reinterpret_cast<const float4*>(K + j * LD + 32 * m);
+                        axpy(k.x, u, acc[m][0]); axpy(k.y, u, acc[m][1]); axpy(k.z, u, acc[m][2]); axpy(k.w, u, acc[m][3]);
+                    }
+                }
+#pragma unroll
+                for (int m = 0; m < ND; ++m)
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) *reinterpret_cast<float4*>(part + (jg * DP + d0 + 32 * m + q) * LV + 4 * cg) = acc[m][q];
             }
         }
-        publish();                                      // (the last reads of the columns lie two barriers back)
-        __syncthreads();                                // this chunk's rows may be overwritten
+        __syncthreads();
+        const float gn = expf(bn);
+#pragma unroll
+        for (int m = 0; m < ND; ++m) {
+            const int d = (tid + 256 * m) >> 2;
+            if (d >= DP) break;
+            S[m] = make_float4(S[m].x * gn, S[m].y * gn, S[m].z * gn, S[m].w * gn);
+#pragma unroll
+            for (int q = 0; q < 4; ++q) add(S[m], *reinterpret_cast<const float4*>(part + (q * DP + d) * LV + 4 * (tid & 3)));
+        }
+        publish();
     }
     asm volatile("cp.async.wait_group 0;\n" ::);
 #pragma unroll
-    for (int q = 0; q < 4; ++q) {
-        const int d = 4 * dg + q;
-        if (holds && d < p.dim) {
-            if (on0) slot[(int64_t)d * p.vdim + col0] = S0[q];
-            if (on1) slot[(int64_t)d * p.vdim + col1] = S1[q];
+    for (int m = 0; m < ND; ++m) {
+        const int d = (tid + 256 * m) >> 2;
+        if (d < p.dim && on) {
+            float* at = slot + (int64_t)d * p.vdim + c4;
+            at[0] = S[m].x; at[1] = S[m].y; at[2] = S[m].z; at[3] = S[m].w;
         }
     }
 }
@@ -432,7 +443,8 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_out_kernel(const DeltaChun
 template <int DP> static int launch_delta_chunk(const DeltaChunkParams& p, int ids, cudaStream_t stream) {
     constexpr int LD = DP + DC_PAD;
     const size_t solve = (size_t)(2 * DC * LD + DC * (DC + DC_PAD)) * sizeof(float);
-    const size_t walk = (size_t)(4 * DC * LD + DC_VT * LD + DC * 16 + 8 * 128) * sizeof(float);
+    constexpr int LV = DC_VT + DC_PAD, PARTS = 8 * DC > 4 * DP ? 8 * DC : 4 * DP;
+    const size_t walk = (size_t)(4 * DC * LD + (DP + DC + PARTS) * LV) * sizeof(float);
     const size_t out = (size_t)(DC * LD + DP * (DC_OT + DC_PAD) + DC * (DC_OT + DC_PAD) + DC * (DC + DC_PAD)) * sizeof(float);
     static AcornPerDevice configured;
     if (!configured.seen()) {
